@@ -3,15 +3,15 @@
 A sequence gets a slot when it starts and gives it back when it ends; slots and pages are
 reused.  Layers are grouped by what they need:
 
-* a KV group per distinct (kv heads, key head size, value head size, window): pools of pages of
+* a KV group per distinct (kv heads, key head size, value head size, window, chunk): pools of pages of
   `page_size` positions, keys `[entry, page, kv_head, position in page, head_dim]` and values
   `[entry, page, kv_head, value_dim, position in page]`, with a page pool and a page list per
   sequence of its own.  A windowed group gives pages back once every position in
-  them has left the window.
+  them has left the window, or lies in a chunk before the next position's.
   A group whose spec pools blocks of positions has a second pair of pools of the same layout, one row per
   complete block, with pages and a page list per sequence of their own; they are never given back before
   the sequence ends.
-* a latent group per distinct (rank, rotated key width) is a KV group with one "head" whose key row is
+* a latent group per distinct (rank, rotated key width, window, chunk) is a KV group with one "head" whose key row is
   the cached row `[latent | rotated key part]` and whose value pool is empty (the values are read out
   of the same row); pages, tables, export and import are those of any KV group.
 * a state group per distinct (shape, dtype): `[entry, slot, *shape]`, zeroed when a slot is
@@ -101,11 +101,12 @@ class KVGroup:
                 self.pooled_pages.alloc_many(self.pooled_pages_needed(slot, new_len)))
 
     def trim(self, slot: int, length: int) -> None:
-        """Gives back the pages no later query can reach (windowed groups only)."""
-        w = self.spec.window
-        if w <= 0:
+        """Gives back the pages no later query can reach (windowed and chunked groups only)."""
+        w, c = self.spec.window, self.spec.chunk
+        if w <= 0 and c <= 0:
             return
-        first_needed = length + 1 - w     # the next query, at position `length`, reaches back to here
+        # the next query, at position `length`, reaches back to here
+        first_needed = max(length + 1 - w if w > 0 else 0, length // c * c if c > 0 else 0)
         if self.pool > 0:                 # the block that is still filling is pooled from its cached rows
             first_needed = min(first_needed, length // self.pool * self.pool)
         lst = self.seq_pages.get(slot, [])

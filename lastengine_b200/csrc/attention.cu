@@ -8,7 +8,9 @@
 // Math as the reference (src/dense.rs:129-146): for query head h the kv head is h / (nh/nkv);
 // score_t = (q . k_t) / sqrt(head_dim) for t in [t0, pos], t0 = pos+1-window when the layer has a
 // window and pos+1 > window, else 0; softmax with the maximum subtracted; o = sum_t p_t v_t.
-// An optional per-head gate multiplies the head's output by sigmoid(gate) (src/dense.rs:147-150).
+// An optional per-head gate multiplies the head's output by sigmoid(gate) (src/dense.rs:147-150); it may also be
+// given per dimension of the head.  Instead of a window a layer may cut its positions into chunks (t0 = the start
+// of pos's chunk).
 // Scores, maximum, exponentials, sums and the value accumulation are float.  The reference's
 // GPU kernels keep the same running (max, sum, acc) per warp and merge them
 // (src/cuda/dense.cu:94-123 whole range, :152-183 split range, :238-247 merge); this kernel lets
@@ -31,8 +33,8 @@ attention_kernel(T* __restrict__ out, float* __restrict__ part, const T* __restr
                  const int* __restrict__ block_table, int bt_width,
                  const int* __restrict__ seq_slot, const int* __restrict__ seq_pos0,
                  const int* __restrict__ seq_qstart, const int* __restrict__ seq_qlen,
-                 const T* __restrict__ gate, int gate_stride, int nh, int nkv, int hd, int vd,
-                 int page_size, int window, float scale, int QT, int HC, int n_splits) {
+                 const T* __restrict__ gate, int gate_stride, int gate_elem, int nh, int nkv, int hd, int vd,
+                 int page_size, int window, int chunk, float scale, int QT, int HC, int n_splits) {
   extern __shared__ float sm[];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int G = nh / nkv;
@@ -86,7 +88,7 @@ attention_kernel(T* __restrict__ out, float* __restrict__ part, const T* __restr
   // keys this block may need: up to the last row's position, from the first row's window start
   const int kv_len = pos0 + qlen;  // keys the cache holds for this sequence after this step's writes
   const int pos_lo = pos0 + row_lo, pos_hi = pos0 + row_lo + nrows - 1;
-  const int key_lo = (window > 0 && pos_lo + 1 > window) ? pos_lo + 1 - window : 0;
+  const int key_lo = first_key(pos_lo, window, chunk);
   const int tile_first = key_lo / 32, tile_last = pos_hi / 32;
   const int n_tiles = tile_last - tile_first + 1;
   const int per_split = (n_tiles + n_splits - 1) / n_splits;
@@ -128,13 +130,15 @@ attention_kernel(T* __restrict__ out, float* __restrict__ part, const T* __restr
       const int i = r / HC, j = r % HC;
       if (i >= nrows || j >= nheads) continue;
       const int qpos = pos0 + row_lo + i;
+      const int lo = first_key(qpos, window, chunk);
+      if (key0 > qpos || key0 + 31 < lo) continue;   // the whole tile lies after this row, or before what it reads
       const float* qv = q_s + r * hd;
       const float* kr = k_s + lane * KS;
       float s = 0.f;
       for (int d = 0; d < hd; d++) s += qv[d] * kr[d];
       s *= scale;
       const int kp = key0 + lane;
-      const bool valid = kp <= qpos && (window <= 0 || kp + window > qpos);
+      const bool valid = kp <= qpos && kp >= lo;
       s = valid ? s : ATT_NEG;
       const float mn = fmaxf(mx[ri], warp_max(s));
       const float p = valid ? expf(s - mn) : 0.f;
@@ -166,16 +170,14 @@ attention_kernel(T* __restrict__ out, float* __restrict__ part, const T* __restr
     const int h = kvh * G + hc * HC + j;
     const size_t m = (size_t)q0 + row_lo + i;
     if (n_splits == 1) {
-      float g = 1.f;
-      if (gate) {
-        float z = to_f32(gate[m * gate_stride + h]);
-        g = 1.0f / (1.0f + expf(-z));
-      }
       const float inv = l[ri] > 0.f ? 1.0f / l[ri] : 0.f;
 #pragma unroll
       for (int jj = 0; jj < HDL; jj++) {
         const int d = lane + 32 * jj;
-        if (d < vd) out[(m * nh + h) * vd + d] = from_f32<T>(acc[ri][jj] * inv * g);
+        if (d < vd) {
+          const float g = gate ? head_gate(gate, m, gate_stride, h, d, vd, gate_elem) : 1.f;
+          out[(m * nh + h) * vd + d] = from_f32<T>(acc[ri][jj] * inv * g);
+        }
       }
     } else {
       float* pp = part + ((m * nh + h) * n_splits + split) * (size_t)(vd + 2);
@@ -195,15 +197,14 @@ attention_kernel(T* __restrict__ out, float* __restrict__ part, const T* __restr
 // (with more, the running sums are rescaled to the new maximum from group to group).
 template <typename T>
 __global__ void attention_merge_kernel(T* __restrict__ out, const float* __restrict__ part,
-                                       const T* __restrict__ gate, int gate_stride, int nh, int hd,
-                                       int n_splits) {
+                                       const T* __restrict__ gate, int gate_stride, int gate_elem, int nh,
+                                       int hd, int n_splits) {
   pdl_trigger();   // the kernel after this one may start and wait (see common.cuh)
   pdl_wait();
   const size_t m = blockIdx.x;
   const int h = blockIdx.y;
   const size_t step = hd + 2;
   const float* pp = part + ((m * nh + h) * n_splits) * step;
-  const float z = gate ? to_f32(gate[m * gate_stride + h]) : 0.f;
   for (int d = threadIdx.x; d < hd; d += blockDim.x) {
     float M = ATT_NEG, L = 0.f, a = 0.f;
     for (int s0 = 0; s0 < n_splits; s0 += 8) {
@@ -230,7 +231,7 @@ __global__ void attention_merge_kernel(T* __restrict__ out, const float* __restr
       }
       M = cm;
     }
-    const float g = gate ? 1.0f / (1.0f + expf(-z)) : 1.f;
+    const float g = gate ? head_gate(gate, m, gate_stride, h, d, hd, gate_elem) : 1.f;
     out[(m * nh + h) * hd + d] = from_f32<T>(a * (L > 0.f ? 1.0f / L : 0.f) * g);
   }
 }
@@ -239,8 +240,8 @@ template <typename T, typename CT, int HDL>
 static int launch_attention(void* out, float* part, const void* q, const void* k_pool,
                             const void* v_pool, const int* block_table, int bt_width,
                             const int* seq_slot, const int* seq_pos0, const int* seq_qstart,
-                            const int* seq_qlen, const void* gate, int gate_stride, int B, int nh,
-                            int nkv, int hd, int vd, int page_size, int window, float scale, int max_qlen,
+                            const int* seq_qlen, const void* gate, int gate_stride, int gate_elem, int B, int nh,
+                            int nkv, int hd, int vd, int page_size, int window, int chunk, float scale, int max_qlen,
                             int n_splits, cudaStream_t st) {
   const int G = nh / nkv;
   const int HC = G < 8 ? G : 8;
@@ -260,8 +261,8 @@ static int launch_attention(void* out, float* part, const void* q, const void* k
   LEB_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "leb_attention: grid too large (%u, %u)", grid.y, grid.z);
   kern<<<grid, 32 * ATT_WARPS, smem, st>>>(
       (T*)out, part, (const T*)q, (const CT*)k_pool, (const CT*)v_pool, block_table, bt_width,
-      seq_slot, seq_pos0, seq_qstart, seq_qlen, (const T*)gate, gate_stride, nh, nkv, hd, vd, page_size,
-      window, scale, QT, HC, n_splits);
+      seq_slot, seq_pos0, seq_qstart, seq_qlen, (const T*)gate, gate_stride, gate_elem, nh, nkv, hd, vd, page_size,
+      window, chunk, scale, QT, HC, n_splits);
   LEB_CHECK_LAUNCH("leb_attention");
   return 0;
 }
@@ -272,8 +273,8 @@ static int launch_attention(void* out, float* part, const void* q, const void* k
 LEB_API int leb_attention(void* out, float* part, const void* q, const void* k_pool,
                           const void* v_pool, int dtype, const int* block_table, int bt_width,
                           const int* seq_slot, const int* seq_pos0, const int* seq_qstart,
-                          const int* seq_qlen, const void* gate, int gate_stride, int M, int B,
-                          int nh, int nkv, int hd, int page_size, int window, float scale,
+                          const int* seq_qlen, const void* gate, int gate_stride, int gate_elem, int M, int B,
+                          int nh, int nkv, int hd, int page_size, int window, int chunk, float scale,
                           int max_qlen, int n_splits, int vd, cudaStream_t st) {
   if (M <= 0 || B <= 0) return 0;
   if (vd <= 0) vd = hd;
@@ -283,23 +284,12 @@ LEB_API int leb_attention(void* out, float* part, const void* q, const void* k_p
   LEB_REQUIRE(page_size % 32 == 0, "leb_attention: page size %d is not a multiple of 32", page_size);
   LEB_REQUIRE(n_splits >= 1 && (n_splits == 1 || (max_qlen == 1 && part)), "leb_attention: splits need single-row sequences and scratch");
   int rc;
-#define LEB_ATT(T, CT)                                                                            \
-  (vd <= 32    ? launch_attention<T, CT, 1>(out, part, q, k_pool, v_pool, block_table, bt_width,  \
-                                            seq_slot, seq_pos0, seq_qstart, seq_qlen, gate,       \
-                                            gate_stride, B, nh, nkv, hd, vd, page_size, window,      \
-                                            scale, max_qlen, n_splits, st)                        \
-   : vd <= 64  ? launch_attention<T, CT, 2>(out, part, q, k_pool, v_pool, block_table, bt_width,  \
-                                            seq_slot, seq_pos0, seq_qstart, seq_qlen, gate,       \
-                                            gate_stride, B, nh, nkv, hd, vd, page_size, window,      \
-                                            scale, max_qlen, n_splits, st)                        \
-   : vd <= 128 ? launch_attention<T, CT, 4>(out, part, q, k_pool, v_pool, block_table, bt_width,  \
-                                            seq_slot, seq_pos0, seq_qstart, seq_qlen, gate,       \
-                                            gate_stride, B, nh, nkv, hd, vd, page_size, window,      \
-                                            scale, max_qlen, n_splits, st)                        \
-               : launch_attention<T, CT, 8>(out, part, q, k_pool, v_pool, block_table, bt_width,  \
-                                            seq_slot, seq_pos0, seq_qstart, seq_qlen, gate,       \
-                                            gate_stride, B, nh, nkv, hd, vd, page_size, window,      \
-                                            scale, max_qlen, n_splits, st))
+#define LEB_ATT_W(T, CT, HDL)                                                                                           \
+  launch_attention<T, CT, HDL>(out, part, q, k_pool, v_pool, block_table, bt_width, seq_slot, seq_pos0, seq_qstart,      \
+                               seq_qlen, gate, gate_stride, gate_elem, B, nh, nkv, hd, vd, page_size, window, chunk, scale, \
+                               max_qlen, n_splits, st)
+#define LEB_ATT(T, CT) \
+  (vd <= 32 ? LEB_ATT_W(T, CT, 1) : vd <= 64 ? LEB_ATT_W(T, CT, 2) : vd <= 128 ? LEB_ATT_W(T, CT, 4) : LEB_ATT_W(T, CT, 8))
   if (dtype == LEB_F32)
     rc = LEB_ATT(float, float);
   else if (dtype == LEB_BF16)
@@ -307,13 +297,14 @@ LEB_API int leb_attention(void* out, float* part, const void* q, const void* k_p
   else
     return leb_fail("leb_attention: unknown dtype %d", dtype);
 #undef LEB_ATT
+#undef LEB_ATT_W
   if (rc) return rc;
   if (n_splits > 1) {
     dim3 grid(M, nh);
     if (dtype == LEB_F32)
-      attention_merge_kernel<float><<<grid, 64, 0, st>>>((float*)out, part, (const float*)gate, gate_stride, nh, vd, n_splits);
+      attention_merge_kernel<float><<<grid, 64, 0, st>>>((float*)out, part, (const float*)gate, gate_stride, gate_elem, nh, vd, n_splits);
     else
-      attention_merge_kernel<bf16><<<grid, 64, 0, st>>>((bf16*)out, part, (const bf16*)gate, gate_stride, nh, vd, n_splits);
+      attention_merge_kernel<bf16><<<grid, 64, 0, st>>>((bf16*)out, part, (const bf16*)gate, gate_stride, gate_elem, nh, vd, n_splits);
     LEB_CHECK_LAUNCH("leb_attention merge");
   }
   return 0;
@@ -321,13 +312,13 @@ LEB_API int leb_attention(void* out, float* part, const void* q, const void* k_p
 
 // Merge of split partial results on its own (for kernels that write the same partial layout).
 LEB_API int leb_attention_merge(void* out, const float* part, int dtype, const void* gate,
-                                int gate_stride, int M, int nh, int hd, int n_splits, cudaStream_t st) {
+                                int gate_stride, int gate_elem, int M, int nh, int hd, int n_splits, cudaStream_t st) {
   if (M <= 0) return 0;
   dim3 grid(M, nh);
   if (dtype == LEB_F32)
-    attention_merge_kernel<float><<<grid, 64, 0, st>>>((float*)out, part, (const float*)gate, gate_stride, nh, hd, n_splits);
+    attention_merge_kernel<float><<<grid, 64, 0, st>>>((float*)out, part, (const float*)gate, gate_stride, gate_elem, nh, hd, n_splits);
   else if (dtype == LEB_BF16)
-    leb_launch(attention_merge_kernel<bf16>, grid, dim3(64), 0, st, (bf16*)out, part, (const bf16*)gate, gate_stride, nh, hd, n_splits);
+    leb_launch(attention_merge_kernel<bf16>, grid, dim3(64), 0, st, (bf16*)out, part, (const bf16*)gate, gate_stride, gate_elem, nh, hd, n_splits);
   else
     return leb_fail("leb_attention_merge: unknown dtype %d", dtype);
   LEB_CHECK_LAUNCH("leb_attention_merge");

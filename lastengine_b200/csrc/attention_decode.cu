@@ -56,6 +56,12 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
+// what bfloat16 left of (lo, hi) packed into `kept`
+__device__ __forceinline__ uint32_t rest_bf16(float lo, float hi, uint32_t kept) {
+  const __nv_bfloat162 k = *reinterpret_cast<const __nv_bfloat162*>(&kept);
+  return pack_bf16(lo - __bfloat162float(k.x), hi - __bfloat162float(k.y));
+}
+
 // zero the 16-bit halves of a value piece whose positions are outside [lo, hi)
 __device__ __forceinline__ uint4 mask_positions(uint4 v, int first, int lo, int hi) {
   uint32_t* w = reinterpret_cast<uint32_t*>(&v);
@@ -74,7 +80,8 @@ __device__ __forceinline__ uint4 mask_positions(uint4 v, int first, int lo, int 
 // block norms and rotates the query heads it needs, and the block whose key range ends with the
 // new position norms and rotates the new key, stores it and the new value in the cache, and only
 // then streams that range.  Same operations in the same order as qk_rope_store_lanes_kernel
-// (rope_cache.cu), so the two ways give the same bits.  Head sizes 64 and 128 with a split-half
+// (rope_cache.cu), so the two ways give the same bits (a norm over the whole row adds its squares in another
+// order than the row kernel there: the same up to a rounding of the sum).  Head sizes 64 and 128 with a
 // rotation over the whole head.
 struct AtdPrep {
   const bf16* q_raw;      // [rows, q_stride]
@@ -87,17 +94,46 @@ struct AtdPrep {
   const float* k_norm_w;
   const float* inv_freq;  // [HD / 2]
   float eps;
+  bool neox;              // pairs (i, i + HD/2), else (2i, 2i + 1)
+  bool row_norm;          // the root mean square of the whole row of heads, weights over the row ([nh HD], [nkv HD])
 };
 
-// One head vector by one warp: norm over the head, split-half rotation, rounded to bfloat16.
+// Sum of squares of n bfloat16 numbers by the whole block (n a multiple of 8, src on a 16-byte boundary or read one by
+// one); `red` holds a float per warp.
+__device__ __forceinline__ float atd_row_ss(const bf16* __restrict__ src, int n, float* red) {
+  float ss = 0.f;
+  if ((((uintptr_t)src) & 15) == 0) {
+    for (int i = threadIdx.x * 8; i < n; i += blockDim.x * 8) {
+      const uint4 w = *reinterpret_cast<const uint4*>(src + i);
+      const bf16* e = reinterpret_cast<const bf16*>(&w);
+#pragma unroll
+      for (int j = 0; j < 8; j++) ss += __bfloat162float(e[j]) * __bfloat162float(e[j]);
+    }
+  } else {
+    for (int i = threadIdx.x; i < n; i += blockDim.x) ss += __bfloat162float(src[i]) * __bfloat162float(src[i]);
+  }
+  ss = warp_sum(ss);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  ss = 0.f;
+  for (int w = 0; w < ATD_WARPS; w++) ss += red[w];
+  __syncthreads();
+  return ss;
+}
+
+// One head vector by one warp: norm over the head (or, with row_r > 0, by the row's factor), rotation, rounded to bfloat16.
 template <int HD>
 __device__ __forceinline__ void atd_prep_head(const bf16* __restrict__ src, const float* __restrict__ nw, float eps,
-                                              const float* cs, const float* sn, bf16* dst, int lane) {
+                                              const float* cs, const float* sn, bf16* dst, int lane, bool neox,
+                                              float row_r) {
   constexpr int EPL = HD / 32, NP = EPL / 2;
   float x[EPL];
 #pragma unroll
   for (int e = 0; e < EPL; e++) x[e] = __bfloat162float(src[lane + 32 * e]);
-  if (nw) {
+  if (row_r > 0.f) {
+#pragma unroll
+    for (int e = 0; e < EPL; e++) x[e] = nw ? x[e] * row_r * nw[lane + 32 * e] : x[e] * row_r;
+  } else if (nw) {
     float ss = 0.f;
 #pragma unroll
     for (int e = 0; e < EPL; e++) ss += x[e] * x[e];
@@ -106,25 +142,35 @@ __device__ __forceinline__ void atd_prep_head(const bf16* __restrict__ src, cons
 #pragma unroll
     for (int e = 0; e < EPL; e++) x[e] = x[e] * r * nw[lane + 32 * e];
   }
+  if (neox) {        // both numbers of a pair in this lane
 #pragma unroll
-  for (int p = 0; p < NP; p++) {
-    const float a = x[p], bb = x[p + NP];
-    x[p] = a * cs[p] - bb * sn[p];
-    x[p + NP] = a * sn[p] + bb * cs[p];
+    for (int p = 0; p < NP; p++) {
+      const float a = x[p], bb = x[p + NP];
+      x[p] = a * cs[p] - bb * sn[p];
+      x[p + NP] = a * sn[p] + bb * cs[p];
+    }
+  } else {           // the pair's other number in the neighbouring lane; cs / sn are per number then
+#pragma unroll
+    for (int e = 0; e < EPL; e++) {
+      const float o = __shfl_xor_sync(0xffffffffu, x[e], 1);
+      x[e] = (lane & 1) ? x[e] * cs[e] + o * sn[e] : x[e] * cs[e] - o * sn[e];
+    }
   }
 #pragma unroll
   for (int e = 0; e < EPL; e++) dst[lane + 32 * e] = __float2bfloat16_rn(x[e]);
 }
 
-template <int HD, int S>  // head_dim, a multiple of 32; stages of a warp's ring
+// HD: head_dim, a multiple of 32; S: stages of a warp's ring; WIDE: the softmax weights enter the second product as two
+// bfloat16 terms, p = hi + lo (16 significant bits; the row sum is of the float p either way)
+template <int HD, int S, bool WIDE>
 __global__ void __launch_bounds__(32 * ATD_WARPS)
 attention_decode_kernel(bf16* __restrict__ out, float* __restrict__ part, const bf16* __restrict__ q,
                         const bf16* __restrict__ k_pool, const bf16* __restrict__ v_pool,
                         const int* __restrict__ block_table, int bt_width,
                         const int* __restrict__ seq_slot, const int* __restrict__ seq_pos0,
                         const int* __restrict__ seq_qstart, const bf16* __restrict__ gate,
-                        int gate_stride, int nh, int nkv, int page_size, int window, float scale,
-                        int n_splits, AtdPrep prep) {
+                        int gate_stride, int gate_elem, int nh, int nkv, int page_size, int window, int chunk,
+                        float scale, int n_splits, AtdPrep prep) {
   constexpr int KB = HD / 32;  // 32-wide pieces of head_dim
   constexpr int NT = HD / 8;   // 8-wide output tiles over head_dim
   constexpr int KBYTES = 32 * HD * 2, STAGE = 2 * KBYTES;   // keys, then values
@@ -178,7 +224,7 @@ attention_decode_kernel(bf16* __restrict__ out, float* __restrict__ part, const 
 
   const int qpos = seq_pos0[b];
   const int kv_len = qpos + 1;
-  const int key_lo = (window > 0 && kv_len > window) ? kv_len - window : 0;
+  const int key_lo = first_key(qpos, window, chunk);
   const int blk_first = key_lo / 32, blk_last = (kv_len - 1) / 32;
   const int n_blk = blk_last - blk_first + 1;
   const int per_split = (n_blk + n_splits - 1) / n_splits;
@@ -229,24 +275,35 @@ attention_decode_kernel(bf16* __restrict__ out, float* __restrict__ part, const 
     if (prep.q_raw) {
       __shared__ __align__(16) bf16 q_s[16 * HD];
       constexpr int NP = HD / 64;
-      float cs[NP], sn[NP];
+      float cs[2 * NP], sn[2 * NP];
 #pragma unroll
-      for (int p = 0; p < NP; p++) {
-        const float th = (float)qpos * prep.inv_freq[lane + 32 * p];
+      for (int p = 0; p < 2 * NP; p++) {
+        if (prep.neox && p >= NP) break;
+        const float th = (float)qpos * prep.inv_freq[prep.neox ? lane + 32 * p : (lane + 32 * p) >> 1];
         cs[p] = cosf(th);
         sn[p] = sinf(th);
       }
+      float rq = 0.f, rk = 0.f;       // the rows' factors; 0: every head is normed on its own
+      if (prep.row_norm) {
+        __shared__ float red[ATD_WARPS];
+        rq = 1.0f / sqrtf(atd_row_ss(prep.q_raw + m_row * prep.q_stride, nh * HD, red) / (float)(nh * HD) + prep.eps);
+        if (prep.k_raw && has_new)
+          rk = 1.0f / sqrtf(atd_row_ss(prep.k_raw + m_row * prep.kv_stride, nkv * HD, red) / (float)(nkv * HD) + prep.eps);
+      }
       for (int hh = warp; hh < G; hh += ATD_WARPS)
-        atd_prep_head<HD>(prep.q_raw + m_row * prep.q_stride + (size_t)(h0 + hh) * HD, prep.q_norm_w, prep.eps, cs, sn,
-                          q_s + hh * HD, lane);
+        atd_prep_head<HD>(prep.q_raw + m_row * prep.q_stride + (size_t)(h0 + hh) * HD,
+                          prep.q_norm_w && prep.row_norm ? prep.q_norm_w + (size_t)(h0 + hh) * HD : prep.q_norm_w, prep.eps,
+                          cs, sn, q_s + hh * HD, lane, prep.neox, rq);
       // the new key and value: the block whose range holds the last block of positions stores them
       // (before it asks for that block's copy, so that the copy finds them in the cache)
       if (prep.k_raw && has_new) {
         const int page = table[qpos / page_size], off = qpos % page_size;
         if (page >= 0) {
           if (warp == ATD_WARPS - 1)
-            atd_prep_head<HD>(prep.k_raw + m_row * prep.kv_stride + (size_t)kvh * HD, prep.k_norm_w, prep.eps, cs, sn,
-                              prep.k_store + (((size_t)page * nkv + kvh) * page_size + off) * HD, lane);
+            atd_prep_head<HD>(prep.k_raw + m_row * prep.kv_stride + (size_t)kvh * HD,
+                              prep.k_norm_w && prep.row_norm ? prep.k_norm_w + (size_t)kvh * HD : prep.k_norm_w, prep.eps,
+                              cs, sn, prep.k_store + (((size_t)page * nkv + kvh) * page_size + off) * HD, lane, prep.neox,
+                              rk);
           for (int d = threadIdx.x; d < HD; d += blockDim.x)
             prep.v_store[(((size_t)page * nkv + kvh) * HD + d) * page_size + off] =
                 prep.v_raw[m_row * prep.kv_stride + (size_t)kvh * HD + d];
@@ -339,7 +396,7 @@ attention_decode_kernel(bf16* __restrict__ out, float* __restrict__ part, const 
       mx[hh] = mn;
     }
     float psum[2] = {0.f, 0.f};
-    uint32_t pa[4][2];  // [tile][head r | head r+8] as bfloat16 pairs
+    uint32_t pa[4][2], pl[WIDE ? 4 : 1][2];  // [tile][head r | head r+8] as bfloat16 pairs
 #pragma unroll
     for (int t = 0; t < 4; t++) {
       float p[4];
@@ -350,6 +407,10 @@ attention_decode_kernel(bf16* __restrict__ out, float* __restrict__ part, const 
       }
       pa[t][0] = pack_bf16(p[0], p[1]);
       pa[t][1] = pack_bf16(p[2], p[3]);
+      if (WIDE) {
+        pl[t][0] = rest_bf16(p[0], p[1], pa[t][0]);
+        pl[t][1] = rest_bf16(p[2], p[3], pa[t][1]);
+      }
     }
 #pragma unroll
     for (int hh = 0; hh < 2; hh++) {
@@ -365,6 +426,10 @@ attention_decode_kernel(bf16* __restrict__ out, float* __restrict__ part, const 
       acc[n][3] *= corr[1];
       mma16816(acc[n], pa[0][0], pa[0][1], pa[1][0], pa[1][1], vf[n].x, vf[n].y);
       mma16816(acc[n], pa[2][0], pa[2][1], pa[3][0], pa[3][1], vf[n].z, vf[n].w);
+      if (WIDE) {
+        mma16816(acc[n], pl[0][0], pl[0][1], pl[1][0], pl[1][1], vf[n].x, vf[n].y);
+        mma16816(acc[n], pl[2][0], pl[2][1], pl[3][0], pl[3][1], vf[n].z, vf[n].w);
+      }
     }
   }
 
@@ -400,7 +465,7 @@ attention_decode_kernel(bf16* __restrict__ out, float* __restrict__ part, const 
     const int h = h0 + hh;
     if (n_splits == 1) {
       float g = 1.f;
-      if (gate) g = 1.0f / (1.0f + expf(-__bfloat162float(gate[m_row * gate_stride + h])));
+      if (gate) g = head_gate(gate, m_row, gate_stride, h, d, HD, gate_elem);
       out[(m_row * nh + h) * HD + d] = __float2bfloat16_rn(L > 0.f ? a / L * g : 0.f);
     } else {
       float* pp = part + ((m_row * nh + h) * n_splits + split) * (size_t)(HD + 2);
@@ -423,37 +488,43 @@ LEB_API int leb_attention_decode_supported(int nh, int nkv, int hd, int page_siz
 static int attention_decode_launch(void* out, float* part, const void* q, const void* k_pool,
                                    const void* v_pool, const int* block_table, int bt_width,
                                    const int* seq_slot, const int* seq_pos0, const int* seq_qstart,
-                                   const void* gate, int gate_stride, int B, int nh, int nkv, int hd,
-                                   int page_size, int window, float scale, int n_splits, AtdPrep prep,
-                                   cudaStream_t st) {
+                                   const void* gate, int gate_stride, int gate_elem, int B, int nh, int nkv, int hd,
+                                   int page_size, int window, int chunk, int wide, float scale, int n_splits,
+                                   AtdPrep prep, cudaStream_t st) {
   if (B <= 0) return 0;
   LEB_REQUIRE(leb_attention_decode_supported(nh, nkv, hd, page_size),
               "leb_attention_decode: sizes not taken (heads %d, kv heads %d, head_dim %d, page %d)", nh, nkv, hd, page_size);
   LEB_REQUIRE(n_splits >= 1 && (n_splits == 1 || part), "leb_attention_decode: splits need scratch");
   dim3 grid(nkv, B, n_splits);
   LEB_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "leb_attention_decode: grid too large");
-#define LEB_ATD(HD_, S_)                                                                          \
+#define LEB_ATD_W(HD_, S_, W_)                                                                    \
   {                                                                                               \
     constexpr int smem = ATD_WARPS * S_ * 2 * 32 * HD_ * 2;                                        \
     static bool set = false;                                                                      \
     if (!set) {                                                                                   \
-      if (cudaFuncSetAttribute(attention_decode_kernel<HD_, S_>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) \
+      if (cudaFuncSetAttribute(attention_decode_kernel<HD_, S_, W_>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) \
         return leb_fail("leb_attention_decode: %d bytes of shared memory per block refused", smem); \
       set = true;                                                                                 \
     }                                                                                             \
-    leb_launch(attention_decode_kernel<HD_, S_>, grid, dim3(32 * ATD_WARPS), smem, st,             \
+    leb_launch(attention_decode_kernel<HD_, S_, W_>, grid, dim3(32 * ATD_WARPS), smem, st,             \
         (bf16*)out, part, (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, block_table,  \
-        bt_width, seq_slot, seq_pos0, seq_qstart, (const bf16*)gate, gate_stride, nh, nkv, page_size, \
-        window, scale, n_splits, prep);                                                           \
+        bt_width, seq_slot, seq_pos0, seq_qstart, (const bf16*)gate, gate_stride, gate_elem, nh, nkv, \
+        page_size, window, chunk, scale, n_splits, prep);                                         \
+  }
+#define LEB_ATD(HD_, S_)                    \
+  {                                         \
+    if (wide) LEB_ATD_W(HD_, S_, true)      \
+    else LEB_ATD_W(HD_, S_, false)          \
   }
   const bool few = (long)grid.x * grid.y * grid.z <= 2L * sm_count();   // an SM gets two blocks at most: deeper rings
   switch (hd) {
-    case 32: LEB_ATD(32, 3); break;
+    case 32: LEB_ATD(32, 3) break;
     case 64: if (few) LEB_ATD(64, 3) else LEB_ATD(64, 2) break;
-    case 96: LEB_ATD(96, 2); break;
-    default: LEB_ATD(128, 2); break;
+    case 96: LEB_ATD(96, 2) break;
+    default: LEB_ATD(128, 2) break;
   }
 #undef LEB_ATD
+#undef LEB_ATD_W
   LEB_CHECK_LAUNCH("leb_attention_decode");
   return 0;
 }
@@ -461,17 +532,18 @@ static int attention_decode_launch(void* out, float* part, const void* q, const 
 LEB_API int leb_attention_decode(void* out, float* part, const void* q, const void* k_pool,
                                  const void* v_pool, const int* block_table, int bt_width,
                                  const int* seq_slot, const int* seq_pos0, const int* seq_qstart,
-                                 const void* gate, int gate_stride, int B, int nh, int nkv, int hd,
-                                 int page_size, int window, float scale, int n_splits,
+                                 const void* gate, int gate_stride, int gate_elem, int B, int nh, int nkv, int hd,
+                                 int page_size, int window, int chunk, int wide, float scale, int n_splits,
                                  cudaStream_t st) {
   return attention_decode_launch(out, part, q, k_pool, v_pool, block_table, bt_width, seq_slot, seq_pos0, seq_qstart, gate,
-                                 gate_stride, B, nh, nkv, hd, page_size, window, scale, n_splits, AtdPrep{}, st);
+                                 gate_stride, gate_elem, B, nh, nkv, hd, page_size, window, chunk, wide, scale, n_splits,
+                                 AtdPrep{}, st);
 }
 
 // Returns 1 when the kernel can norm, rotate and store the step's q, k and v itself: head size 64 or
-// 128 and a split-half rotation over the whole head.
+// 128 and a rotation over the whole head (split-half or adjacent pairs).
 LEB_API int leb_attention_decode_prep_supported(int nh, int nkv, int hd, int page_size, int rope_dim, int neox) {
-  return leb_attention_decode_supported(nh, nkv, hd, page_size) && (hd == 64 || hd == 128) && rope_dim == hd && neox != 0;
+  return leb_attention_decode_supported(nh, nkv, hd, page_size) && (hd == 64 || hd == 128) && rope_dim == hd;
 }
 
 // The same with the step's q, k and v as the projection left them (rows of q_stride / kv_stride
@@ -483,24 +555,25 @@ LEB_API int leb_attention_decode_prep(void* out, float* part, const void* q_raw,
                                       const int* block_table, int bt_width, const int* seq_slot,
                                       const int* seq_pos0, const int* seq_qstart, const float* q_norm_w,
                                       const float* k_norm_w, float eps, const float* inv_freq, int rope_dim,
-                                      int neox, const void* gate, int gate_stride, int B, int nh, int nkv,
-                                      int hd, int page_size, int window, float scale, int n_splits,
+                                      int neox, int row_norm, const void* gate, int gate_stride, int gate_elem, int B, int nh, int nkv,
+                                      int hd, int page_size, int window, int chunk, int wide, float scale, int n_splits,
                                       cudaStream_t st) {
   LEB_REQUIRE(leb_attention_decode_prep_supported(nh, nkv, hd, page_size, rope_dim, neox),
               "leb_attention_decode_prep: sizes not taken (head_dim %d, rope_dim %d, split-half %d)", hd, rope_dim, neox);
   LEB_REQUIRE(q_raw && inv_freq, "leb_attention_decode_prep: q and the frequencies are required");
   LEB_REQUIRE((k_raw == nullptr) == (v_raw == nullptr), "leb_attention_decode_prep: keys and values come together");
   AtdPrep prep{(const bf16*)q_raw, (const bf16*)k_raw, (const bf16*)v_raw, q_stride, kv_stride, (bf16*)k_pool,
-               (bf16*)v_pool, q_norm_w, k_norm_w, inv_freq, eps};
+               (bf16*)v_pool, q_norm_w, k_norm_w, inv_freq, eps, neox != 0, row_norm != 0};
   return attention_decode_launch(out, part, nullptr, k_pool, v_pool, block_table, bt_width, seq_slot, seq_pos0, seq_qstart,
-                                 gate, gate_stride, B, nh, nkv, hd, page_size, window, scale, n_splits, prep, st);
+                                 gate, gate_stride, gate_elem, B, nh, nkv, hd, page_size, window, chunk, wide, scale, n_splits,
+                                 prep, st);
 }
 
 // ---- the same step for callers that cannot allocate (see leb_no_alloc.h) ---------------------------
 #include "leb_no_alloc.h"
 
 extern "C" int leb_attention_merge(void* out, const float* part, int dtype, const void* gate, int gate_stride,
-                                   int M, int nh, int hd, int n_splits, cudaStream_t st);
+                                   int gate_elem, int M, int nh, int hd, int n_splits, cudaStream_t st);
 
 // The split partial results of leb_attention_decode_static.  In host code this name is only a
 // handle for cudaGetSymbolAddress, not a device address.
@@ -537,9 +610,9 @@ LEB_API int leb_attention_decode_static(void* out, const void* q, const void* k_
     scratch = g_static_scratch_ptr[dev];
   }
   int rc = leb_attention_decode(out, scratch, q, k_pool, v_pool, block_table, bt_width, seq_slot, seq_pos0,
-                                seq_qstart, gate, gate_stride, B, nh, nkv, hd, page_size, window, scale, n_splits, st);
+                                seq_qstart, gate, gate_stride, 0, B, nh, nkv, hd, page_size, window, 0, 0, scale, n_splits, st);
   if (rc) return rc;
   if (n_splits > 1)
-    return leb_attention_merge(out, scratch, LEB_BF16, gate, gate_stride, B, nh, hd, n_splits, st);
+    return leb_attention_merge(out, scratch, LEB_BF16, gate, gate_stride, 0, B, nh, hd, n_splits, st);
   return 0;
 }

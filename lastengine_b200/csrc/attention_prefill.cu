@@ -32,6 +32,11 @@ __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
   __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<uint32_t*>(&v);
 }
+// what bfloat16 left of (lo, hi) packed into `kept`
+__device__ __forceinline__ uint32_t rest2(float lo, float hi, uint32_t kept) {
+  const __nv_bfloat162 k = *reinterpret_cast<const __nv_bfloat162*>(&kept);
+  return pack2(lo - __bfloat162float(k.x), hi - __bfloat162float(k.y));
+}
 __device__ __forceinline__ uint4 mask_tail(uint4 v, int first, int hi) {
   uint32_t* w = reinterpret_cast<uint32_t*>(&v);
 #pragma unroll
@@ -42,15 +47,17 @@ __device__ __forceinline__ uint4 mask_tail(uint4 v, int first, int hi) {
   return v;
 }
 
-template <int HD, int MT>  // head_dim (multiple of 32); 16-row tiles per warp
+// HD: head_dim (multiple of 32); MT: 16-row tiles per warp.  WIDE: the softmax weights enter the second product as two
+// bfloat16 terms, p = hi + lo (16 significant bits; the row sum is of the float p either way).
+template <int HD, int MT, bool WIDE>
 __global__ void __launch_bounds__(32 * ATP_WARPS)
 attention_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ q,
                          const bf16* __restrict__ k_pool, const bf16* __restrict__ v_pool,
                          const int* __restrict__ block_table, int bt_width,
                          const int* __restrict__ seq_slot, const int* __restrict__ seq_pos0,
                          const int* __restrict__ seq_qstart, const int* __restrict__ seq_qlen,
-                         const bf16* __restrict__ gate, int gate_stride, int nh, int nkv, int page_size,
-                         int window, float scale, int QT) {
+                         const bf16* __restrict__ gate, int gate_stride, int gate_elem, int nh, int nkv,
+                         int page_size, int window, int chunk, float scale, int QT) {
   constexpr int KB = HD / 32, NT = HD / 8;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int r = lane >> 2, c = lane & 3;
@@ -71,7 +78,7 @@ attention_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ q,
   if (row0 >= nrows) return;
 
   // rows of this lane: tile mt, halves 0 (row r) and 1 (row r + 8)
-  int rpos[MT][2], rhead[MT][2];
+  int rpos[MT][2], rhead[MT][2], rlo[MT][2];
   bool rok[MT][2];
 #pragma unroll
   for (int mt = 0; mt < MT; mt++)
@@ -81,6 +88,7 @@ attention_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ q,
       rok[mt][hh] = row < nrows;
       rpos[mt][hh] = p_lo + row / G;       // position within this step's rows of the sequence
       rhead[mt][hh] = row % G;
+      rlo[mt][hh] = first_key(pos0 + rpos[mt][hh], window, chunk);
     }
 
   if (slot < 0) {   // padding sequence: zeros
@@ -115,7 +123,8 @@ attention_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ q,
   const int first_pos = pos0 + p_lo + row0 / G;
   const int last_row = min(nrows, row0 + MT * 16) - 1;
   const int key_hi = pos0 + p_lo + last_row / G;
-  const int key_lo = (window > 0 && first_pos + 1 > window) ? first_pos + 1 - window : 0;
+  const int key_lo = first_key(first_pos, window, chunk);
+  const int lo_last = first_key(key_hi, window, chunk);      // no row of this warp starts later than here
 
   float mx[MT][2], l[MT][2], acc[MT][NT][4];
 #pragma unroll
@@ -169,7 +178,7 @@ attention_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ q,
 #pragma unroll
       for (int n = 0; n < NT; n++) vf[n] = mask_tail(vf[n], key0 + 8 * c, kv_len);
     }
-    const bool need_mask = window > 0 || key0 + 31 > qmin;
+    const bool need_mask = key0 < lo_last || key0 + 31 > qmin;
 
 #pragma unroll
     for (int mt = 0; mt < MT; mt++) {
@@ -193,7 +202,7 @@ attention_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ q,
             const int hh = e >> 1;
             const int kp = key0 + 8 * c + 2 * t + (e & 1);
             const int qp = pos0 + rpos[mt][hh];
-            const bool valid = kp <= qp && (window <= 0 || kp + window > qp);
+            const bool valid = kp <= qp && kp >= rlo[mt][hh];
             s[t][e] = valid ? s[t][e] * scale2 : ATP_NEG;
             tmax[hh] = fmaxf(tmax[hh], s[t][e]);
           }
@@ -216,7 +225,7 @@ attention_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ q,
         mx[mt][hh] = mn;
       }
       float psum[2] = {0.f, 0.f};
-      uint32_t pa[4][2];
+      uint32_t pa[4][2], pl[WIDE ? 4 : 1][2];
 #pragma unroll
       for (int t = 0; t < 4; t++) {
         float p[4];
@@ -228,6 +237,10 @@ attention_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ q,
         }
         pa[t][0] = pack2(p[0], p[1]);
         pa[t][1] = pack2(p[2], p[3]);
+        if (WIDE) {
+          pl[t][0] = rest2(p[0], p[1], pa[t][0]);
+          pl[t][1] = rest2(p[2], p[3], pa[t][1]);
+        }
       }
 #pragma unroll
       for (int hh = 0; hh < 2; hh++) {
@@ -247,6 +260,10 @@ attention_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ q,
         }
         mma16816p(acc[mt][n], pa[0][0], pa[0][1], pa[1][0], pa[1][1], vf[n].x, vf[n].y);
         mma16816p(acc[mt][n], pa[2][0], pa[2][1], pa[3][0], pa[3][1], vf[n].z, vf[n].w);
+        if (WIDE) {
+          mma16816p(acc[mt][n], pl[0][0], pl[0][1], pl[1][0], pl[1][1], vf[n].x, vf[n].y);
+          mma16816p(acc[mt][n], pl[2][0], pl[2][1], pl[3][0], pl[3][1], vf[n].z, vf[n].w);
+        }
       }
     }
   };
@@ -275,13 +292,17 @@ attention_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ q,
       if (!rok[mt][hh]) continue;
       const size_t m = q0 + rpos[mt][hh];
       const int h = h0 + rhead[mt][hh];
-      float g = 1.f;
-      if (gate) g = 1.0f / (1.0f + expf(-__bfloat162float(gate[m * gate_stride + h])));
+      const float g = gate && !gate_elem ? head_gate(gate, m, gate_stride, h, 0, HD, 0) : 1.f;
       const float inv = l[mt][hh] > 0.f ? g / l[mt][hh] : 0.f;
       bf16* o = out + (m * nh + h) * HD;
 #pragma unroll
       for (int n = 0; n < NT; n++) {
-        const uint32_t v = pack2(acc[mt][n][2 * hh] * inv, acc[mt][n][2 * hh + 1] * inv);
+        float f0 = inv, f1 = inv;
+        if (gate && gate_elem) {
+          f0 *= head_gate(gate, m, gate_stride, h, 8 * n + 2 * c, HD, 1);
+          f1 *= head_gate(gate, m, gate_stride, h, 8 * n + 2 * c + 1, HD, 1);
+        }
+        const uint32_t v = pack2(acc[mt][n][2 * hh] * f0, acc[mt][n][2 * hh + 1] * f1);
         *reinterpret_cast<uint32_t*>(o + 8 * n + 2 * c) = v;
       }
     }
@@ -296,8 +317,9 @@ LEB_API int leb_attention_prefill_supported(int nh, int nkv, int hd, int page_si
 LEB_API int leb_attention_prefill(void* out, const void* q, const void* k_pool, const void* v_pool,
                                   const int* block_table, int bt_width, const int* seq_slot,
                                   const int* seq_pos0, const int* seq_qstart, const int* seq_qlen,
-                                  const void* gate, int gate_stride, int B, int nh, int nkv, int hd,
-                                  int page_size, int window, float scale, int max_qlen, cudaStream_t st) {
+                                  const void* gate, int gate_stride, int gate_elem, int B, int nh, int nkv, int hd,
+                                  int page_size, int window, int chunk, int wide, float scale, int max_qlen,
+                                  cudaStream_t st) {
   if (B <= 0 || max_qlen <= 0) return 0;
   LEB_REQUIRE(leb_attention_prefill_supported(nh, nkv, hd, page_size),
               "leb_attention_prefill: sizes not taken (heads %d, kv heads %d, head_dim %d, page %d)", nh, nkv, hd, page_size);
@@ -308,11 +330,14 @@ LEB_API int leb_attention_prefill(void* out, const void* q, const void* k_pool, 
   if (QT < 1) QT = 1;
   dim3 grid(ceil_div(max_qlen, QT), nkv, B);
   LEB_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "leb_attention_prefill: grid too large");
-#define LEB_ATP(HD_, MT_)                                                                            \
-  attention_prefill_kernel<HD_, MT_><<<grid, 32 * ATP_WARPS, 0, st>>>(                               \
+#define LEB_ATP_W(HD_, MT_, W_)                                                                      \
+  attention_prefill_kernel<HD_, MT_, W_><<<grid, 32 * ATP_WARPS, 0, st>>>(                               \
       (bf16*)out, (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, block_table, bt_width,   \
-      seq_slot, seq_pos0, seq_qstart, seq_qlen, (const bf16*)gate, gate_stride, nh, nkv, page_size,  \
-      window, scale, QT)
+      seq_slot, seq_pos0, seq_qstart, seq_qlen, (const bf16*)gate, gate_stride, gate_elem, nh, nkv,  \
+      page_size, window, chunk, scale, QT)
+#define LEB_ATP(HD_, MT_)                \
+  if (wide) LEB_ATP_W(HD_, MT_, true);   \
+  else LEB_ATP_W(HD_, MT_, false)
   switch (hd) {
     case 32: LEB_ATP(32, 2); break;
     case 64: LEB_ATP(64, 1); break;
@@ -320,6 +345,7 @@ LEB_API int leb_attention_prefill(void* out, const void* q, const void* k_pool, 
     default: LEB_ATP(128, 1); break;
   }
 #undef LEB_ATP
+#undef LEB_ATP_W
   LEB_CHECK_LAUNCH("leb_attention_prefill");
   return 0;
 }

@@ -79,8 +79,9 @@ __device__ __forceinline__ int atc_blocks_seen(int qpos, int window, int pool) {
   return (window > 0 && pool > 0 && past > 0) ? past / pool : 0;
 }
 
+// WIDE: the weights as two terms as POOLED has them, for layers without pooled blocks too.
 // GS query heads per kv head (1, 2, 4, 8): a tile is GS heads x 128/GS positions; VD: width of a value head (64 or 32)
-template <int GS, bool POOLED, int VD>
+template <int GS, bool POOLED, bool WIDE, int VD>
 __global__ void __launch_bounds__(ATC_THREADS, 2)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_pk,
@@ -88,8 +89,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             const int* __restrict__ block_table, int bt_width, const int* __restrict__ pool_table,
                             int pt_width, const int* __restrict__ seq_slot,
                             const int* __restrict__ seq_pos0, const int* __restrict__ seq_qstart,
-                            const int* __restrict__ seq_qlen, const bf16* __restrict__ gate, int gate_stride,
-                            int nh, int nkv, int window, int pool, float scale, const float* __restrict__ head_scale,
+                            const int* __restrict__ seq_qlen, const bf16* __restrict__ gate, int gate_stride, int gate_elem,
+                            int nh, int nkv, int window, int chunk, int pool, float scale, const float* __restrict__ head_scale,
                             const float* __restrict__ freq_v, int* __restrict__ status) {
   constexpr int HD = 64, PAGE = 64, TP = 128 / GS, NS = ATC_STAGES;
   constexpr int Q_BYTES = 128 * HD * 2, KV_BYTES = PAGE * HD * 2, V_BYTES = VD * PAGE * 2;
@@ -128,7 +129,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   }
   const int q_lo = pos0 + row0;                  // position of the tile's first query
   const int key_hi = q_lo + rows;                // keys [.., key_hi) exist for this tile
-  const int key_lo_tile = window > 0 ? max(0, q_lo - window + 1) : 0;
+  const int key_lo_tile = first_key(q_lo, window, chunk);
   const int jb0 = key_lo_tile / PAGE, nblk = (key_hi - 1) / PAGE - jb0 + 1;
   const int* table = block_table + (size_t)b * bt_width;
   const int nb_tile = POOLED ? atc_blocks_seen(key_hi - 1, window, pool) : 0;   // pooled blocks the tile's last row sees
@@ -211,7 +212,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         if (!mbar_wait(&v_full[s], (i / NS) & 1, abort_flag)) { atomicExch(status, 15); ok = false; break; }
         tc_fence_after();
         const uint32_t va = smem_u32(sv + s * V_BYTES);
-        if (POOLED) {
+        if (WIDE) {
           const uint32_t t_p = t_s0 + 64 * (i & 1);   // hi in the scores' first 32 columns, lo in the next 32
 #pragma unroll
           for (int kk = 0; kk < PAGE / 16; kk++)
@@ -233,7 +234,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const int r = threadIdx.x, g = r / TP, pi = r % TP;
     const bool row_valid = pi < rows;
     const int qpos = q_lo + pi;
-    const int key_lo_row = window > 0 ? max(0, qpos - window + 1) : 0;
+    const int key_lo_row = first_key(qpos, window, chunk);
     const uint32_t lane_base = (uint32_t)(warp * 32) << 16;
     const float scale2 = (head_scale ? head_scale[h0 + g] : scale) * 1.4426950408889634f;
     const int nb_row = POOLED ? atc_blocks_seen(qpos, window, pool) : 0;
@@ -288,7 +289,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         if (move) m_used = m_new;
       }
       const float m_ref = m_used > 0.5f * ATC_NEG ? m_used : 0.f;
-      uint32_t pk[32], pl[POOLED ? 32 : 1];
+      uint32_t pk[32], pl[WIDE ? 32 : 1];
       float ps[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int c = 0; c < PAGE; c += 2) {
@@ -297,7 +298,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         ps[(c >> 1) & 3] += p0 + p1;
         __nv_bfloat162 pp = __floats2bfloat162_rn(p0, p1);
         pk[c >> 1] = *reinterpret_cast<uint32_t*>(&pp);
-        if (POOLED) {
+        if (WIDE) {
           __nv_bfloat162 pr = __floats2bfloat162_rn(p0 - __bfloat162float(pp.x), p1 - __bfloat162float(pp.y));
           pl[c >> 1] = *reinterpret_cast<uint32_t*>(&pr);
         }
@@ -306,7 +307,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       // P[bsel] was last read by the product of page i-2
       if (i >= 2 && !mbar_wait(&pv_done[bsel], ((i - 2) >> 1) & 1, abort_flag)) { atomicExch(status, 18); ok = false; break; }
       tc_fence_after();
-      if (POOLED) {
+      if (WIDE) {
         tmem_st32(t_s0 + 64 * bsel + lane_base, pk);
         tmem_st32(t_s0 + 64 * bsel + 32 + lane_base, pl);
       } else {
@@ -337,7 +338,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     if (ok) {
       tc_fence_after();
       float inv = l > 0.f ? 1.0f / l : 0.f;
-      if (gate && row_valid) inv *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(m_base + pi) * gate_stride + h0 + g])));
+      if (gate && !gate_elem && row_valid) inv *= head_gate(gate, m_base + pi, gate_stride, h0 + g, 0, VD, 0);
       uint4* orow = reinterpret_cast<uint4*>(out + ((m_base + pi) * nh + h0 + g) * VD);
       uint32_t o[VD];
       tmem_ld32(t_o + lane_base, o);
@@ -346,6 +347,23 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       if (row_valid) {
 #pragma unroll
         for (int c = 0; c < VD; c++) o[c] = __float_as_uint(__uint_as_float(o[c]) * inv);
+        if (gate && gate_elem) {
+          const bf16* grow = gate + (m_base + pi) * (size_t)gate_stride + (h0 + g) * VD;
+          if ((((uintptr_t)grow) & 15) == 0) {
+#pragma unroll
+            for (int c = 0; c < VD; c += 8) {
+              const uint4 w = *reinterpret_cast<const uint4*>(grow + c);
+              const bf16* z = reinterpret_cast<const bf16*>(&w);
+#pragma unroll
+              for (int e = 0; e < 8; e++)
+                o[c + e] = __float_as_uint(__fdividef(__uint_as_float(o[c + e]), 1.0f + __expf(-__bfloat162float(z[e]))));
+            }
+          } else {
+#pragma unroll
+            for (int c = 0; c < VD; c++)
+              o[c] = __float_as_uint(__fdividef(__uint_as_float(o[c]), 1.0f + __expf(-__bfloat162float(grow[c]))));
+          }
+        }
         if (POOLED && freq_v) {
           // values were cached turned by their positions: the sum is turned back by the query's (pairs c, c + VD/2)
           const float fpos = (float)qpos;
@@ -383,13 +401,13 @@ LEB_API int leb_attention_prefill_tc_supported(int nh, int nkv, int hd, int page
   return G == 1 || G == 2 || G == 4 || G == 8;
 }
 
-template <bool POOLED, int VD>
+template <bool POOLED, bool WIDE, int VD>
 static int launch_attention_prefill_tc(const char* who, void* out, const void* q, int q_stride, int M, const void* k_pool,
                                        const void* v_pool, int n_pages, const int* block_table, int bt_width,
                                        const void* pk_pool, const void* pv_pool, int n_pooled_pages, const int* pool_table,
                                        int pt_width, const int* seq_slot, const int* seq_pos0, const int* seq_qstart,
-                                       const int* seq_qlen, const void* gate, int gate_stride, int B, int nh, int nkv,
-                                       int hd, int page_size, int window, int pool, float scale, const float* head_scale,
+                                       const int* seq_qlen, const void* gate, int gate_stride, int gate_elem, int B, int nh, int nkv,
+                                       int hd, int page_size, int window, int chunk, int pool, float scale, const float* head_scale,
                                        const float* freq_v, int max_qlen, int* status, cudaStream_t st) {
   if (B <= 0 || max_qlen <= 0 || M <= 0) return 0;
   LEB_REQUIRE(leb_attention_prefill_tc_supported(nh, nkv, hd, page_size),
@@ -419,13 +437,13 @@ static int launch_attention_prefill_tc(const char* who, void* out, const void* q
   {                                                                                                               \
     static bool set = false;                                                                                      \
     if (!set) {                                                                                                   \
-      if (cudaFuncSetAttribute(attention_prefill_tc_kernel<GS_, POOLED, VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) \
+      if (cudaFuncSetAttribute(attention_prefill_tc_kernel<GS_, POOLED, WIDE, VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) \
         return leb_fail("%s: %zu bytes of shared memory per block refused", who, smem);                         \
       set = true;                                                                                                 \
     }                                                                                                             \
-    leb_launch(attention_prefill_tc_kernel<GS_, POOLED, VD>, grid, dim3(ATC_THREADS), smem, st,                       \
+    leb_launch(attention_prefill_tc_kernel<GS_, POOLED, WIDE, VD>, grid, dim3(ATC_THREADS), smem, st,                       \
         mq, mk, mv, mpk, mpv, (bf16*)out, block_table, bt_width, pool_table, pt_width, seq_slot, seq_pos0, seq_qstart, \
-        seq_qlen, (const bf16*)gate, gate_stride, nh, nkv, window, pooled ? pool : 0, scale, head_scale, freq_v, status); \
+        seq_qlen, (const bf16*)gate, gate_stride, gate_elem, nh, nkv, window, chunk, pooled ? pool : 0, scale, head_scale, freq_v, status); \
   }
   switch (G) {
     case 1: LEB_ATC(1); break;
@@ -445,13 +463,14 @@ static int launch_attention_prefill_tc(const char* who, void* out, const void* q
 LEB_API int leb_attention_prefill_tc(void* out, const void* q, int q_stride, int M, const void* k_pool,
                                      const void* v_pool, int n_pages, const int* block_table, int bt_width,
                                      const int* seq_slot, const int* seq_pos0, const int* seq_qstart,
-                                     const int* seq_qlen, const void* gate, int gate_stride, int B, int nh, int nkv,
-                                     int hd, int page_size, int window, float scale, int max_qlen, int* status,
-                                     cudaStream_t st) {
-  return launch_attention_prefill_tc<false, 64>("leb_attention_prefill_tc", out, q, q_stride, M, k_pool, v_pool, n_pages,
-                                            block_table, bt_width, nullptr, nullptr, 0, nullptr, 0, seq_slot, seq_pos0,
-                                            seq_qstart, seq_qlen, gate, gate_stride, B, nh, nkv, hd, page_size, window, 0,
-                                            scale, nullptr, nullptr, max_qlen, status, st);
+                                     const int* seq_qlen, const void* gate, int gate_stride, int gate_elem, int B, int nh,
+                                     int nkv, int hd, int page_size, int window, int chunk, int wide, float scale,
+                                     int max_qlen, int* status, cudaStream_t st) {
+#define LEB_ATC_ARGS "leb_attention_prefill_tc", out, q, q_stride, M, k_pool, v_pool, n_pages, block_table, bt_width, nullptr, \
+                     nullptr, 0, nullptr, 0, seq_slot, seq_pos0, seq_qstart, seq_qlen, gate, gate_stride, gate_elem, B, nh, nkv, \
+                     hd, page_size, window, chunk, 0, scale, nullptr, nullptr, max_qlen, status, st
+  return wide ? launch_attention_prefill_tc<false, true, 64>(LEB_ATC_ARGS) : launch_attention_prefill_tc<false, false, 64>(LEB_ATC_ARGS);
+#undef LEB_ATC_ARGS
 }
 
 // The same over a window with pooled blocks behind it (pool 0: none): pk_pool / pv_pool hold one row per
@@ -467,9 +486,9 @@ LEB_API int leb_attention_pooled_tc(void* out, const void* q, int q_stride, int 
   LEB_REQUIRE(head_scale != nullptr, "leb_attention_pooled_tc: a factor per head is required");
   LEB_REQUIRE(vd == 64 || vd == 32, "leb_attention_pooled_tc: value heads of %d numbers (64 or 32)", vd);
 #define LEB_APT_ARGS "leb_attention_pooled_tc", out, q, q_stride, M, k_pool, v_pool, n_pages, block_table, bt_width, pk_pool, \
-                     pv_pool, n_pooled_pages, pool_table, pt_width, seq_slot, seq_pos0, seq_qstart, seq_qlen, nullptr, 0, B, nh, \
-                     nkv, hd, page_size, window, pool, 1.0f, head_scale, freq_v, max_qlen, status, st
-  const int rc = vd == 64 ? launch_attention_prefill_tc<true, 64>(LEB_APT_ARGS) : launch_attention_prefill_tc<true, 32>(LEB_APT_ARGS);
+                     pv_pool, n_pooled_pages, pool_table, pt_width, seq_slot, seq_pos0, seq_qstart, seq_qlen, nullptr, 0, 0, B, nh, \
+                     nkv, hd, page_size, window, 0, pool, 1.0f, head_scale, freq_v, max_qlen, status, st
+  const int rc = vd == 64 ? launch_attention_prefill_tc<true, true, 64>(LEB_APT_ARGS) : launch_attention_prefill_tc<true, true, 32>(LEB_APT_ARGS);
 #undef LEB_APT_ARGS
   return rc;
 }

@@ -154,6 +154,22 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   return red[32];
 }
 
+// First key position the query at `pos` reads: 0, the start of its window of `window` positions, or the start of its
+// chunk of `chunk` positions counted from the sequence's first (each where positive; never falls as pos grows).
+__device__ __forceinline__ int first_key(int pos, int window, int chunk) {
+  int lo = (window > 0 && pos + 1 > window) ? pos + 1 - window : 0;
+  if (chunk > 0) lo = max(lo, pos - pos % chunk);
+  return lo;
+}
+
+// The factor sigmoid(gate) of a head's result: one per (row, head), or with `elem` one per dimension of the head
+// (gate [rows, heads, width]).
+template <typename T>
+__device__ __forceinline__ float head_gate(const T* gate, size_t row, int stride, int h, int d, int width, int elem) {
+  const float z = to_f32(gate[row * stride + (elem ? h * width + d : h)]);
+  return 1.0f / (1.0f + expf(-z));
+}
+
 static inline int ceil_div(int a, int b) { return (a + b - 1) / b; }
 
 // SMs of the current device, asked once per device (device_info.cu); launch shapes that are

@@ -566,6 +566,129 @@ __global__ void activation_kernel(TO* __restrict__ a, const float* __restrict__ 
   a[i] = from_f32<TO>(r);
 }
 
+// x += y / sqrt(mean(y^2) + eps) * w per row: a sublayer's result is normed on its way into the residual stream.  With
+// `h` the launch also leaves the new rows there in h's type, for the sublayer that reads the stream itself next.
+// Rows of up to 4096 numbers on the 16-byte grid stay in registers between the sum of squares and the sum (CH groups
+// of four numbers a thread); others are read twice.
+template <typename TH, int CH>
+__global__ void __launch_bounds__(256)
+outnorm_residual_vec_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ w, float eps,
+                            TH* __restrict__ h, int D) {
+  __shared__ float red[33];
+  pdl_trigger();   // the kernel after this one may start and wait (see common.cuh)
+  pdl_wait();
+  const size_t m = blockIdx.x;
+  const float4* y4 = reinterpret_cast<const float4*>(y + m * D);
+  float4* x4 = reinterpret_cast<float4*>(x + m * D);
+  const float4* w4 = reinterpret_cast<const float4*>(w);
+  const int n4 = D >> 2;
+  float4 v[CH], xv[CH];
+  float s = 0.f;
+#pragma unroll
+  for (int c = 0; c < CH; c++) {
+    const int i = threadIdx.x + c * 256;
+    if (i < n4) {
+      v[c] = y4[i];
+      xv[c] = x4[i];
+      s += (v[c].x * v[c].x + v[c].y * v[c].y) + (v[c].z * v[c].z + v[c].w * v[c].w);
+    }
+  }
+  s = block_sum(s, red);
+  const float r = 1.0f / sqrtf(s / (float)D + eps);
+#pragma unroll
+  for (int c = 0; c < CH; c++) {
+    const int i = threadIdx.x + c * 256;
+    if (i < n4) {
+      const float4 ww = w4[i];
+      const float4 o = make_float4(xv[c].x + v[c].x * r * ww.x, xv[c].y + v[c].y * r * ww.y, xv[c].z + v[c].z * r * ww.z,
+                                   xv[c].w + v[c].w * r * ww.w);
+      x4[i] = o;
+      if (h) {
+        if (sizeof(TH) == 2) {
+          __nv_bfloat162 lo = __floats2bfloat162_rn(o.x, o.y), hi = __floats2bfloat162_rn(o.z, o.w);
+          reinterpret_cast<uint2*>(h + m * D)[i] = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+        } else {
+          reinterpret_cast<float4*>(h + m * D)[i] = o;
+        }
+      }
+    }
+  }
+}
+
+template <typename TH>
+__global__ void __launch_bounds__(256)
+outnorm_residual_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ w, float eps,
+                        TH* __restrict__ h, int D) {
+  __shared__ float red[33];
+  pdl_trigger();   // the kernel after this one may start and wait (see common.cuh)
+  pdl_wait();
+  const size_t m = blockIdx.x;
+  float s = 0.f;
+  for (int i = threadIdx.x; i < D; i += blockDim.x) s += y[m * D + i] * y[m * D + i];
+  const float r = 1.0f / sqrtf(block_sum(s, red) / (float)D + eps);
+  for (int i = threadIdx.x; i < D; i += blockDim.x) {
+    const float o = x[m * D + i] + y[m * D + i] * r * w[i];
+    x[m * D + i] = o;
+    if (h) h[m * D + i] = from_f32<TH>(o);
+  }
+}
+
+LEB_API int leb_outnorm_residual(float* x, const float* y, const float* w, float eps, void* h, int h_dtype, int M, int D,
+                                 cudaStream_t st) {
+  if (M <= 0 || D <= 0) return 0;
+  LEB_REQUIRE(!h || h_dtype == LEB_F32 || h_dtype == LEB_BF16, "leb_outnorm_residual: unknown dtype %d", h_dtype);
+  const bool b16 = h && h_dtype == LEB_BF16;
+  const bool vec = D % 4 == 0 && D <= 4096 && ((((uintptr_t)x | (uintptr_t)y | (uintptr_t)w) & 15) == 0) &&
+                   ((uintptr_t)h & 15) == 0;
+  const dim3 grid(M), block(256);
+#define LEB_ONR(CH_)                                                                                                       \
+  (b16 ? leb_launch(outnorm_residual_vec_kernel<bf16, CH_>, grid, block, 0, st, x, y, w, eps, (bf16*)h, D)               \
+       : leb_launch(outnorm_residual_vec_kernel<float, CH_>, grid, block, 0, st, x, y, w, eps, (float*)h, D))
+  if (vec) {
+    const int ch = ceil_div(D / 4, 256);
+    if (ch <= 1) LEB_ONR(1);
+    else if (ch <= 2) LEB_ONR(2);
+    else LEB_ONR(4);
+  } else if (b16) {
+    leb_launch(outnorm_residual_kernel<bf16>, grid, block, 0, st, x, y, w, eps, (bf16*)h, D);
+  } else {
+    leb_launch(outnorm_residual_kernel<float>, grid, block, 0, st, x, y, w, eps, (float*)h, D);
+  }
+#undef LEB_ONR
+  LEB_CHECK_LAUNCH("leb_outnorm_residual");
+  return 0;
+}
+
+// z -> cap tanh(scale z / cap) in place (cap <= 0: z -> scale z); four numbers a thread.
+__global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ z, float scale, float cap, size_t n) {
+  pdl_trigger();   // the kernel after this one may start and wait (see common.cuh)
+  pdl_wait();
+  const size_t i0 = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (i0 + 4 <= n && ((uintptr_t)z & 15) == 0) {
+    float4 v = *reinterpret_cast<float4*>(z + i0);
+    v.x *= scale; v.y *= scale; v.z *= scale; v.w *= scale;
+    if (cap > 0.f) {
+      v.x = cap * tanhf(v.x / cap);
+      v.y = cap * tanhf(v.y / cap);
+      v.z = cap * tanhf(v.z / cap);
+      v.w = cap * tanhf(v.w / cap);
+    }
+    *reinterpret_cast<float4*>(z + i0) = v;
+    return;
+  }
+  for (size_t i = i0; i < n && i < i0 + 4; i++) {
+    const float t = z[i] * scale;
+    z[i] = cap > 0.f ? cap * tanhf(t / cap) : t;
+  }
+}
+
+LEB_API int leb_softcap(float* z, float scale, float cap, size_t n, cudaStream_t st) {
+  if (n == 0) return 0;
+  leb_launch(softcap_kernel, dim3((unsigned)((n + 1023) / 1024)), dim3(256), 0, st, z, scale, cap, n);
+  LEB_CHECK_LAUNCH("leb_softcap");
+  return 0;
+}
+
 LEB_API int leb_activation(void* a, int out_dtype, const float* x, int ldx, int M, int F, int act, cudaStream_t st) {
   const size_t total = (size_t)M * F;
   if (total == 0) return 0;

@@ -4,7 +4,7 @@
 //   c_q = rmsnorm(W_dq h),  q_h = W_uq,h c_q = [q_h^n (dim) | q_h^r (rot)]      q_h^r rotated by position
 //   [a | r] = W_dkv h,  c = rmsnorm(a) (rank),  k^r = rotate(r) (rot)              cached: [c | k^r]
 //   k_h = W_uk,h c,  v_h = W_uv,h c
-//   s_h(i, j) = scale (q_h^n . k_h(j) + q_h^r . k^r(j)),  j <= i
+//   s_h(i, j) = scale (q_h^n . k_h(j) + q_h^r . k^r(j)),  j <= i (and in i's window or chunk where a layer has one)
 //   p = softmax over {s_h(i, j)} and one more logit sink_h that has no key and no value
 //   o_h = sum_j p_j v_h(j)
 //
@@ -22,10 +22,77 @@
 // sums are float; sinf/cosf are the full-range versions.
 #include "common.cuh"
 
-// Rotation of the first `rot_dims` of `n` numbers, pairs (2i, 2i + 1): (u, v) -> (u cos a - v sin a,
-// v cos a + u sin a), a = pos * inv_freq[i]; the rest passes unchanged.
-__device__ __forceinline__ float rot_pair(float u, float v, float c, float s, int odd) {
-  return odd ? v * c + u * s : u * c - v * s;
+// Rotation of the first `rot_dims` of a vector's numbers: pair t is (2t, 2t + 1), or with `neox` (t, t + rot_dims / 2);
+// (u, v) -> (u cos a - v sin a, v cos a + u sin a), a = pos * inv_freq[t]; the rest passes unchanged.  The unit t of
+// such a vector of `rot` numbers is pair t while t < rot_dims / 2, then single numbers.
+template <typename T, typename CT>
+__device__ __forceinline__ void rotate_unit(CT* __restrict__ dst, const T* __restrict__ src, int t, float pos,
+                                            const float* __restrict__ inv_freq, int rot_dims, int neox) {
+  const int half = rot_dims / 2;
+  if (t >= half) {
+    const int d = rot_dims + t - half;
+    dst[d] = from_f32<CT>(to_f32(src[d]));
+    return;
+  }
+  const int ia = neox ? t : 2 * t, ib = neox ? t + half : 2 * t + 1;
+  const float u = to_f32(src[ia]), v = to_f32(src[ib]);
+  const float a = pos * inv_freq[t];
+  const float c = cosf(a), s = sinf(a);
+  dst[ia] = from_f32<CT>(u * c - v * s);
+  dst[ib] = from_f32<CT>(v * c + u * s);
+}
+
+// The cache row [c | k^r] of row m: lat = `rank` numbers of the latent before its norm, then `rot` of the shared key part
+// before its rotation.  By the whole block; rows of padding sequences touch no cache.
+template <typename T, typename CT>
+__device__ __forceinline__ void latent_cache_row(const T* __restrict__ lat, int m, CT* __restrict__ pool,
+                                                 const int* __restrict__ block_table, int bt_width,
+                                                 const int* __restrict__ row_seq, const int* __restrict__ row_pos,
+                                                 const int* __restrict__ seq_slot, const float* __restrict__ wkv, float eps,
+                                                 const float* __restrict__ inv_freq, int rot_dims, int neox, int rank, int rot,
+                                                 int page_size, float* red) {
+  const int b = row_seq[m], pos = row_pos[m];
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < rank; i += blockDim.x) {
+    const float v = to_f32(lat[i]);
+    ss += v * v;
+  }
+  ss = block_sum(ss, red);
+  if (seq_slot[b] < 0) return;      // a padding sequence touches no cache
+  const int page = block_table[(size_t)b * bt_width + pos / page_size];
+  if (page < 0) return;
+  const float r = 1.0f / sqrtf(ss / (float)rank + eps);
+  CT* dst = pool + ((size_t)page * page_size + pos % page_size) * (size_t)(rank + rot);
+  for (int i = threadIdx.x; i < rank; i += blockDim.x) dst[i] = from_f32<CT>(to_f32(lat[i]) * r * wkv[i]);
+  for (int t = threadIdx.x; t < rot - rot_dims / 2; t += blockDim.x)
+    rotate_unit<T, CT>(dst + rank, lat + rank, t, (float)pos, inv_freq, rot_dims, neox);
+}
+
+// Row m of q [H * (dim + rot)] -> qn [H, M, dim_p] (the unrotated parts, head-major, zeros from dim to dim_p) and
+// qr [M, H, rot] (the rotated parts).  By the whole block; `wide`: 16-byte pieces.
+template <typename T>
+__device__ __forceinline__ void latent_split_row(T* __restrict__ qn, T* __restrict__ qr, const T* __restrict__ row, int m,
+                                                 float pos, const float* __restrict__ inv_freq, int rot_dims, int neox, int M,
+                                                 int H, int dim, int dim_p, int rot, bool wide) {
+  const int hw = dim + rot;
+  constexpr int PER = 16 / (int)sizeof(T);          // elements of a 16-byte piece
+  if (wide) {
+    const int pieces = dim / PER;
+    for (int i = threadIdx.x; i < H * pieces; i += blockDim.x) {
+      const int h = i / pieces, c = i - h * pieces;
+      reinterpret_cast<uint4*>(qn + ((size_t)h * M + m) * dim)[c] = reinterpret_cast<const uint4*>(row + h * hw)[c];
+    }
+  } else {
+    for (int i = threadIdx.x; i < H * dim_p; i += blockDim.x) {
+      const int h = i / dim_p, d = i - h * dim_p;
+      qn[((size_t)h * M + m) * dim_p + d] = d < dim ? row[h * hw + d] : from_f32<T>(0.f);
+    }
+  }
+  const int units = rot - rot_dims / 2;
+  for (int i = threadIdx.x; i < H * units; i += blockDim.x) {
+    const int h = i / units, t = i - h * units;
+    rotate_unit<T, T>(qr + ((size_t)m * H + h) * rot, row + h * hw + dim, t, pos, inv_freq, rot_dims, neox);
+  }
 }
 
 // One block per row.  in [M, ld_in]: columns [0, q_rank) the query latent before its norm, then
@@ -38,7 +105,7 @@ latent_prep_kernel(T* __restrict__ cq, const T* __restrict__ in, int ld_in, CT* 
                    const int* __restrict__ block_table, int bt_width, const int* __restrict__ row_seq,
                    const int* __restrict__ row_pos, const int* __restrict__ seq_slot,
                    const float* __restrict__ wq, const float* __restrict__ wkv, float eps,
-                   const float* __restrict__ inv_freq, int rot_dims, int q_rank, int rank, int rot,
+                   const float* __restrict__ inv_freq, int rot_dims, int neox, int q_rank, int rank, int rot,
                    int page_size) {
   __shared__ float red[33];
   pdl_wait();
@@ -50,89 +117,46 @@ latent_prep_kernel(T* __restrict__ cq, const T* __restrict__ in, int ld_in, CT* 
     ss += v * v;
   }
   ss = block_sum(ss, red);
-  float r = 1.0f / sqrtf(ss / (float)q_rank + eps);
+  const float r = 1.0f / sqrtf(ss / (float)q_rank + eps);
   for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
     cq[(size_t)m * q_rank + i] = from_f32<T>(to_f32(row[i]) * r * wq[i]);
   if (!pool) return;
-  const int b = row_seq[m], pos = row_pos[m];
-  const T* lat = row + q_rank;
-  ss = 0.f;
-  for (int i = threadIdx.x; i < rank; i += blockDim.x) {
-    const float v = to_f32(lat[i]);
-    ss += v * v;
-  }
-  ss = block_sum(ss, red);
-  if (seq_slot[b] < 0) return;      // a padding sequence touches no cache
-  const int page = block_table[(size_t)b * bt_width + pos / page_size];
-  if (page < 0) return;
-  r = 1.0f / sqrtf(ss / (float)rank + eps);
-  CT* dst = pool + ((size_t)page * page_size + pos % page_size) * (size_t)(rank + rot);
-  for (int i = threadIdx.x; i < rank; i += blockDim.x) dst[i] = from_f32<CT>(to_f32(lat[i]) * r * wkv[i]);
-  const T* kr = lat + rank;
-  for (int i = threadIdx.x; i < rot; i += blockDim.x) {
-    float v = to_f32(kr[i]);
-    if (i < rot_dims) {
-      const float a = (float)pos * inv_freq[i >> 1];
-      v = rot_pair(to_f32(kr[i & ~1]), to_f32(kr[i | 1]), cosf(a), sinf(a), i & 1);
-    }
-    dst[rank + i] = from_f32<CT>(v);
-  }
+  latent_cache_row<T, CT>(row + q_rank, m, pool, block_table, bt_width, row_seq, row_pos, seq_slot, wkv, eps, inv_freq, rot_dims,
+                          neox, rank, rot, page_size, red);
 }
 
-// q [M, H * (dim + rot)] -> qn [H, M, dim_p] (the unrotated parts, head-major, zeros from dim to
-// dim_p) and qr [M, H, rot] (the rotated parts).  One block per row.
+// q [M, H * (dim + rot)] -> qn and qr, one block per row.
 template <typename T>
 __global__ void __launch_bounds__(256)
 latent_q_split_kernel(T* __restrict__ qn, T* __restrict__ qr, const T* __restrict__ q,
-                      const int* __restrict__ row_pos, const float* __restrict__ inv_freq, int rot_dims,
-                      int M, int H, int dim, int dim_p, int rot) {
+                      const int* __restrict__ row_pos, const float* __restrict__ inv_freq, int rot_dims, int neox,
+                      int M, int H, int dim, int dim_p, int rot, int wide) {
   pdl_wait();
   const int m = blockIdx.x;
-  const int hw = dim + rot;
-  const T* row = q + (size_t)m * H * hw;
-  constexpr int PER = 16 / (int)sizeof(T);          // elements of a 16-byte piece
-  if (dim_p == dim && dim % PER == 0 && hw % PER == 0 && (((uintptr_t)q | (uintptr_t)qn) & 15) == 0) {
-    const int pieces = dim / PER;
-    for (int i = threadIdx.x; i < H * pieces; i += blockDim.x) {
-      const int h = i / pieces, c = i - h * pieces;
-      reinterpret_cast<uint4*>(qn + ((size_t)h * M + m) * dim)[c] = reinterpret_cast<const uint4*>(row + h * hw)[c];
-    }
-  } else {
-    for (int i = threadIdx.x; i < H * dim_p; i += blockDim.x) {
-      const int h = i / dim_p, d = i - h * dim_p;
-      qn[((size_t)h * M + m) * dim_p + d] = d < dim ? row[h * hw + d] : from_f32<T>(0.f);
-    }
-  }
-  const float pos = (float)row_pos[m];
-  if (rot % 2 == 0) {       // a thread per pair: one sine and cosine for both numbers
-    const int hp = rot / 2;
-    for (int i = threadIdx.x; i < H * hp; i += blockDim.x) {
-      const int h = i / hp, t = i - h * hp;
-      const T* r = row + h * hw + dim + 2 * t;
-      float u = to_f32(r[0]), v = to_f32(r[1]);
-      if (2 * t < rot_dims) {
-        const float a = pos * inv_freq[t];
-        const float c = cosf(a), sn = sinf(a);
-        const float u2 = u * c - v * sn;
-        v = v * c + u * sn;
-        u = u2;
-      }
-      T* o = qr + ((size_t)m * H + h) * rot + 2 * t;
-      o[0] = from_f32<T>(u);
-      o[1] = from_f32<T>(v);
-    }
-    return;
-  }
-  for (int i = threadIdx.x; i < H * rot; i += blockDim.x) {
-    const int h = i / rot, d = i - h * rot;
-    const T* r = row + h * hw + dim;
-    float v = to_f32(r[d]);
-    if (d < rot_dims) {
-      const float a = pos * inv_freq[d >> 1];
-      v = rot_pair(to_f32(r[d & ~1]), to_f32(r[d | 1]), cosf(a), sinf(a), d & 1);
-    }
-    qr[(size_t)m * H * rot + i] = from_f32<T>(v);
-  }
+  latent_split_row<T>(qn, qr, q + (size_t)m * H * (dim + rot), m, (float)row_pos[m], inv_freq, rot_dims, neox, M, H, dim, dim_p, rot,
+                      wide != 0);
+}
+
+// Both jobs in one launch where q comes straight from a projection of the row (no query latent): in [M, ld_in] holds
+// q [H * (dim + rot)], then (with `pool`) `rank` latent columns and `rot` columns of the shared key part.  Blocks (m, 0)
+// split q, blocks (m, 1) write the cache row.
+template <typename T>
+__global__ void __launch_bounds__(256)
+latent_rows_kernel(T* __restrict__ qn, T* __restrict__ qr, const T* __restrict__ in, int ld_in, T* __restrict__ pool,
+                   const int* __restrict__ block_table, int bt_width, const int* __restrict__ row_seq,
+                   const int* __restrict__ row_pos, const int* __restrict__ seq_slot, const float* __restrict__ wkv, float eps,
+                   const float* __restrict__ inv_freq, int rot_dims, int neox, int M, int H, int dim, int dim_p, int rank,
+                   int rot, int page_size, int wide) {
+  __shared__ float red[33];
+  pdl_trigger();   // the kernel after this one may start and wait (see common.cuh)
+  pdl_wait();
+  const int m = blockIdx.x;
+  const T* row = in + (size_t)m * ld_in;
+  if (blockIdx.y == 0)
+    latent_split_row<T>(qn, qr, row, m, (float)row_pos[m], inv_freq, rot_dims, neox, M, H, dim, dim_p, rot, wide != 0);
+  else
+    latent_cache_row<T, T>(row + H * (dim + rot), m, pool, block_table, bt_width, row_seq, row_pos, seq_slot, wkv, eps, inv_freq,
+                           rot_dims, neox, rank, rot, page_size, red);
 }
 
 // in [H, M, w] -> out [M, H * w], one piece per thread: an element, or 16 bytes where the rows allow it
@@ -164,7 +188,8 @@ latent_attention_kernel(T* __restrict__ out, int ld_out, float* __restrict__ par
                         const int* __restrict__ block_table, int bt_width, const int* __restrict__ seq_slot,
                         const int* __restrict__ seq_pos0, const int* __restrict__ seq_qstart,
                         const int* __restrict__ seq_qlen, const float* __restrict__ sink, int M, int H,
-                        int rank, int rot, int page_size, float scale, int QT, int HC, int n_splits) {
+                        int rank, int rot, int page_size, int window, int chunk, float scale, int QT, int HC,
+                        int n_splits) {
   extern __shared__ float sm[];
   pdl_wait();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -217,10 +242,10 @@ latent_attention_kernel(T* __restrict__ out, int ld_out, float* __restrict__ par
 
   const int kv_len = pos0 + qlen;
   const int pos_hi = pos0 + row_lo + nrows - 1;
-  const int n_tiles = pos_hi / 32 + 1;
-  const int per_split = (n_tiles + n_splits - 1) / n_splits;
-  const int t_lo = split * per_split;
-  const int t_hi = min(n_tiles, t_lo + per_split);
+  const int tile_first = first_key(pos0 + row_lo, window, chunk) / 32, tile_end = pos_hi / 32 + 1;
+  const int per_split = (tile_end - tile_first + n_splits - 1) / n_splits;
+  const int t_lo = tile_first + split * per_split;
+  const int t_hi = min(tile_end, t_lo + per_split);
 
   float mx[LAT_RPW], l[LAT_RPW], acc[LAT_RPW][HDL];
 #pragma unroll
@@ -250,13 +275,14 @@ latent_attention_kernel(T* __restrict__ out, int ld_out, float* __restrict__ par
       const int i = r / HC, j = r % HC;
       if (i >= nrows || j >= nheads) continue;
       const int qpos = pos0 + row_lo + i;
-      if (key0 > qpos) continue;   // the whole tile lies after this row
+      const int lo = first_key(qpos, window, chunk);
+      if (key0 > qpos || key0 + 31 < lo) continue;   // the whole tile lies after this row, or before what it reads
       const float* qv = q_s + r * dk;
       const float* kr = k_s + lane * KS;
       float s = 0.f;
       for (int d = 0; d < dk; d++) s += qv[d] * kr[d];
       s *= scale;
-      const bool valid = key0 + lane <= qpos;
+      const bool valid = key0 + lane <= qpos && key0 + lane >= lo;
       s = valid ? s : LAT_NEG;
       const float mn = fmaxf(mx[ri], warp_max(s));
       const float p = valid ? expf(s - mn) : 0.f;
@@ -338,10 +364,41 @@ __global__ void latent_merge_kernel(T* __restrict__ out, int ld_out, const float
 }
 
 // ---------------------------------------------------------------------------------------------
+// Whether the unrotated parts of q move in 16-byte pieces: sizes, the row stride and the addresses on that grid.
+static bool latent_wide(int dtype, int dim, int dim_p, int stride, uintptr_t addr) {
+  const int per = dtype == LEB_BF16 ? 8 : 4;
+  return dim_p == dim && dim % per == 0 && stride % per == 0 && (addr & 15) == 0;
+}
+
+LEB_API int leb_latent_rows(void* qn, void* qr, const void* in, int ld_in, int dtype, void* pool, const int* block_table,
+                            int bt_width, const int* row_seq, const int* row_pos, const int* seq_slot, const float* wkv,
+                            float eps, const float* inv_freq, int rot_dims, int neox, int M, int H, int dim, int dim_p,
+                            int rank, int rot, int page_size, cudaStream_t st) {
+  if (M <= 0) return 0;
+  LEB_REQUIRE(H >= 1 && dim >= 1 && dim_p >= dim && rot >= 0, "leb_latent_rows: sizes out of range");
+  LEB_REQUIRE(!pool || (rank >= 1 && wkv && block_table && row_seq && seq_slot),
+              "leb_latent_rows: a cache write needs the latent's size, its norm weight and the step's tables");
+  LEB_REQUIRE(row_pos && rot_dims >= 0 && rot_dims <= rot && rot_dims % 2 == 0 && (rot_dims == 0 || inv_freq),
+              "leb_latent_rows: %d rotated dimensions of %d", rot_dims, rot);
+  LEB_REQUIRE(dtype == LEB_F32 || dtype == LEB_BF16, "leb_latent_rows: unknown dtype %d", dtype);
+  const int wide = latent_wide(dtype, dim, dim_p, dim + rot, (uintptr_t)in | (uintptr_t)qn) && ld_in % (dtype == LEB_BF16 ? 8 : 4) == 0;
+  const dim3 grid(M, pool ? 2 : 1), block(256);
+  if (dtype == LEB_F32)
+    leb_launch(latent_rows_kernel<float>, grid, block, 0, st, (float*)qn, (float*)qr, (const float*)in, ld_in, (float*)pool,
+               block_table, bt_width, row_seq, row_pos, seq_slot, wkv, eps, inv_freq, rot_dims, neox, M, H, dim, dim_p, rank, rot,
+               page_size, wide);
+  else
+    leb_launch(latent_rows_kernel<bf16>, grid, block, 0, st, (bf16*)qn, (bf16*)qr, (const bf16*)in, ld_in, (bf16*)pool,
+               block_table, bt_width, row_seq, row_pos, seq_slot, wkv, eps, inv_freq, rot_dims, neox, M, H, dim, dim_p, rank, rot,
+               page_size, wide);
+  LEB_CHECK_LAUNCH("leb_latent_rows");
+  return 0;
+}
+
 LEB_API int leb_latent_prep(void* cq, const void* in, int ld_in, int dtype, void* pool, const int* block_table,
                             int bt_width, const int* row_seq, const int* row_pos, const int* seq_slot,
                             const float* wq, const float* wkv, float eps, const float* inv_freq, int rot_dims,
-                            int M, int q_rank, int rank, int rot, int page_size, cudaStream_t st) {
+                            int neox, int M, int q_rank, int rank, int rot, int page_size, cudaStream_t st) {
   if (M <= 0) return 0;
   LEB_REQUIRE(q_rank >= 1 && wq, "leb_latent_prep: the query latent needs a width and a norm weight");
   LEB_REQUIRE(!pool || (rank >= 1 && rot >= 0 && wkv && block_table && row_seq && row_pos && seq_slot),
@@ -351,11 +408,11 @@ LEB_API int leb_latent_prep(void* cq, const void* in, int ld_in, int dtype, void
   LebPlainLaunches plain(true);
   if (dtype == LEB_F32)
     leb_launch(latent_prep_kernel<float, float>, dim3(M), dim3(128), 0, st, (float*)cq, (const float*)in, ld_in,
-               (float*)pool, block_table, bt_width, row_seq, row_pos, seq_slot, wq, wkv, eps, inv_freq, rot_dims,
+               (float*)pool, block_table, bt_width, row_seq, row_pos, seq_slot, wq, wkv, eps, inv_freq, rot_dims, neox,
                q_rank, rank, rot, page_size);
   else if (dtype == LEB_BF16)
     leb_launch(latent_prep_kernel<bf16, bf16>, dim3(M), dim3(128), 0, st, (bf16*)cq, (const bf16*)in, ld_in,
-               (bf16*)pool, block_table, bt_width, row_seq, row_pos, seq_slot, wq, wkv, eps, inv_freq, rot_dims,
+               (bf16*)pool, block_table, bt_width, row_seq, row_pos, seq_slot, wq, wkv, eps, inv_freq, rot_dims, neox,
                q_rank, rank, rot, page_size);
   else
     return leb_fail("leb_latent_prep: unknown dtype %d", dtype);
@@ -364,19 +421,20 @@ LEB_API int leb_latent_prep(void* cq, const void* in, int ld_in, int dtype, void
 }
 
 LEB_API int leb_latent_q_split(void* qn, void* qr, const void* q, int dtype, const int* row_pos,
-                               const float* inv_freq, int rot_dims, int M, int H, int dim, int dim_p, int rot,
+                               const float* inv_freq, int rot_dims, int neox, int M, int H, int dim, int dim_p, int rot,
                                cudaStream_t st) {
   if (M <= 0) return 0;
   LEB_REQUIRE(H >= 1 && dim >= 1 && dim_p >= dim && rot >= 0, "leb_latent_q_split: sizes out of range");
   LEB_REQUIRE(rot_dims >= 0 && rot_dims <= rot && rot_dims % 2 == 0 && (rot_dims == 0 || inv_freq),
               "leb_latent_q_split: %d rotated dimensions of %d", rot_dims, rot);
+  const int wide = latent_wide(dtype, dim, dim_p, dim + rot, (uintptr_t)q | (uintptr_t)qn);
   LebPlainLaunches plain(true);
   if (dtype == LEB_F32)
     leb_launch(latent_q_split_kernel<float>, dim3(M), dim3(256), 0, st, (float*)qn, (float*)qr, (const float*)q,
-               row_pos, inv_freq, rot_dims, M, H, dim, dim_p, rot);
+               row_pos, inv_freq, rot_dims, neox, M, H, dim, dim_p, rot, wide);
   else if (dtype == LEB_BF16)
     leb_launch(latent_q_split_kernel<bf16>, dim3(M), dim3(256), 0, st, (bf16*)qn, (bf16*)qr, (const bf16*)q, row_pos,
-               inv_freq, rot_dims, M, H, dim, dim_p, rot);
+               inv_freq, rot_dims, neox, M, H, dim, dim_p, rot, wide);
   else
     return leb_fail("leb_latent_q_split: unknown dtype %d", dtype);
   LEB_CHECK_LAUNCH("leb_latent_q_split");
@@ -406,7 +464,8 @@ template <typename T, int HDL>
 static int launch_latent(void* out, int ld_out, float* part, const void* qt, const void* qr, const void* pool,
                          const int* block_table, int bt_width, const int* seq_slot, const int* seq_pos0,
                          const int* seq_qstart, const int* seq_qlen, const float* sink, int M, int B, int H, int rank,
-                         int rot, int page_size, float scale, int max_qlen, int n_splits, cudaStream_t st) {
+                         int rot, int page_size, int window, int chunk, float scale, int max_qlen, int n_splits,
+                         cudaStream_t st) {
   const int HC = H < 8 ? H : 8;
   int QT = 32 / HC;
   if (QT > max_qlen) QT = max_qlen;
@@ -424,7 +483,7 @@ static int launch_latent(void* out, int ld_out, float* part, const void* qt, con
   LEB_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "leb_latent_attention: grid too large (%u, %u)", grid.y, grid.z);
   leb_launch(kern, grid, dim3(32 * LAT_WARPS), smem, st, (T*)out, ld_out, part, (const T*)qt, (const T*)qr,
              (const T*)pool, block_table, bt_width, seq_slot, seq_pos0, seq_qstart, seq_qlen, sink, M, H, rank, rot,
-             page_size, scale, QT, HC, n_splits);
+             page_size, window, chunk, scale, QT, HC, n_splits);
   LEB_CHECK_LAUNCH("leb_latent_attention");
   return 0;
 }
@@ -434,20 +493,21 @@ extern "C" int leb_latent_attention_mma_supported(int rank, int rot, int page_si
 extern "C" int leb_latent_attention_mma(void* out, float* part, const void* qt, const void* qr, const void* pool,
                                         const int* block_table, int bt_width, const int* seq_slot, const int* seq_pos0,
                                         const int* seq_qstart, const int* seq_qlen, const float* sink, int M, int B, int H,
-                                        int rank, int rot, int page_size, float scale, int max_qlen, int n_splits,
-                                        cudaStream_t st);
+                                        int rank, int rot, int page_size, int window, int chunk, int wide,
+                                        float scale, int max_qlen, int n_splits, cudaStream_t st);
 static int g_latent_mma = 1;
 LEB_API void leb_set_latent_mma(int on) { g_latent_mma = on ? 1 : 0; }
 
 // qt [H, M, rank] (queries taken into the latent space), qr [M, H, rot] (rotated parts), pool
 // [page][page_size][rank + rot], sink [H] float or null; out [H, M, ld_out] (ld_out >= rank, the
-// rest zeros).  part: float scratch of M*H*n_splits*(rank+2), used when n_splits > 1 (then every
+// rest zeros).  window / chunk > 0: a row reads its last `window` positions / its own chunk only; wide: the weights of
+// the tensor-core kernel enter the product with the values as two terms (the general kernel's are float anyway).  part: float scratch of M*H*n_splits*(rank+2), used when n_splits > 1 (then every
 // sequence brings one row).
 LEB_API int leb_latent_attention(void* out, int ld_out, float* part, const void* qt, const void* qr, const void* pool,
                                  int dtype, const int* block_table, int bt_width, const int* seq_slot,
                                  const int* seq_pos0, const int* seq_qstart, const int* seq_qlen, const float* sink,
-                                 int M, int B, int H, int rank, int rot, int page_size, float scale, int max_qlen,
-                                 int n_splits, cudaStream_t st) {
+                                 int M, int B, int H, int rank, int rot, int page_size, int window, int chunk, int wide,
+                                 float scale, int max_qlen, int n_splits, cudaStream_t st) {
   if (M <= 0 || B <= 0) return 0;
   LEB_REQUIRE(rank >= 1 && rank <= 512, "leb_latent_attention: latent size %d outside 1..512", rank);
   LEB_REQUIRE(rot >= 0 && rot <= 256, "leb_latent_attention: %d rotated dimensions outside 0..256", rot);
@@ -461,12 +521,12 @@ LEB_API int leb_latent_attention(void* out, int ld_out, float* part, const void*
                    (((uintptr_t)qt | (uintptr_t)qr | (uintptr_t)pool) & 15) == 0;
 #define LEB_LAT(T, L)                                                                                              \
   launch_latent<T, L>(out, ld_out, part, qt, qr, pool, block_table, bt_width, seq_slot, seq_pos0, seq_qstart, seq_qlen, \
-                      sink, M, B, H, rank, rot, page_size, scale, max_qlen, n_splits, st)
+                      sink, M, B, H, rank, rot, page_size, window, chunk, scale, max_qlen, n_splits, st)
 #define LEB_LAT_T(T) \
   (rank <= 32 ? LEB_LAT(T, 1) : rank <= 64 ? LEB_LAT(T, 2) : rank <= 128 ? LEB_LAT(T, 4) : rank <= 256 ? LEB_LAT(T, 8) : LEB_LAT(T, 16))
   if (mma)
     rc = leb_latent_attention_mma(out, part, qt, qr, pool, block_table, bt_width, seq_slot, seq_pos0, seq_qstart, seq_qlen,
-                                  sink, M, B, H, rank, rot, page_size, scale, max_qlen, n_splits, st);
+                                  sink, M, B, H, rank, rot, page_size, window, chunk, wide, scale, max_qlen, n_splits, st);
   else if (dtype == LEB_F32) rc = LEB_LAT_T(float);
   else if (dtype == LEB_BF16) rc = LEB_LAT_T(bf16);
   else return leb_fail("leb_latent_attention: unknown dtype %d", dtype);

@@ -40,14 +40,17 @@ __device__ __forceinline__ uint32_t lm_smem(const void* p) { return (uint32_t)__
 
 // NT: n8-tiles of the latent a warp sums at most (rank <= 32 * NT).  BN: cached rows per tile, 64 where two
 // stages of them fit shared memory beside the queries (rows of up to 512 numbers), else 32.
-template <int NT, int BN>
+// WIDE: the softmax weights enter the second product as two bfloat16 terms, p = hi + lo (16 significant bits; the sums
+// of p are float either way).
+template <int NT, int BN, bool WIDE>
 __global__ void __launch_bounds__(256, 1)
 latent_attention_mma_kernel(bf16* __restrict__ out, float* __restrict__ part, const bf16* __restrict__ qt,
                             const bf16* __restrict__ qr, const bf16* __restrict__ pool,
                             const int* __restrict__ block_table, int bt_width, const int* __restrict__ seq_slot,
                             const int* __restrict__ seq_pos0, const int* __restrict__ seq_qstart,
                             const int* __restrict__ seq_qlen, const float* __restrict__ sink, int M, int H,
-                            int rank, int rot, int page_size, float scale, int QT, int HC, int n_splits) {
+                            int rank, int rot, int page_size, int window, int chunk, float scale, int QT, int HC,
+                            int n_splits) {
   extern __shared__ __align__(16) unsigned char lm_sm[];
   pdl_wait();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -75,7 +78,8 @@ latent_attention_mma_kernel(bf16* __restrict__ out, float* __restrict__ part, co
   bf16* k_s = q_s + LM_BM * LDK;                                   // [2][32][LDK]
   float* s_s = reinterpret_cast<float*>(k_s + 2 * LM_BN * LDK);    // [64][BN + 1]
   bf16* p_s = reinterpret_cast<bf16*>(s_s + LM_BM * LDS);          // [64][LDP]
-  float* c_s = reinterpret_cast<float*>(p_s + LM_BM * LDP);        // [64]
+  bf16* pl_s = p_s + LM_BM * LDP;                                  // [64][LDP] (WIDE)
+  float* c_s = reinterpret_cast<float*>(p_s + (WIDE ? 2 : 1) * LM_BM * LDP);   // [64]
 
   if (slot < 0) {                            // a padding sequence: defined output, no cache access
     for (int r = warp; r < R; r += 8) {
@@ -109,15 +113,15 @@ latent_attention_mma_kernel(bf16* __restrict__ out, float* __restrict__ part, co
     }
     *reinterpret_cast<uint4*>(q_s + (size_t)r * LDK + c * 8) = v;
   }
-  for (int idx = tid; idx < LM_BM * LDP; idx += 256) p_s[idx] = __float2bfloat16_rn(0.f);
+  for (int idx = tid; idx < (WIDE ? 2 : 1) * LM_BM * LDP; idx += 256) p_s[idx] = __float2bfloat16_rn(0.f);
   if (tid < LM_BM) c_s[tid] = 1.f;
 
   const int kv_len = pos0 + qlen;
   const int pos_hi = pos0 + row_lo + nrows - 1;
-  const int n_tiles = pos_hi / LM_BN + 1;
-  const int per_split = (n_tiles + n_splits - 1) / n_splits;
-  const int t_lo = split * per_split;
-  const int t_hi = min(n_tiles, t_lo + per_split);
+  const int tile_first = first_key(pos0 + row_lo, window, chunk) / LM_BN, tile_end = pos_hi / LM_BN + 1;
+  const int per_split = (tile_end - tile_first + n_splits - 1) / n_splits;
+  const int t_lo = tile_first + split * per_split;
+  const int t_hi = min(tile_end, t_lo + per_split);
 
   auto load_tile = [&](int stage, int tile) {
     const int key0 = tile * LM_BN;
@@ -207,12 +211,13 @@ latent_attention_mma_kernel(bf16* __restrict__ out, float* __restrict__ part, co
       for (int half = 0; half < 2; half++) {
         const int r = 16 * s_mt + g + 8 * half;
         const int qpos = pos0 + row_lo + r / HC;
+        const int lo = first_key(qpos, window, chunk);
 #pragma unroll
         for (int nt = 0; nt < KW / 8; nt++)
 #pragma unroll
           for (int e = 0; e < 2; e++) {
             const int col = KW * s_kh + 8 * nt + 2 * tg + e;
-            s_s[r * LDS + col] = key0 + col <= qpos ? (s[0][nt][2 * half + e] + s[1][nt][2 * half + e]) * scale : LM_NEG;
+            s_s[r * LDS + col] = key0 + col <= qpos && key0 + col >= lo ? (s[0][nt][2 * half + e] + s[1][nt][2 * half + e]) * scale : LM_NEG;
           }
       }
     }
@@ -236,7 +241,7 @@ latent_attention_mma_kernel(bf16* __restrict__ out, float* __restrict__ part, co
       float tsum = 0.f;
 #pragma unroll
       for (int c = 0; c < BN / 32; c++) {
-        uint32_t pk[4];
+        uint32_t pk[4], pl[4];
 #pragma unroll
         for (int j = 0; j < 8; j += 2) {
           const float p0 = sv[8 * c + j] > 0.5f * LM_NEG ? expf(sv[8 * c + j] - mn) : 0.f;
@@ -244,8 +249,13 @@ latent_attention_mma_kernel(bf16* __restrict__ out, float* __restrict__ part, co
           tsum += p0 + p1;
           __nv_bfloat162 two = __floats2bfloat162_rn(p0, p1);
           pk[j >> 1] = *reinterpret_cast<uint32_t*>(&two);
+          if (WIDE) {
+            __nv_bfloat162 rest = __floats2bfloat162_rn(p0 - __bfloat162float(two.x), p1 - __bfloat162float(two.y));
+            pl[j >> 1] = *reinterpret_cast<uint32_t*>(&rest);
+          }
         }
         *reinterpret_cast<uint4*>(p_s + sm_r * LDP + 32 * c + 8 * sm_q) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+        if (WIDE) *reinterpret_cast<uint4*>(pl_s + sm_r * LDP + 32 * c + 8 * sm_q) = make_uint4(pl[0], pl[1], pl[2], pl[3]);
       }
       tsum += __shfl_xor_sync(0xffffffffu, tsum, 1);
       tsum += __shfl_xor_sync(0xffffffffu, tsum, 2);
@@ -273,9 +283,13 @@ latent_attention_mma_kernel(bf16* __restrict__ out, float* __restrict__ part, co
       const bool two = 32 * o_mh + 16 < R;
 #pragma unroll
       for (int ks = 0; ks < BN / 16; ks++) {
-        uint32_t a[2][4], bb[4], bn[4];
+        uint32_t a[2][4], al[WIDE ? 2 : 1][4], bb[4], bn[4];
         lm_ldsm4(a[0], p_addr + ks * 32);
         lm_ldsm4(a[1], p_addr + 16 * LDP * 2 + ks * 32);
+        if (WIDE) {
+          lm_ldsm4(al[0], p_addr + LM_BM * LDP * 2 + ks * 32);
+          lm_ldsm4(al[WIDE ? 1 : 0], p_addr + (LM_BM + 16) * LDP * 2 + ks * 32);
+        }
         const uint32_t v_addr = k_base + vb_off + (uint32_t)(ks * 16 * LDK * 2);
         lm_ldsm4t(bb, v_addr);
 #pragma unroll
@@ -287,6 +301,14 @@ latent_attention_mma_kernel(bf16* __restrict__ out, float* __restrict__ part, co
             if (two) {
               lm_mma(o[1][2 * np], a[1], bb[0], bb[1]);
               if (2 * np + 1 < ntu) lm_mma(o[1][2 * np + 1], a[1], bb[2], bb[3]);
+            }
+            if (WIDE) {
+              lm_mma(o[0][2 * np], al[0], bb[0], bb[1]);
+              if (2 * np + 1 < ntu) lm_mma(o[0][2 * np + 1], al[0], bb[2], bb[3]);
+              if (two) {
+                lm_mma(o[1][2 * np], al[WIDE ? 1 : 0], bb[0], bb[1]);
+                if (2 * np + 1 < ntu) lm_mma(o[1][2 * np + 1], al[WIDE ? 1 : 0], bb[2], bb[3]);
+              }
             }
           }
 #pragma unroll
@@ -349,22 +371,29 @@ latent_attention_mma_kernel(bf16* __restrict__ out, float* __restrict__ part, co
   }
 }
 
+// Shared memory of a block: queries, two stages of cached rows of dk numbers, scores, weights (one or two terms), factors.
+static size_t lm_smem_bytes(int dk, int bn, bool wide) {
+  return (size_t)(LM_BM + 2 * bn) * (dk + 8) * 2 + (size_t)LM_BM * (bn + 1) * 4 + (size_t)(wide ? 2 : 1) * LM_BM * (bn + 8) * 2 +
+         LM_BM * 4;
+}
+
 // Whether the tensor-core kernel takes these sizes (bfloat16 only; the caller checks the type).
 LEB_API int leb_latent_attention_mma_supported(int rank, int rot, int page_size) {
   return rank >= 32 && rank <= 512 && rank % 32 == 0 && rot >= 0 && rot <= 256 && rot % 16 == 0 && page_size % 64 == 0;
 }
 
-template <int NT, int BN>
+template <int NT, int BN, bool WIDE>
 static int launch_latent_mma(bf16* out, float* part, const bf16* qt, const bf16* qr, const bf16* pool,
                              const int* block_table, int bt_width, const int* seq_slot, const int* seq_pos0,
                              const int* seq_qstart, const int* seq_qlen, const float* sink, int M, int B, int H, int rank,
-                             int rot, int page_size, float scale, int max_qlen, int n_splits, cudaStream_t st) {
+                             int rot, int page_size, int window, int chunk, float scale, int max_qlen, int n_splits,
+                             cudaStream_t st) {
   const int HC = H < LM_BM ? H : LM_BM;
   int QT = LM_BM / HC;
   if (QT > max_qlen) QT = max_qlen;
   const int dk = rank + rot;
-  const size_t smem = (size_t)(LM_BM + 2 * BN) * (dk + 8) * 2 + (size_t)LM_BM * (BN + 1) * 4 + (size_t)LM_BM * (BN + 8) * 2 + LM_BM * 4;
-  auto kern = latent_attention_mma_kernel<NT, BN>;
+  const size_t smem = lm_smem_bytes(dk, BN, WIDE);
+  auto kern = latent_attention_mma_kernel<NT, BN, WIDE>;
   static size_t smem_set = 0;
   if (smem > 48 * 1024 && smem > smem_set) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -374,7 +403,7 @@ static int launch_latent_mma(bf16* out, float* part, const bf16* qt, const bf16*
   dim3 grid(ceil_div(max_qlen, QT), ceil_div(H, HC), B * n_splits);
   LEB_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "leb_latent_attention_mma: grid too large (%u, %u)", grid.y, grid.z);
   leb_launch(kern, grid, dim3(256), smem, st, out, part, qt, qr, pool, block_table, bt_width, seq_slot, seq_pos0,
-             seq_qstart, seq_qlen, sink, M, H, rank, rot, page_size, scale, QT, HC, n_splits);
+             seq_qstart, seq_qlen, sink, M, H, rank, rot, page_size, window, chunk, scale, QT, HC, n_splits);
   LEB_CHECK_LAUNCH("leb_latent_attention_mma");
   return 0;
 }
@@ -384,8 +413,8 @@ static int launch_latent_mma(bf16* out, float* part, const bf16* qt, const bf16*
 LEB_API int leb_latent_attention_mma(void* out, float* part, const void* qt, const void* qr, const void* pool,
                                      const int* block_table, int bt_width, const int* seq_slot, const int* seq_pos0,
                                      const int* seq_qstart, const int* seq_qlen, const float* sink, int M, int B, int H,
-                                     int rank, int rot, int page_size, float scale, int max_qlen, int n_splits,
-                                     cudaStream_t st) {
+                                     int rank, int rot, int page_size, int window, int chunk, int wide, float scale,
+                                     int max_qlen, int n_splits, cudaStream_t st) {
   if (M <= 0 || B <= 0) return 0;
   LEB_REQUIRE(leb_latent_attention_mma_supported(rank, rot, page_size),
               "leb_latent_attention_mma: latent %d + %d with pages of %d is not a shape of this kernel", rank, rot, page_size);
@@ -393,13 +422,15 @@ LEB_API int leb_latent_attention_mma(void* out, float* part, const void* qt, con
               "leb_latent_attention_mma: splits need single-row sequences and scratch");
   LEB_REQUIRE((((uintptr_t)qt | (uintptr_t)qr | (uintptr_t)pool) & 15) == 0, "leb_latent_attention_mma: operands must be 16-byte aligned");
   LebPlainLaunches plain(true);
-#define LEB_LM(NT_, BN_)                                                                                                   \
-  launch_latent_mma<NT_, BN_>((bf16*)out, part, (const bf16*)qt, (const bf16*)qr, (const bf16*)pool, block_table, bt_width, \
-                              seq_slot, seq_pos0, seq_qstart, seq_qlen, sink, M, B, H, rank, rot, page_size, scale, max_qlen,  \
-                              n_splits, st)
+#define LEB_LM_W(NT_, BN_, W_)                                                                                             \
+  launch_latent_mma<NT_, BN_, W_>((bf16*)out, part, (const bf16*)qt, (const bf16*)qr, (const bf16*)pool, block_table, bt_width, \
+                              seq_slot, seq_pos0, seq_qstart, seq_qlen, sink, M, B, H, rank, rot, page_size, window, chunk, scale, \
+                              max_qlen, n_splits, st)
+#define LEB_LM(NT_, BN_) (wide ? LEB_LM_W(NT_, BN_, true) : LEB_LM_W(NT_, BN_, false))
   if (rank <= 64) return LEB_LM(2, 64);
   if (rank <= 128) return LEB_LM(4, 64);
-  if (rank <= 256) return LEB_LM(8, 64);
+  if (rank <= 256 && lm_smem_bytes(rank + rot, 64, wide != 0) <= 227 * 1024) return LEB_LM(8, 64);
   return LEB_LM(16, 32);         // two stages of 64 rows of up to 768 numbers would not fit beside the queries
 #undef LEB_LM
+#undef LEB_LM_W
 }

@@ -1,4 +1,4 @@
-// Per-head RMSNorm on q and k, rotary position encoding, and the write of k and v into the
+// RMSNorm on q and k (per head, or over the whole projected row), rotary position encoding, and the write of k and v into the
 // paged cache, one launch for all rows of a step.
 //
 // Order as in the reference (src/dense.rs:119-128): norm each head of q and k over head_dim with
@@ -253,6 +253,176 @@ __global__ void __launch_bounds__(ROPE_WARPS * 32) qk_rope_store_lanes_kernel(
       }
     }
   }
+}
+
+// The same job where q and k are normed over their whole projected row (all heads at once, a weight per number of the
+// row) instead of head by head.  Block (m, 0): row m's q, block (m, 1): its k (sum of squares, norm, rotation, q out or
+// cache write); blocks (x >= M, 0): value tiles as above.
+// FAST (bfloat16, adjacent pairs, heads stored as wide as they are and a multiple of 8): a thread keeps its pieces of
+// eight numbers in registers (up to NC of them) between the sum and the rotation.
+template <typename T, typename CT, bool FAST, int NC>
+__global__ void __launch_bounds__(256) qk_row_norm_rope_store_kernel(
+    T* __restrict__ q_out, const T* __restrict__ q_in, int q_stride, const T* __restrict__ k_in,
+    const T* __restrict__ v_in, int kv_stride, CT* __restrict__ k_pool, CT* __restrict__ v_pool,
+    const int* __restrict__ block_table, int bt_width, const int* __restrict__ row_seq,
+    const int* __restrict__ row_pos, const int* __restrict__ seq_slot,
+    const float* __restrict__ q_norm_w, const float* __restrict__ k_norm_w, float eps,
+    const float* __restrict__ inv_freq, int rope_dim, int neox, int M, int nh, int nkv, int hd,
+    int page_size, int vd, int hin, int vin) {
+  extern __shared__ __align__(16) float sm[];
+  __shared__ float red[33];
+  pdl_trigger();   // the kernel after this one may start and wait (see common.cuh)
+  pdl_wait();
+  if ((int)blockIdx.x >= M) {
+    if (blockIdx.y == 0)
+      store_value_tile<T, CT>(blockIdx.x - M, v_in, kv_stride, v_pool, block_table, bt_width, row_seq, row_pos,
+                              seq_slot, M, nkv, vd, page_size, 0, eps, vin);
+    return;
+  }
+  const int m = blockIdx.x;
+  const bool is_q = blockIdx.y == 0;
+  const int b = row_seq[m], pos = row_pos[m];
+  const int heads = is_q ? nh : nkv, n = heads * hin, half = rope_dim / 2;
+  CT* kbase = nullptr;
+  if (!is_q) {
+    if (seq_slot[b] < 0) return;     // padding rows and positions outside what the layer keeps own no cache
+    const int page = block_table[(size_t)b * bt_width + pos / page_size];
+    if (page < 0) return;
+    kbase = k_pool + ((size_t)page * nkv * page_size + pos % page_size) * hd;
+  }
+  const T* src = is_q ? q_in + (size_t)m * q_stride : k_in + (size_t)m * kv_stride;
+  const float* nw = is_q ? q_norm_w : k_norm_w;
+  float* cs = sm;                    // [half] cosine, [half] sine
+  float* row = sm + rope_dim;        // [heads * hin] (not FAST)
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    const float th = (float)pos * inv_freq[i];
+    cs[i] = cosf(th);
+    cs[half + i] = sinf(th);
+  }
+  float ss = 0.f;
+  if constexpr (FAST) {
+    const int pieces = n / 8, ppd = hd / 8;
+    uint4 v[NC];
+#pragma unroll
+    for (int c = 0; c < NC; c++) {
+      const int p = threadIdx.x + c * 256;
+      if (p < pieces) {
+        v[c] = reinterpret_cast<const uint4*>(src)[p];
+        const bf16* e = reinterpret_cast<const bf16*>(&v[c]);
+#pragma unroll
+        for (int j = 0; j < 8; j++) ss += to_f32(e[j]) * to_f32(e[j]);
+      }
+    }
+    ss = block_sum(ss, red);
+    const float r = 1.0f / sqrtf(ss / (float)n + eps);
+#pragma unroll
+    for (int c = 0; c < NC; c++) {
+      const int p = threadIdx.x + c * 256;
+      if (p >= pieces) break;
+      const int h = p / ppd, d0 = (p - h * ppd) * 8;
+      const bf16* e = reinterpret_cast<const bf16*>(&v[c]);
+      const float4 wa = reinterpret_cast<const float4*>(nw)[2 * p], wb = reinterpret_cast<const float4*>(nw)[2 * p + 1];
+      const float ww[8] = {wa.x, wa.y, wa.z, wa.w, wb.x, wb.y, wb.z, wb.w};
+      uint4 o;
+      uint32_t* op = reinterpret_cast<uint32_t*>(&o);
+#pragma unroll
+      for (int j = 0; j < 4; j++) {
+        float a = to_f32(e[2 * j]) * r * ww[2 * j], bb = to_f32(e[2 * j + 1]) * r * ww[2 * j + 1];
+        const int pi = d0 / 2 + j;
+        if (pi < half) {
+          const float c0 = cs[pi], s0 = cs[half + pi];
+          const float a2 = a * c0 - bb * s0;
+          bb = a * s0 + bb * c0;
+          a = a2;
+        }
+        __nv_bfloat162 two = __floats2bfloat162_rn(a, bb);
+        op[j] = *reinterpret_cast<uint32_t*>(&two);
+      }
+      CT* dst = is_q ? (CT*)(q_out + ((size_t)m * nh + h) * hd) : kbase + (size_t)h * page_size * hd;
+      *reinterpret_cast<uint4*>(dst + d0) = o;
+    }
+  } else {
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+      const float x = to_f32(src[i]);
+      row[i] = x;
+      ss += x * x;
+    }
+    ss = block_sum(ss, red);
+    const float r = 1.0f / sqrtf(ss / (float)n + eps);
+    // units of a head: `half` rotated pairs, then the numbers that pass, then the zeros a wider stored head ends with
+    const int units = half + hd - rope_dim;
+    for (int i = threadIdx.x; i < heads * units; i += blockDim.x) {
+      const int h = i / units, u = i - h * units;
+      const float* hv = row + h * hin;
+      const float* hw = nw + h * hin;
+      T* qo = q_out + ((size_t)m * nh + h) * hd;
+      CT* ko = is_q ? nullptr : kbase + (size_t)h * page_size * hd;
+      if (u < half) {
+        const int ia = neox ? u : 2 * u, ib = neox ? u + half : 2 * u + 1;
+        const float a = hv[ia] * r * hw[ia], bb = hv[ib] * r * hw[ib];
+        const float oa = a * cs[u] - bb * cs[half + u], ob = a * cs[half + u] + bb * cs[u];
+        if (is_q) { qo[ia] = from_f32<T>(oa); qo[ib] = from_f32<T>(ob); }
+        else { ko[ia] = from_f32<CT>(oa); ko[ib] = from_f32<CT>(ob); }
+      } else {
+        const int d = rope_dim + u - half;
+        const float a = d < hin ? hv[d] * r * hw[d] : 0.f;
+        if (is_q) qo[d] = from_f32<T>(a);
+        else ko[d] = from_f32<CT>(a);
+      }
+    }
+  }
+}
+
+// q, k and v of a step's rows: the root mean square of the whole q row and of the whole k row (weights [nh * hin] and
+// [nkv * hin]), rotation of every head, q out and the write of k and v into the pages.  k_in null: q alone.
+LEB_API int leb_qk_row_norm_rope_store(void* q_out, const void* q_in, int q_stride, const void* k_in,
+                                       const void* v_in, int kv_stride, void* k_pool, void* v_pool,
+                                       int dtype, const int* block_table, int bt_width, const int* row_seq,
+                                       const int* row_pos, const int* seq_slot, const float* q_norm_w,
+                                       const float* k_norm_w, float eps, const float* inv_freq, int rope_dim,
+                                       int neox, int M, int nh, int nkv, int hd, int page_size, int vd,
+                                       int hin, int vin, cudaStream_t st) {
+  if (M <= 0) return 0;
+  if (!inv_freq) rope_dim = 0;
+  if (hin <= 0) hin = hd;
+  if (vd <= 0) vd = hd;
+  if (vin <= 0) vin = vd;
+  LEB_REQUIRE(nh >= 1 && nkv >= 1 && hd >= 1 && hin <= hd && vin <= vd && rope_dim >= 0 && rope_dim <= hin && rope_dim % 2 == 0,
+              "leb_qk_row_norm_rope_store: heads %d/%d of %d (stored %d), %d rotated, values of %d (stored %d)", nh, nkv, hin, hd,
+              rope_dim, vin, vd);
+  LEB_REQUIRE(q_norm_w && (!k_in || k_norm_w), "leb_qk_row_norm_rope_store: the rows' norm weights are required");
+  LEB_REQUIRE(dtype == LEB_F32 || dtype == LEB_BF16, "leb_qk_row_norm_rope_store: unknown dtype %d", dtype);
+  const int tiles = k_in ? ceil_div(M, VT_ROWS) * nkv : 0;
+  const dim3 grid(M + tiles, k_in ? 2 : 1), block(256);
+  const int wide = (nh > nkv ? nh : nkv) * hin;
+  const uintptr_t al = (uintptr_t)q_out | (uintptr_t)q_in | (uintptr_t)k_in | (uintptr_t)k_pool | (uintptr_t)q_norm_w | (uintptr_t)k_norm_w;
+  const bool fast = dtype == LEB_BF16 && (!neox || rope_dim == 0) && hin == hd && hd % 8 == 0 && wide <= 8 * 256 * 4 &&
+                    (al & 15) == 0 && q_stride % 8 == 0 && kv_stride % 8 == 0;
+#define LEB_QRN_ARGS(T)                                                                                                    \
+  (T*)q_out, (const T*)q_in, q_stride, (const T*)k_in, (const T*)v_in, kv_stride, (T*)k_pool, (T*)v_pool, block_table,     \
+      bt_width, row_seq, row_pos, seq_slot, q_norm_w, k_norm_w, eps, inv_freq, rope_dim, neox, M, nh, nkv, hd, page_size, vd, hin, vin
+  if (fast) {
+    const size_t smem = (size_t)rope_dim * sizeof(float);
+    if (wide <= 8 * 256) leb_launch(qk_row_norm_rope_store_kernel<bf16, bf16, true, 1>, grid, block, smem, st, LEB_QRN_ARGS(bf16));
+    else if (wide <= 8 * 256 * 2) leb_launch(qk_row_norm_rope_store_kernel<bf16, bf16, true, 2>, grid, block, smem, st, LEB_QRN_ARGS(bf16));
+    else leb_launch(qk_row_norm_rope_store_kernel<bf16, bf16, true, 4>, grid, block, smem, st, LEB_QRN_ARGS(bf16));
+  } else {
+    const size_t smem = (size_t)(rope_dim + wide) * sizeof(float);
+    LEB_REQUIRE(smem <= 200 * 1024, "leb_qk_row_norm_rope_store: a row of %d numbers does not fit shared memory", wide);
+    static bool set = false;
+    if (smem > 40 * 1024 && !set) {
+      cudaFuncSetAttribute(qk_row_norm_rope_store_kernel<float, float, false, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+      cudaFuncSetAttribute(qk_row_norm_rope_store_kernel<bf16, bf16, false, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+      set = true;
+    }
+    if (dtype == LEB_F32)
+      leb_launch(qk_row_norm_rope_store_kernel<float, float, false, 1>, grid, block, smem, st, LEB_QRN_ARGS(float));
+    else
+      leb_launch(qk_row_norm_rope_store_kernel<bf16, bf16, false, 1>, grid, block, smem, st, LEB_QRN_ARGS(bf16));
+  }
+#undef LEB_QRN_ARGS
+  LEB_CHECK_LAUNCH("leb_qk_row_norm_rope_store");
+  return 0;
 }
 
 LEB_API int leb_qk_rope_store(void* q_out, const void* q_in, int q_stride, const void* k_in,

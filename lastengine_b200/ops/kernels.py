@@ -99,14 +99,15 @@ def _declare(L) -> None:
         "leb_add": [P, P, S, P],
         "leb_shortconv": [P, P, I, P, P, P, P, P, P, P, I, I, I, I, P],
         "leb_qk_rope_store": [P, P, I, P, P, I, P, P, I, P, I, P, P, P, P, P, F, P, I, I, I, I, I, I, I, I, I, I, I, P],
-        "leb_attention": [P, P, P, P, P, I, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, I, P],
+        "leb_attention": [P, P, P, P, P, I, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, I, I, P],
         "leb_gated_act": [P, I, P, I, I, I, I, F, F, P],
         "leb_layernorm": [P, I, P, P, P, I, I, F, P],
         "leb_scaled_residual": [P, P, F, P, I, P, F, I, I, P],
-        "leb_latent_prep": [P, P, I, I, P, P, I, P, P, P, P, P, F, P, I, I, I, I, I, I, P],
-        "leb_latent_q_split": [P, P, P, I, P, P, I, I, I, I, I, I, P],
+        "leb_latent_prep": [P, P, I, I, P, P, I, P, P, P, P, P, F, P, I, I, I, I, I, I, I, P],
+        "leb_latent_q_split": [P, P, P, I, P, P, I, I, I, I, I, I, I, P],
+        "leb_latent_rows": [P, P, P, I, I, P, P, I, P, P, P, P, F, P, I, I, I, I, I, I, I, I, I, P],
         "leb_heads_to_rows": [P, P, I, I, I, I, P],
-        "leb_latent_attention": [P, I, P, P, P, P, I, P, I, P, P, P, P, P, I, I, I, I, I, I, F, I, I, P],
+        "leb_latent_attention": [P, I, P, P, P, P, I, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, P],
         "leb_latent_attention_mma_supported": [I, I, I],
         "leb_gemm_bf16_any": [P, I, P, P, I, I, I, I, I, I, P, I, S, P],
         "leb_gated_residual": [P, P, P, I, I, P, P, I, P, F, I, I, P],
@@ -133,16 +134,16 @@ def _declare(L) -> None:
         "leb_penalties_slots": [P, P, P, P, I, I, I, F, F, P],
         "leb_history_append": [P, P, P, P, I, I, P],
         "leb_attention_decode_supported": [I, I, I, I],
-        "leb_attention_decode": [P, P, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, P],
-        "leb_attention_merge": [P, P, I, P, I, I, I, I, I, P],
+        "leb_attention_decode": [P, P, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P],
+        "leb_attention_merge": [P, P, I, P, I, I, I, I, I, I, P],
         "leb_attention_decode_prep_supported": [I, I, I, I, I, I],
-        "leb_attention_decode_prep": [P, P, P, I, P, P, I, P, P, P, I, P, P, P, P, P, F, P, I, I, P, I, I, I, I, I, I, I, F, I, P],
+        "leb_attention_decode_prep": [P, P, P, I, P, P, I, P, P, P, I, P, P, P, P, P, F, P, I, I, I, P, I, I, I, I, I, I, I, I, I, I, F, I, P],
         "leb_attention_prefill_supported": [I, I, I, I],
         "leb_attention_prefill_tc_supported": [I, I, I, I],
-        "leb_attention_prefill_tc": [P, P, I, I, P, P, I, P, I, P, P, P, P, P, I, I, I, I, I, I, I, F, I, P, P],
+        "leb_attention_prefill_tc": [P, P, I, I, P, P, I, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, P],
         "leb_attention_pooled_tc": [P, P, I, I, P, P, I, P, I, P, P, I, P, I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P, P],
         "leb_attention_pooled_tc_value_dim": [I],
-        "leb_attention_prefill": [P, P, P, P, P, I, P, P, P, P, P, I, I, I, I, I, I, I, F, I, P],
+        "leb_attention_prefill": [P, P, P, P, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P],
         "leb_gemm_bf16_skinny_slices": [I, I],
         "leb_gemm_bf16_skinny_supported": [P, P, I, I, I],
         "leb_gemm_bf16_skinny": [P, I, P, P, I, I, I, I, I, I, P, I, P, I, I, F, P, P, P, P, P],
@@ -168,6 +169,9 @@ def _declare(L) -> None:
         "leb_postnorm_residual": [P, P, F, P, P, F, P, I, I, I, P],
         "leb_layernorm_bias": [P, I, P, P, P, P, I, I, F, P],
         "leb_embed_positions": [P, P, I, P, I, P, P, P, I, I, I, I, F, P],
+        "leb_qk_row_norm_rope_store": [P, P, I, P, P, I, P, P, I, P, I, P, P, P, P, P, F, P, I, I, I, I, I, I, I, I, I, I, P],
+        "leb_outnorm_residual": [P, P, P, F, P, I, I, I, P],
+        "leb_softcap": [P, F, F, S, P],
         "leb_cast_rows": [P, I, P, S, P],
         "leb_pooled_attn_prep": [P, P, P, I, P, I, P, P, P, F, P, I, P, P, I, P, P, P, I, I, I, I, I, I, P],
         "leb_pool_blocks": [P, P, P, P, I, P, I, P, I, P, P, P, I, I, I, I, I, I, I, P],
@@ -329,6 +333,27 @@ def postnorm_residual(x: torch.Tensor, y: torch.Tensor, alpha: float, w: torch.T
         assert h.shape == (M, D)
     _check(lib().leb_postnorm_residual(_ptr(x), _ptr(y), float(alpha), _ptr(w), _ptr(bias), float(eps), _ptr(h),
                                        _dt(h, "postnorm_residual.h") if h is not None else F32, M, D, _stream()))
+
+
+def outnorm_residual(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, eps: float, h: torch.Tensor | None = None) -> None:
+    """x += y / sqrt(mean(y^2) + eps) * w per row (x, y float [M, D]); with `h` [M, D] the launch also leaves the
+    new rows there in h's type (the input of the sublayer that reads the stream next)."""
+    _cuda(x, "outnorm_residual.x", torch.float32)
+    _cuda(y, "outnorm_residual.y", torch.float32)
+    _cuda(w, "outnorm_residual.w", torch.float32)
+    M, D = x.shape
+    assert y.shape == (M, D) and w.numel() == D
+    if h is not None:
+        _cuda(h, "outnorm_residual.h")
+        assert h.shape == (M, D)
+    _check(lib().leb_outnorm_residual(_ptr(x), _ptr(y), _ptr(w), float(eps), _ptr(h),
+                                      _dt(h, "outnorm_residual.h") if h is not None else F32, M, D, _stream()))
+
+
+def softcap(z: torch.Tensor, scale: float, cap: float) -> None:
+    """z <- cap tanh(scale z / cap) in place (float; cap 0: z <- scale z)."""
+    _cuda(z, "softcap.z", torch.float32)
+    _check(lib().leb_softcap(_ptr(z), float(scale), float(cap), z.numel(), _stream()))
 
 
 def embed_positions(x: torch.Tensor, h: torch.Tensor | None, table: torch.Tensor, tokens: torch.Tensor,
@@ -1034,16 +1059,54 @@ def qk_rope_store(q_out: torch.Tensor, q_in: torch.Tensor, k_in: torch.Tensor | 
         _stream()))
 
 
+def qk_row_norm_rope_store(q_out: torch.Tensor, q_in: torch.Tensor, k_in: torch.Tensor | None, v_in: torch.Tensor | None,
+                           k_pool: torch.Tensor | None, v_pool: torch.Tensor | None, block_table: torch.Tensor, batch,
+                           q_norm_w: torch.Tensor, k_norm_w: torch.Tensor | None, eps: float,
+                           inv_freq: torch.Tensor | None, rope_dim: int, neox: bool, nh: int, nkv: int, hd: int,
+                           page_size: int, vd: int | None = None, hd_in: int | None = None, vd_in: int | None = None) -> None:
+    """`qk_rope_store` where q and k are divided by the root mean square of their whole projected row, before heads
+    are cut out of it, and multiplied by weights over the row (q_norm_w [nh * hd_in], k_norm_w [nkv * hd_in])."""
+    vd = hd if vd is None else int(vd)
+    hd_in = hd if hd_in is None else int(hd_in)
+    vd_in = vd if vd_in is None else int(vd_in)
+    _cuda(q_out, "qk_row_norm_rope_store.q_out")
+    _cuda(q_in, "qk_row_norm_rope_store.q_in", q_out.dtype, contiguous=False)
+    _cuda(q_norm_w, "qk_row_norm_rope_store.q_norm_w", torch.float32)
+    M = q_out.shape[0]
+    assert q_out.shape[1] == nh * hd and q_in.shape == (M, nh * hd_in) and q_in.stride(-1) == 1 and q_norm_w.numel() == nh * hd_in
+    kv_stride = 0
+    if k_in is not None:
+        _cuda(k_in, "qk_row_norm_rope_store.k_in", q_out.dtype, contiguous=False)
+        _cuda(v_in, "qk_row_norm_rope_store.v_in", q_out.dtype, contiguous=False)
+        _cuda(k_norm_w, "qk_row_norm_rope_store.k_norm_w", torch.float32)
+        assert k_in.shape == (M, nkv * hd_in) and v_in.shape == (M, nkv * vd_in) and k_norm_w.numel() == nkv * hd_in
+        assert k_in.stride(0) == v_in.stride(0) and k_in.stride(-1) == 1 and v_in.stride(-1) == 1
+        kv_stride = k_in.stride(0)
+        _cuda(k_pool, "qk_row_norm_rope_store.k_pool", q_out.dtype)
+        _cuda(v_pool, "qk_row_norm_rope_store.v_pool", q_out.dtype)
+        assert k_pool.shape[1:] == (nkv, page_size, hd) and v_pool.shape[1:] == (nkv, vd, page_size)
+    _cuda(block_table, "qk_row_norm_rope_store.block_table", torch.int32)
+    if inv_freq is not None:
+        _cuda(inv_freq, "qk_row_norm_rope_store.inv_freq", torch.float32)
+        assert inv_freq.numel() == rope_dim // 2
+    _check(lib().leb_qk_row_norm_rope_store(
+        _ptr(q_out), _ptr(q_in), q_in.stride(0), _ptr(k_in), _ptr(v_in), kv_stride, _ptr(k_pool), _ptr(v_pool),
+        _dt(q_out, "qk_row_norm_rope_store"), _ptr(block_table), block_table.shape[1], _ptr(batch.row_seq),
+        _ptr(batch.row_pos), _ptr(batch.seq_slot), _ptr(q_norm_w), _ptr(k_norm_w), float(eps), _ptr(inv_freq),
+        rope_dim if inv_freq is not None else 0, int(neox), M, nh, nkv, hd, page_size, vd, hd_in, vd_in, _stream()))
+
+
 _sm_counts: dict[int, int] = {}
 
 
 def latent_prep(cq: torch.Tensor, proj: torch.Tensor, pool: torch.Tensor | None, block_table, batch,
                 q_norm_w: torch.Tensor, kv_norm_w: torch.Tensor | None, eps: float, inv_freq: torch.Tensor | None,
-                rot_dims: int, rank: int, rot: int, page_size: int) -> None:
+                rot_dims: int, rank: int, rot: int, page_size: int, neox: bool = False) -> None:
     """The rows of a step of a latent-attention layer after the down projections: proj [M, q_rank
     (+ rank + rot)] -> cq [M, q_rank] = rmsnorm(proj[:, :q_rank]) * q_norm_w, and with `pool`
     [page, page_size, rank + rot] the cache row [rmsnorm(latent) * kv_norm_w | rotated key part] at every
-    row's position (pairs (2i, 2i+1) of the first rot_dims dimensions turned by pos * inv_freq[i])."""
+    row's position (pairs (2i, 2i+1), or with `neox` (i, i + rot_dims/2), of the first rot_dims dimensions
+    turned by pos * inv_freq[i])."""
     _cuda(cq, "latent_prep.cq")
     _cuda(proj, "latent_prep.proj", cq.dtype, contiguous=False)
     _cuda(q_norm_w, "latent_prep.q_norm_w", torch.float32)
@@ -1060,12 +1123,12 @@ def latent_prep(cq: torch.Tensor, proj: torch.Tensor, pool: torch.Tensor | None,
     _check(lib().leb_latent_prep(_ptr(cq), _ptr(proj), proj.stride(0), _dt(cq, "latent_prep.cq"), _ptr(pool),
                                  _ptr(block_table), block_table.shape[1] if block_table is not None else 0,
                                  _ptr(batch.row_seq), _ptr(batch.row_pos), _ptr(batch.seq_slot), _ptr(q_norm_w),
-                                 _ptr(kv_norm_w), float(eps), _ptr(inv_freq) if rot_dims else None, int(rot_dims), M, q_rank,
+                                 _ptr(kv_norm_w), float(eps), _ptr(inv_freq) if rot_dims else None, int(rot_dims), int(neox), M, q_rank,
                                  int(rank), int(rot), int(page_size), _stream()))
 
 
 def latent_q_split(qn: torch.Tensor, qr: torch.Tensor, q: torch.Tensor, row_pos: torch.Tensor,
-                   inv_freq: torch.Tensor | None, rot_dims: int, H: int, dim: int, rot: int) -> None:
+                   inv_freq: torch.Tensor | None, rot_dims: int, H: int, dim: int, rot: int, neox: bool = False) -> None:
     """q [M, H * (dim + rot)] -> qn [H, M, dim_p] (each head's first `dim` numbers, head-major, zeros
     behind them) and qr [M, H, rot] (each head's last `rot` numbers, rotated by the row's position)."""
     _cuda(q, "latent_q_split.q")
@@ -1075,7 +1138,34 @@ def latent_q_split(qn: torch.Tensor, qr: torch.Tensor, q: torch.Tensor, row_pos:
     dim_p = qn.shape[2]
     assert q.shape[1] == H * (dim + rot) and qn.shape[:2] == (H, M) and dim_p >= dim and qr.numel() == M * H * rot
     _check(lib().leb_latent_q_split(_ptr(qn), _ptr(qr), _ptr(q), _dt(q, "latent_q_split.q"), _ptr(row_pos),
-                                    _ptr(inv_freq) if rot_dims else None, int(rot_dims), M, H, dim, dim_p, rot, _stream()))
+                                    _ptr(inv_freq) if rot_dims else None, int(rot_dims), int(neox), M, H, dim, dim_p, rot, _stream()))
+
+
+def latent_rows(qn: torch.Tensor, qr: torch.Tensor, proj: torch.Tensor, pool: torch.Tensor | None, block_table, batch,
+                kv_norm_w: torch.Tensor | None, eps: float, inv_freq: torch.Tensor | None, rot_dims: int, neox: bool,
+                H: int, dim: int, rank: int, rot: int, page_size: int) -> None:
+    """`latent_q_split` and the cache row of `latent_prep` in one launch, for layers whose q comes straight from the
+    row's projection: proj [M, H * (dim + rot) (+ rank + rot)] -> qn [H, M, dim_p], qr [M, H, rot] and, with `pool`,
+    the cache row at every row's position."""
+    _cuda(proj, "latent_rows.proj")
+    _cuda(qn, "latent_rows.qn", proj.dtype)
+    _cuda(qr, "latent_rows.qr", proj.dtype)
+    M = proj.shape[0]
+    dim_p = qn.shape[2]
+    assert qn.shape[:2] == (H, M) and dim_p >= dim and qr.numel() == M * H * rot
+    assert proj.shape[1] == H * (dim + rot) + (rank + rot if pool is not None else 0)
+    if pool is not None:
+        _cuda(pool, "latent_rows.pool", proj.dtype)
+        _cuda(kv_norm_w, "latent_rows.kv_norm_w", torch.float32)
+        assert kv_norm_w.numel() == rank and pool.shape[-1] == rank + rot and pool.shape[-2] == page_size
+    if rot_dims:
+        _cuda(inv_freq, "latent_rows.inv_freq", torch.float32)
+        assert inv_freq.numel() == rot_dims // 2
+    _check(lib().leb_latent_rows(_ptr(qn), _ptr(qr), _ptr(proj), proj.stride(0), _dt(proj, "latent_rows.proj"), _ptr(pool),
+                                 _ptr(block_table), block_table.shape[1] if block_table is not None else 0,
+                                 _ptr(batch.row_seq), _ptr(batch.row_pos), _ptr(batch.seq_slot), _ptr(kv_norm_w), float(eps),
+                                 _ptr(inv_freq) if rot_dims else None, int(rot_dims), int(neox), M, H, dim, dim_p, int(rank),
+                                 int(rot), int(page_size), _stream()))
 
 
 def heads_to_rows(out: torch.Tensor, src: torch.Tensor) -> None:
@@ -1103,7 +1193,17 @@ def set_latent_mma(on: bool) -> None:
     lib().leb_set_latent_mma(1 if on else 0)
 
 
-def latent_attention_splits(batch, H: int, mma: bool = False, rank: int = 0) -> int:
+def _read_length(max_kvlen: int, window: int = 0, chunk: int = 0) -> int:
+    """The most cached positions a row reads: its sequence, its window or its chunk."""
+    n = max_kvlen
+    if window > 0:
+        n = min(n, window)
+    if chunk > 0:
+        n = min(n, chunk)
+    return n
+
+
+def latent_attention_splits(batch, H: int, mma: bool = False, rank: int = 0, window: int = 0, chunk: int = 0) -> int:
     """Pieces the key range of a decode step is cut into so that the blocks fill the SMs (1 for prompts).
     The tensor-core kernel takes up to 64 heads in a block that is alone on its SM, the general one 8 in
     blocks of which an SM holds several; a piece is at least 128 cached rows (measured at 2,048 positions:
@@ -1112,13 +1212,15 @@ def latent_attention_splits(batch, H: int, mma: bool = False, rank: int = 0) -> 
         return 1
     blocks = batch.n_seqs * -(-H // (64 if mma else 8))
     want = max(1, ((1 if mma else 2) * sm_count()) // max(1, blocks))
-    return int(max(1, min(want, batch.max_kvlen // 128, 64)))
+    return int(max(1, min(want, _read_length(batch.max_kvlen, window, chunk) // 128, 64)))
 
 
 def latent_attention(out: torch.Tensor, qt: torch.Tensor, qr: torch.Tensor, pool: torch.Tensor, block_table, batch,
                      sink: torch.Tensor | None, rank: int, rot: int, page_size: int, scale: float,
-                     n_splits: int = 1, scratch: torch.Tensor | None = None) -> None:
-    """Causal attention of every row over its sequence's cached rows [c | k^r] (pool [page, page_size,
+                     n_splits: int = 1, scratch: torch.Tensor | None = None, window: int = 0, chunk: int = 0,
+                     wide: bool = False) -> None:
+    """Causal attention of every row (over the last `window` positions, or within chunks of `chunk`, where given;
+    `wide`: softmax weights of 16 significant bits in the bfloat16 product) over its sequence's cached rows [c | k^r] (pool [page, page_size,
     rank + rot]): query vectors qt [H, M, rank] and qr [M, H, rot]; scores scale * ([qt | qr] . [c | k^r]);
     softmax with `sink` [H] as one more logit without a value; out [H, M, >= rank] = sum p c."""
     _cuda(out, "latent_attention.out")
@@ -1136,7 +1238,8 @@ def latent_attention(out: torch.Tensor, qt: torch.Tensor, qr: torch.Tensor, pool
     _check(lib().leb_latent_attention(_ptr(out), ld, _ptr(scratch), _ptr(qt), _ptr(qr), _ptr(pool), _dt(out, "latent_attention.out"),
                                       _ptr(block_table), block_table.shape[1], _ptr(batch.seq_slot), _ptr(batch.seq_pos0),
                                       _ptr(batch.seq_qstart), _ptr(batch.seq_qlen), _ptr(sink), M, batch.n_seqs, H, int(rank),
-                                      int(rot), int(page_size), float(scale), batch.max_qlen, int(n_splits), _stream()))
+                                      int(rot), int(page_size), int(window), int(chunk), int(wide), float(scale), batch.max_qlen,
+                                      int(n_splits), _stream()))
 
 
 def sm_count() -> int:
@@ -1148,7 +1251,7 @@ def sm_count() -> int:
     return n
 
 
-def attention_splits(batch, nkv: int, G: int, sm_count: int | None = None, hd: int = 64) -> int:
+def attention_splits(batch, nkv: int, G: int, sm_count: int | None = None, hd: int = 64, chunk: int = 0) -> int:
     """How many blocks share one sequence's key range in a decode step (1 for prompts).
 
     Measured on B200 (head size 64, 8 kv heads, times with the merge of the splits): a block has a
@@ -1164,7 +1267,7 @@ def attention_splits(batch, nkv: int, G: int, sm_count: int | None = None, hd: i
         return 1
     if sm_count is None:
         sm_count = globals()["sm_count"]()
-    kv = max(int(batch.max_kvlen), 1)
+    kv = max(_read_length(int(batch.max_kvlen), 0, chunk), 1)
     per = max(batch.n_seqs * nkv * ((G + 15) // 16), 1)
     stage_bytes = 2 * 32 * hd * 2 * (3 if hd <= 32 else 2) * 4          # a block's rings: 4 warps, keys and values
     slots = sm_count * max(1, min(3, (227 * 1024) // stage_bytes))      # blocks that run at once
@@ -1181,7 +1284,9 @@ class RawQKV:
     """A decode step's q, k and v as the projection left them, for the decode attention kernel that
     norms, rotates and stores them itself (`decode_attention_takes_raw` says when it can)."""
 
-    def __init__(self, q_in, k_in, v_in, q_norm_w, k_norm_w, eps, inv_freq, rope_dim, neox):
+    def __init__(self, q_in, k_in, v_in, q_norm_w, k_norm_w, eps, inv_freq, rope_dim, neox, row_norm: bool = False):
+        """`row_norm`: q and k are normed over their whole row, with weights over the row."""
+        self.row_norm = bool(row_norm)
         self.q_in, self.k_in, self.v_in = q_in, k_in, v_in
         self.q_norm_w, self.k_norm_w, self.eps = q_norm_w, k_norm_w, float(eps)
         self.inv_freq, self.rope_dim, self.neox = inv_freq, int(rope_dim), bool(neox)
@@ -1191,26 +1296,38 @@ def decode_attention_takes_raw(dtype: torch.dtype, batch, M: int, nh: int, nkv: 
                                inv_freq, rope_dim: int, neox: bool) -> bool:
     """Whether `attention(..., raw=...)` will do the per-head norm, the rotation and the cache write
     of this step itself: a bfloat16 decode step (one row per sequence) whose sizes the tensor-core
-    decode kernel takes, with a split-half rotation over the whole head."""
+    decode kernel takes, with a rotation over the whole head."""
     return bool(dtype == torch.bfloat16 and batch.max_qlen == 1 and M == batch.n_seqs and inv_freq is not None
                 and lib().leb_attention_decode_prep_supported(nh, nkv, hd, page_size, int(rope_dim), 1 if neox else 0))
+
+
+def _gate_layout(gate: torch.Tensor | None, M: int, nh: int, width: int, dtype: torch.dtype) -> tuple[int, int]:
+    """(row stride, one factor per number of a head?) of an attention gate: [M, nh] or [M, nh * width]."""
+    if gate is None:
+        return 0, 0
+    _cuda(gate, "attention.gate", dtype, contiguous=False)
+    assert gate.shape in ((M, nh), (M, nh * width)) and gate.stride(-1) == 1
+    return gate.stride(0), int(gate.shape[1] != nh)
 
 
 def attention(out: torch.Tensor, q: torch.Tensor | None, k_pool: torch.Tensor, v_pool: torch.Tensor,
               block_table: torch.Tensor, batch, nh: int, nkv: int, hd: int, page_size: int,
               window: int, scale: float, gate: torch.Tensor | None = None,
               n_splits: int = 1, scratch: torch.Tensor | None = None, raw: RawQKV | None = None,
-              vd: int | None = None) -> None:
+              vd: int | None = None, chunk: int = 0, wide: bool = False) -> None:
     """Causal attention of the step's rows over the paged cache (which already holds their keys;
     with `raw`, the kernel puts the step's keys and values there itself and `q` is not used).
-    `vd`: width of a value head where it differs from the key head's (the general kernel then)."""
+    `vd`: width of a value head where it differs from the key head's (the general kernel then).
+    `gate`: [rows, heads], a factor sigmoid(gate) per head, or [rows, heads * value width], one per number.
+    `chunk` > 0: a row reads its own chunk of that many positions only, counted from the sequence's first.
+    `wide`: the softmax weights enter the bfloat16 product with the values as two terms (16 significant bits)."""
     _cuda(out, "attention.out")
     if vd is not None and vd != hd:
         return _attention_general(out, q, k_pool, v_pool, block_table, batch, nh, nkv, hd, int(vd), page_size, window,
-                                  scale, gate, n_splits, scratch)
+                                  scale, gate, n_splits, scratch, chunk)
     if raw is not None:
         return _attention_decode_raw(out, raw, k_pool, v_pool, block_table, batch, nh, nkv, hd, page_size, window,
-                                     scale, gate, n_splits, scratch)
+                                     scale, gate, n_splits, scratch, chunk, wide)
     _cuda(q, "attention.q", out.dtype)
     _cuda(k_pool, "attention.k_pool", out.dtype)
     _cuda(v_pool, "attention.v_pool", out.dtype)
@@ -1218,11 +1335,7 @@ def attention(out: torch.Tensor, q: torch.Tensor | None, k_pool: torch.Tensor, v
     M = out.shape[0]
     assert out.shape == (M, nh * hd) and q.shape == (M, nh * hd)
     assert k_pool.shape[1:] == (nkv, page_size, hd) and v_pool.shape[1:] == (nkv, hd, page_size)
-    gate_stride = 0
-    if gate is not None:
-        _cuda(gate, "attention.gate", out.dtype, contiguous=False)
-        assert gate.shape == (M, nh) and gate.stride(-1) == 1
-        gate_stride = gate.stride(0)
+    gate_stride, gate_elem = _gate_layout(gate, M, nh, hd, out.dtype)
     if n_splits > 1:
         need = M * nh * n_splits * (hd + 2)
         if scratch is None or scratch.numel() < need or scratch.dtype != torch.float32:
@@ -1235,10 +1348,10 @@ def attention(out: torch.Tensor, q: torch.Tensor | None, k_pool: torch.Tensor, v
         _check(L.leb_attention_decode(
             _ptr(out), _ptr(scratch), _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(block_table),
             block_table.shape[1], _ptr(batch.seq_slot), _ptr(batch.seq_pos0), _ptr(batch.seq_qstart),
-            _ptr(gate), gate_stride, batch.n_seqs, nh, nkv, hd, page_size, window, float(scale), n_splits,
-            _stream()))
+            _ptr(gate), gate_stride, gate_elem, batch.n_seqs, nh, nkv, hd, page_size, window, chunk, int(wide), float(scale),
+            n_splits, _stream()))
         if n_splits > 1:
-            _check(L.leb_attention_merge(_ptr(out), _ptr(scratch), BF16, _ptr(gate), gate_stride, M, nh, hd,
+            _check(L.leb_attention_merge(_ptr(out), _ptr(scratch), BF16, _ptr(gate), gate_stride, gate_elem, M, nh, hd,
                                          n_splits, _stream()))
         return
     if (out.dtype == torch.bfloat16 and n_splits == 1 and batch.max_qlen >= TC_ATTENTION_MIN_ROWS
@@ -1247,8 +1360,8 @@ def attention(out: torch.Tensor, q: torch.Tensor | None, k_pool: torch.Tensor, v
         _check(L.leb_attention_prefill_tc(
             _ptr(out), _ptr(q), q.stride(0), M, _ptr(k_pool), _ptr(v_pool), k_pool.shape[0], _ptr(block_table),
             block_table.shape[1], _ptr(batch.seq_slot), _ptr(batch.seq_pos0), _ptr(batch.seq_qstart),
-            _ptr(batch.seq_qlen), _ptr(gate), gate_stride, batch.n_seqs, nh, nkv, hd, page_size, window, float(scale),
-            batch.max_qlen, _ptr(_status_word(out.device)), _stream()))
+            _ptr(batch.seq_qlen), _ptr(gate), gate_stride, gate_elem, batch.n_seqs, nh, nkv, hd, page_size, window, chunk,
+            int(wide), float(scale), batch.max_qlen, _ptr(_status_word(out.device)), _stream()))
         return
     if (out.dtype == torch.bfloat16 and n_splits == 1
             and L.leb_attention_prefill_supported(nh, nkv, hd, page_size)):
@@ -1256,18 +1369,18 @@ def attention(out: torch.Tensor, q: torch.Tensor | None, k_pool: torch.Tensor, v
         _check(L.leb_attention_prefill(
             _ptr(out), _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(block_table), block_table.shape[1],
             _ptr(batch.seq_slot), _ptr(batch.seq_pos0), _ptr(batch.seq_qstart), _ptr(batch.seq_qlen),
-            _ptr(gate), gate_stride, batch.n_seqs, nh, nkv, hd, page_size, window, float(scale),
+            _ptr(gate), gate_stride, gate_elem, batch.n_seqs, nh, nkv, hd, page_size, window, chunk, int(wide), float(scale),
             batch.max_qlen, _stream()))
         return
     _check(L.leb_attention(
         _ptr(out), _ptr(scratch), _ptr(q), _ptr(k_pool), _ptr(v_pool), _dt(out, "attention"),
         _ptr(block_table), block_table.shape[1], _ptr(batch.seq_slot), _ptr(batch.seq_pos0),
-        _ptr(batch.seq_qstart), _ptr(batch.seq_qlen), _ptr(gate), gate_stride, M, batch.n_seqs, nh, nkv,
-        hd, page_size, window, float(scale), batch.max_qlen, n_splits, hd, _stream()))
+        _ptr(batch.seq_qstart), _ptr(batch.seq_qlen), _ptr(gate), gate_stride, gate_elem, M, batch.n_seqs, nh, nkv,
+        hd, page_size, window, chunk, float(scale), batch.max_qlen, n_splits, hd, _stream()))
 
 
 def _attention_general(out, q, k_pool, v_pool, block_table, batch, nh, nkv, hd, vd, page_size, window, scale, gate,
-                       n_splits, scratch) -> None:
+                       n_splits, scratch, chunk=0) -> None:
     """The general kernel with value heads of their own width."""
     _cuda(q, "attention.q", out.dtype)
     _cuda(k_pool, "attention.k_pool", out.dtype)
@@ -1276,11 +1389,7 @@ def _attention_general(out, q, k_pool, v_pool, block_table, batch, nh, nkv, hd, 
     M = out.shape[0]
     assert out.shape == (M, nh * vd) and q.shape == (M, nh * hd)
     assert k_pool.shape[1:] == (nkv, page_size, hd) and v_pool.shape[1:] == (nkv, vd, page_size)
-    gate_stride = 0
-    if gate is not None:
-        _cuda(gate, "attention.gate", out.dtype, contiguous=False)
-        assert gate.shape == (M, nh) and gate.stride(-1) == 1
-        gate_stride = gate.stride(0)
+    gate_stride, gate_elem = _gate_layout(gate, M, nh, vd, out.dtype)
     if n_splits > 1:
         need = M * nh * n_splits * (vd + 2)
         if scratch is None or scratch.numel() < need or scratch.dtype != torch.float32:
@@ -1288,12 +1397,12 @@ def _attention_general(out, q, k_pool, v_pool, block_table, batch, nh, nkv, hd, 
     _check(lib().leb_attention(
         _ptr(out), _ptr(scratch), _ptr(q), _ptr(k_pool), _ptr(v_pool), _dt(out, "attention"),
         _ptr(block_table), block_table.shape[1], _ptr(batch.seq_slot), _ptr(batch.seq_pos0),
-        _ptr(batch.seq_qstart), _ptr(batch.seq_qlen), _ptr(gate), gate_stride, M, batch.n_seqs, nh, nkv,
-        hd, page_size, window, float(scale), batch.max_qlen, n_splits, vd, _stream()))
+        _ptr(batch.seq_qstart), _ptr(batch.seq_qlen), _ptr(gate), gate_stride, gate_elem, M, batch.n_seqs, nh, nkv,
+        hd, page_size, window, chunk, float(scale), batch.max_qlen, n_splits, vd, _stream()))
 
 
 def _attention_decode_raw(out, raw: RawQKV, k_pool, v_pool, block_table, batch, nh, nkv, hd, page_size, window,
-                          scale, gate, n_splits, scratch) -> None:
+                          scale, gate, n_splits, scratch, chunk=0, wide=False) -> None:
     M = out.shape[0]
     if not decode_attention_takes_raw(out.dtype, batch, M, nh, nkv, hd, page_size, raw.inv_freq, raw.rope_dim, raw.neox):
         raise KernelError("attention: this step's q, k and v must be normed, rotated and stored before the call")
@@ -1310,15 +1419,12 @@ def _attention_decode_raw(out, raw: RawQKV, k_pool, v_pool, block_table, batch, 
         assert raw.k_in.shape == (M, nkv * hd) and raw.v_in.shape == (M, nkv * hd)
         assert raw.k_in.stride(0) == raw.v_in.stride(0) and raw.k_in.stride(-1) == 1 and raw.v_in.stride(-1) == 1
         kv_stride = raw.k_in.stride(0)
-    for name, t in (("q_norm_w", raw.q_norm_w), ("k_norm_w", raw.k_norm_w), ("inv_freq", raw.inv_freq)):
+    for name, t, heads in (("q_norm_w", raw.q_norm_w, nh), ("k_norm_w", raw.k_norm_w, nkv), ("inv_freq", raw.inv_freq, 0)):
         if t is not None:
             _cuda(t, f"attention.{name}", torch.float32)
+            assert not heads or t.numel() == (heads * hd if raw.row_norm else hd)
     assert raw.inv_freq.numel() == hd // 2
-    gate_stride = 0
-    if gate is not None:
-        _cuda(gate, "attention.gate", out.dtype, contiguous=False)
-        assert gate.shape == (M, nh) and gate.stride(-1) == 1
-        gate_stride = gate.stride(0)
+    gate_stride, gate_elem = _gate_layout(gate, M, nh, hd, out.dtype)
     if n_splits > 1:
         need = M * nh * n_splits * (hd + 2)
         if scratch is None or scratch.numel() < need or scratch.dtype != torch.float32:
@@ -1328,10 +1434,11 @@ def _attention_decode_raw(out, raw: RawQKV, k_pool, v_pool, block_table, batch, 
         _ptr(out), _ptr(scratch), _ptr(raw.q_in), raw.q_in.stride(0), _ptr(raw.k_in), _ptr(raw.v_in), kv_stride,
         _ptr(k_pool), _ptr(v_pool), _ptr(block_table), block_table.shape[1], _ptr(batch.seq_slot), _ptr(batch.seq_pos0),
         _ptr(batch.seq_qstart), _ptr(raw.q_norm_w), _ptr(raw.k_norm_w), raw.eps, _ptr(raw.inv_freq), raw.rope_dim,
-        1 if raw.neox else 0, _ptr(gate), gate_stride, batch.n_seqs, nh, nkv, hd, page_size, window, float(scale),
-        n_splits, _stream()))
+        1 if raw.neox else 0, int(raw.row_norm), _ptr(gate), gate_stride, gate_elem, batch.n_seqs, nh, nkv, hd, page_size, window,
+        chunk, int(wide), float(scale), n_splits, _stream()))
     if n_splits > 1:
-        _check(L.leb_attention_merge(_ptr(out), _ptr(scratch), BF16, _ptr(gate), gate_stride, M, nh, hd, n_splits, _stream()))
+        _check(L.leb_attention_merge(_ptr(out), _ptr(scratch), BF16, _ptr(gate), gate_stride, gate_elem, M, nh, hd, n_splits,
+                                     _stream()))
 
 
 # ----------------------------------------------------------------------------------------------

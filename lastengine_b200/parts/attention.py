@@ -16,6 +16,12 @@ a weight (`qk_norm="unit"`); every value head divided by its root mean square be
 numbers, since a rotation of pairs leaves the head's sum of squares as it was.  `names` renames
 the tensors under the part's prefix.
 
+q and k may also be normed over their whole projected row, before heads are cut out of it, with weights over the row
+(`qk_norm="row"`); the output gate may be a factor per number of every head, sigmoid(Wg h) with Wg [heads * v_head_dim,
+hidden] (`output_gate="numbers"`); instead of a window the positions may be cut into chunks of `chunk`, counted from the
+sequence's first: a row reads its own chunk up to itself.  `wide_weights`: the softmax weights enter the bfloat16
+product with the values as two bfloat16 terms (16 significant bits) instead of one.
+
 Key and value heads of different widths are cached at the wider of the two when that is a size the
 tensor-core attention kernels take: the narrower heads are stored with zeros behind them (a zero
 dimension changes no score and adds nothing to a value; the scale is explicit and the norms run over
@@ -38,10 +44,12 @@ class AttentionMixer(Mixer):
     split_norm = True
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int,
-                 norm_eps: float, qk_norm: bool = True, position: PartSpec | None = None,
-                 window: int = 0, output_gate: bool = False, own_kv: bool = True,
+                 norm_eps: float, qk_norm: bool | str = True, position: PartSpec | None = None,
+                 window: int = 0, output_gate: bool | str = False, own_kv: bool = True,
                  scale: float | None = None, v_head_dim: int | None = None, conv_taps: int = 0,
-                 v_norm: bool = False, names: dict[str, str] | None = None):
+                 v_norm: bool = False, names: dict[str, str] | None = None, chunk: int = 0, wide_weights: bool = False):
+        if qk_norm not in (True, False, "unit", "row") or output_gate not in (True, False, "numbers"):
+            raise ValueError(f"qk_norm {qk_norm!r} (True, False, 'unit', 'row') / output_gate {output_gate!r} (True, False, 'numbers')")
         if num_heads % num_kv_heads != 0:
             raise ValueError(f"{num_heads} heads do not divide into {num_kv_heads} kv heads")
         if head_dim > 256:
@@ -49,6 +57,7 @@ class AttentionMixer(Mixer):
         self.D, self.nh, self.nkv, self.hd = int(hidden_size), int(num_heads), int(num_kv_heads), int(head_dim)
         self.eps = float(norm_eps)
         self.qk_unit = qk_norm == "unit"            # divided by the root mean square, no weight
+        self.qk_row = qk_norm == "row"              # over the whole projected row, weights over the row
         self.qk_norm = bool(qk_norm) and not self.qk_unit
         self.vd = self.hd if v_head_dim is None else int(v_head_dim)
         if self.vd > 256:
@@ -66,8 +75,10 @@ class AttentionMixer(Mixer):
                   "gate": "gate_proj.weight", "q_norm": "q_layernorm.weight", "k_norm": "k_layernorm.weight",
                   "q_conv": "q_conv.weight", "k_conv": "k_conv.weight", "v_conv": "v_conv.weight"}
         self.n.update(names or {})
-        self.window = int(window)
-        self.output_gate = bool(output_gate)
+        self.window, self.chunk, self.wide = int(window), int(chunk), bool(wide_weights)
+        self.output_gate, self.gate_numbers = bool(output_gate), output_gate == "numbers"
+        if self.qk_row and (self.v_norm or not own_kv):
+            raise NotImplementedError("norms over whole rows beside normed values or a layer that reads another's cache")
         self.own_kv = bool(own_kv)
         self.scale = float(scale) if scale is not None else 1.0 / math.sqrt(self.hd)
         pos = position or PartSpec("none")
@@ -83,11 +94,11 @@ class AttentionMixer(Mixer):
             t[n["k"]] = TensorSpec((nkv * hd, D), MATRIX)
             t[n["v"]] = TensorSpec((nkv * vd, D), MATRIX)
         if self.qk_norm:
-            t[n["q_norm"]] = TensorSpec((hd,), NORM)
+            t[n["q_norm"]] = TensorSpec((nh * hd if self.qk_row else hd,), NORM)
             if self.own_kv:
-                t[n["k_norm"]] = TensorSpec((hd,), NORM)
+                t[n["k_norm"]] = TensorSpec((nkv * hd if self.qk_row else hd,), NORM)
         if self.output_gate:
-            t[n["gate"]] = TensorSpec((nh, D), MATRIX)
+            t[n["gate"]] = TensorSpec((nh * vd if self.gate_numbers else nh, D), MATRIX)
         if self.taps:
             t[n["q_conv"]] = TensorSpec((nh * hd, self.taps), VECTOR, std=0.5)
             t[n["k_conv"]] = TensorSpec((nkv * hd, self.taps), VECTOR, std=0.5)
@@ -97,7 +108,7 @@ class AttentionMixer(Mixer):
         return t
 
     def cache_spec(self):
-        kv = KVSpec(self.nkv, self.khd, self.window, None if self.kvd == self.khd else self.kvd)
+        kv = KVSpec(self.nkv, self.khd, self.window, None if self.kvd == self.khd else self.kvd, chunk=self.chunk)
         if self.taps <= 1:       # a single tap looks at the current row only
             return kv
         # the convolution's memory: the last taps-1 projected values of every q, k and v channel
@@ -109,13 +120,11 @@ class AttentionMixer(Mixer):
         if self.own_kv:
             parts += [tensors[n["k"]], tensors[n["v"]]]
         if self.output_gate:
-            parts.append(tensors[n["gate"]])
+            parts.append(self._cached_width(tensors[n["gate"]], 0) if self.gate_numbers else tensors[n["gate"]])
         self.w_in = torch.cat(parts, dim=0).contiguous() if len(parts) > 1 else parts[0].contiguous()
         self.w_out = tensors[n["o"]].contiguous()
-        if self.kvd != self.vd:      # zero columns where the cached value heads are wider than the heads
-            w = torch.zeros((self.D, self.nh, self.kvd), dtype=self.w_out.dtype, device=self.w_out.device)
-            w[:, :, : self.vd] = self.w_out.view(self.D, self.nh, self.vd)
-            self.w_out = w.view(self.D, self.nh * self.kvd).contiguous()
+        self.w_out = self._cached_width(self.w_out, 1)
+        self.n_gate = 0 if not self.output_gate else self.nh * self.kvd if self.gate_numbers else self.nh
         if self.qk_norm:
             self.q_norm_w = tensors[n["q_norm"]].contiguous()
             self.k_norm_w = tensors[n["k_norm"]].contiguous() if self.own_kv else None
@@ -126,6 +135,16 @@ class AttentionMixer(Mixer):
             self.w_conv = torch.cat([tensors[n["q_conv"]], tensors[n["k_conv"]], tensors[n["v_conv"]]],
                                     dim=0).to(torch.float32).contiguous()
         self.position.load({n[len("position."):]: v for n, v in tensors.items() if n.startswith("position.")}, env)
+
+    def _cached_width(self, w: torch.Tensor, dim: int) -> torch.Tensor:
+        """w with zeros along `dim` (heads of v_head_dim) where the cached value heads are wider than the heads."""
+        if self.kvd == self.vd:
+            return w
+        shape = list(w.shape)
+        shape[dim: dim + 1] = [self.nh, self.kvd]
+        out = torch.zeros(shape, dtype=w.dtype, device=w.device)
+        out.narrow(dim + 1, 0, self.vd).copy_(w.unflatten(dim, (self.nh, self.vd)))
+        return out.flatten(dim, dim + 1).contiguous()
 
     def split_reader_weight(self):
         return self.w_in
@@ -165,7 +184,7 @@ class AttentionMixer(Mixer):
             v_in = proj[:, col + nkv * hd: col + nkv * (hd + vd)]
             col += nkv * (hd + vd)
         if self.output_gate:
-            gate = proj[:, col: col + nh]
+            gate = proj[:, col: col + self.n_gate]
         if self.n_extra:
             self.extra_out = proj[:, proj.shape[1] - self.n_extra:]
         if self.taps:
@@ -184,7 +203,13 @@ class AttentionMixer(Mixer):
         if (rotary is not None and plain_v and khd == hd
                 and kernels.decode_attention_takes_raw(env.dtype, batch, M, nh, nkv, hd, cache.page_size, *rotary)):
             # a decode step: the attention kernel norms and rotates q and k and stores k and v itself
-            raw = kernels.RawQKV(q_in, k_in, v_in, self.q_norm_w, self.k_norm_w if writes else None, self.eps, *rotary)
+            raw = kernels.RawQKV(q_in, k_in, v_in, self.q_norm_w, self.k_norm_w if writes else None, self.eps, *rotary,
+                                 row_norm=self.qk_row)
+        elif self.qk_row:
+            if rotary is None or not writes:
+                raise NotImplementedError("norms over whole rows with a position encoding that is no rotation, or another layer's cache")
+            kernels.qk_row_norm_rope_store(q, q_in, k_in, v_in, kp, vp, cache.block_table, batch, self.q_norm_w, self.k_norm_w,
+                                           self.eps, *rotary, nh, nkv, khd, cache.page_size, vd=kvd, hd_in=hd, vd_in=vd)
         elif rotary is not None:
             # per-head norm, rotation and the cache write in one launch
             kernels.qk_rope_store(q, q_in, k_in, v_in, kp, vp, cache.block_table, batch, self.q_norm_w,
@@ -209,12 +234,12 @@ class AttentionMixer(Mixer):
             kernels.qk_rope_store(q, qn, kn, vn, kp, vp, cache.block_table, batch, None, None, self.eps,
                                   None, 0, True, nh, nkv, hd, cache.page_size)
         o = ws.get("attn.o", (M, nh * kvd), env.dtype)
-        n_splits = kernels.attention_splits(batch, nkv, nh // nkv, hd=khd)
+        n_splits = kernels.attention_splits(batch, nkv, nh // nkv, hd=khd, chunk=self.chunk)
         scratch = None
         if n_splits > 1:
             scratch = ws.get("attn.part", (M * nh * n_splits * (max(khd, kvd) + 2),), torch.float32)
         kernels.attention(o, None if raw is not None else q, cache.k, cache.v, cache.block_table, batch, nh, nkv, khd,
                           cache.page_size, self.window, self.scale, gate=gate, n_splits=n_splits, scratch=scratch, raw=raw,
-                          vd=kvd)
+                          vd=kvd, chunk=self.chunk, wide=self.wide)
         kernels.linear(out, o, self.w_out, kernels.ACCUMULATE if accumulate else kernels.STORE,
                        emit=emit if accumulate else None)

@@ -69,7 +69,8 @@ class TensorSpec:
 
 @dataclass(frozen=True)
 class KVSpec:
-    """Keys and values that grow with the sequence; `window` > 0 keeps only the last ones.
+    """Keys and values that grow with the sequence; `window` > 0 keeps only the last ones, `chunk` > 0 only those
+    of the chunk of that many positions (counted from the sequence's first) the next position lies in.
     `v_head_dim`: width of a value head where it differs from a key head's (None: the same).
     `pool` > 0: beside them one pooled key and value row for every complete block of `pool` positions,
     in pages of their own (block b in row b); they stay when the window has let the block's positions go."""
@@ -78,6 +79,7 @@ class KVSpec:
     window: int = 0
     v_head_dim: int | None = None
     pool: int = 0
+    chunk: int = 0
 
     @property
     def value_dim(self) -> int:
@@ -88,13 +90,15 @@ class KVSpec:
 class LatentSpec:
     """One row per position that stands for every head's key and value: a latent vector of `rank`
     numbers followed by `rope_dim` numbers of a rotated key part shared by all heads.  Paged like keys
-    and values (one pool of rows `[position][rank + rope_dim]`, nothing stored apart for the values)."""
+    and values (one pool of rows `[position][rank + rope_dim]`, nothing stored apart for the values); `window`
+    and `chunk` as there."""
     rank: int
     rope_dim: int
+    window: int = 0
+    chunk: int = 0
 
     # how the cache's page groups see it: one "head" whose key row is the whole cached row
     n_kv_heads = 1
-    window = 0
     value_dim = 0
 
     @property

@@ -3,6 +3,9 @@
 parallel_residual (further down): x += mult * (Mixer(norm(x)) + FeedForward(norm(x))), with one norm for both
 sublayers or one each.
 
+post_norm_residual and output_norm_residual (at the end): the sublayers read the stream itself, and the norm comes
+after each sum, or on each sublayer's result before its sum.
+
 pre_norm_residual (src/dense.rs:178-194):
     x += [post_norm](Mixer(norm(x)));  x += [post_norm](FeedForward(norm(x)))
 The norms after the mixer and after the feed-forward are the reference's own lfm3 layout and
@@ -302,6 +305,10 @@ class PostNormResidualBlock:
         self.mixer, self.ffn, self.mixer_norm, self.ffn_norm = mixer, ffn, mixer_norm, ffn_norm
         self.alpha = float(alpha)
 
+    def _sum(self, x, y, norm, h) -> None:
+        """A sublayer's float result y goes into the stream x; h (or None) takes the new stream in its own type."""
+        kernels.postnorm_residual(x, y, self.alpha, norm.weight, norm.bias, norm.eps, h=h)
+
     def parts(self) -> dict[str, object]:
         p = {"mixer": self.mixer, "mixer_norm": self.mixer_norm}
         if self.ffn is not None:
@@ -330,13 +337,31 @@ class PostNormResidualBlock:
         feeds_next = (not f32) and nxt is not None and isinstance(nxt[1], PostNormResidualBlock)
         y = ws.get("block.t", (M, D), torch.float32)
         self.mixer.forward(h, y, False, batch, cache, env)
-        n1 = self.mixer_norm
         if self.ffn is None:
-            kernels.postnorm_residual(x, y, self.alpha, n1.weight, n1.bias, n1.eps, h=other if feeds_next else None)
+            self._sum(x, y, self.mixer_norm, other if feeds_next else None)
             return StreamRows(other) if feeds_next else None
-        kernels.postnorm_residual(x, y, self.alpha, n1.weight, n1.bias, n1.eps, h=other)
+        self._sum(x, y, self.mixer_norm, other)
         h2 = x if f32 else other
         self.ffn.forward(h2, y, False, batch, env)
-        n2 = self.ffn_norm
-        kernels.postnorm_residual(x, y, self.alpha, n2.weight, n2.bias, n2.eps, h=h if feeds_next else None)
+        self._sum(x, y, self.ffn_norm, h if feeds_next else None)
         return StreamRows(h) if feeds_next else None
+
+
+@BLOCKS.register("output_norm_residual")
+class OutputNormResidualBlock(PostNormResidualBlock):
+    """x <- x + norm1(Mixer(x));  x <- x + norm2(FeedForward(x)): the sublayers read the stream itself, as in the
+    post-norm arrangement, and only their results are normed (RMS norms) on the way into it.  Stream, sums and norms
+    are float; norm, sum and the copy of the new stream for the next sublayer are one launch."""
+
+    def __init__(self, mixer, ffn, mixer_norm, ffn_norm=None, post_mixer_norm=None, post_ffn_norm=None):
+        if post_mixer_norm is not None or post_ffn_norm is not None:
+            raise ValueError("the output-norm arrangement names its two norms mixer_norm and ffn_norm")
+        if (ffn is None) != (ffn_norm is None):
+            raise ValueError("a feed-forward and its norm come together or not at all")
+        for n in (mixer_norm, ffn_norm):
+            if n is not None and hasattr(n, "bias"):
+                raise ValueError("the output-norm arrangement takes RMS norms")
+        self.mixer, self.ffn, self.mixer_norm, self.ffn_norm = mixer, ffn, mixer_norm, ffn_norm
+
+    def _sum(self, x, y, norm, h) -> None:
+        kernels.outnorm_residual(x, y, norm.weight, norm.eps, h=h)

@@ -1,7 +1,8 @@
 """Token embedding and output head.
 
 x = embed[token] (src/dense.rs:172-177), times a constant where the design has one; logits = W_out . norm(x) with W_out the head's own
-matrix, or the embedding when the model ties them (src/dense.rs:195-196).  Logits are float.
+matrix, or the embedding when the model ties them (src/dense.rs:195-196), times a constant and soft-capped where the
+design has that.  Logits are float.
 """
 from __future__ import annotations
 
@@ -62,8 +63,12 @@ class TokenPositionEmbedding(TokenEmbedding):
 
 @HEADS.register("linear_head")
 class LinearHead(Part):
-    def __init__(self, vocab_size: int, hidden_size: int, tied: bool):
+    def __init__(self, vocab_size: int, hidden_size: int, tied: bool, scale: float = 1.0, softcap: float = 0.0):
+        """The logits z of the product become scale * z and, with `softcap` c > 0, c tanh(scale * z / c)."""
         self.V, self.D, self.tied = int(vocab_size), int(hidden_size), bool(tied)
+        self.scale, self.softcap = float(scale), float(softcap)
+        if self.softcap < 0:
+            raise ValueError(f"a cap on the logits must be positive (or 0 for none), got {softcap}")
         self.weight: torch.Tensor | None = None
 
     def tensors(self) -> dict[str, TensorSpec]:
@@ -81,3 +86,5 @@ class LinearHead(Part):
 
     def forward(self, logits: torch.Tensor, xn: torch.Tensor) -> None:
         kernels.linear(logits, xn, self.weight)
+        if self.scale != 1.0 or self.softcap > 0:
+            kernels.softcap(logits, self.scale, self.softcap)
