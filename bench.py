@@ -25,7 +25,7 @@ A step is one decode step of the whole batch.  One JSON line goes to stdout:
 
 Weights (1.8 GB) are far larger than L2, so consecutive steps cannot be served from L2.
 
-`--compare zekivik` (or `lenesun`, `kisilix`, `tevilix`) leaves all of that aside and prints a line of its own: prompt and decode times
+`--compare zekivik` (or `lenesun`, `kisilix`, `tevilix`, `zafilix`) leaves all of that aside and prints a line of its own: prompt and decode times
 of that design at a few layer sizes beside the closest LFM3 model at equal sizes, with every kernel entry point's time.
 """
 from __future__ import annotations
@@ -518,6 +518,71 @@ def _tevilix_kernel_work(cfg: dict, rows: int, batch: int, context: int) -> dict
     return {"bytes": by, "flops": fl}
 
 
+# ---- the Zafilix design beside LFM3 attention layers and the Lenesun design (--compare zafilix) ------------------
+def zafilix_config(width: int, ff: int, heads: int, kv_heads: int, dim: int, chunk: int, lat_heads: int, lat_dim: int,
+                   rot_dim: int, lat_vdim: int, kv_rank: int, window: int, layers: int, vocab: int, q_rank: int = 0) -> dict:
+    """Chunked attention and windowed latent attention alternate, every layer with the dense feed-forward; every layer
+    has tensors of its own.  (`q_rank` is the Lenesun side's.)"""
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+           "rot": {"dims": dim, "base": 500000.0, "scaling": {"factor": 4.0}}, "mask": {"size": chunk}}
+    lat = {"heads": lat_heads, "dim": lat_dim, "rot_dim": rot_dim, "vdim": lat_vdim, "kv_rank": kv_rank,
+           "scale": (lat_dim + rot_dim) ** -0.5, "rot": {"dims": rot_dim, "base": 10000.0}, "mask": {"size": window}}
+    ls = [{"type": "latent_attention" if i % 2 else "attention", "mixer": lat if i % 2 else att,
+           "mlp": {"kind": "dense", "ff": ff}} for i in range(layers)]
+    return {"architecture": "Zafilix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "logit_scale": 0.5, "logit_softcap": 30.0, "layers": ls}
+
+
+def lfm3_attention_like(width: int, ff: int, heads: int, kv_heads: int, dim: int, layers: int, vocab: int) -> dict:
+    """The closest design for the attention layers: the same heads and (gated) feed-forward width in every layer."""
+    return dict(lfm3_like(width, ff, heads, kv_heads, dim, layers, vocab), layer_types=["attention"] * layers)
+
+
+def lenesun_latent_like(width: int, heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int, kv_rank: int, layers: int,
+                        vocab: int) -> dict:
+    """The closest design for the latent layers: the same latent sizes in every layer, no feed-forward."""
+    cfg = lenesun_config(width, heads, dim, rot_dim, vdim, q_rank, kv_rank, 1, 1, 8, layers, vocab)
+    return dict(cfg, layers=[dict(cfg["layers"][0], mlp=None) for _ in range(layers)])
+
+
+ZAFILIX_SIZES = {
+    "w2048": dict(width=2048, ff=5632, heads=32, kv_heads=8, dim=64, chunk=4096, lat_heads=16, lat_dim=128, rot_dim=64,
+                  lat_vdim=128, kv_rank=512, window=1024, layers=6, q_rank=768),
+    "w1024": dict(width=1024, ff=4096, heads=16, kv_heads=4, dim=64, chunk=768, lat_heads=8, lat_dim=64, rot_dim=32,
+                  lat_vdim=64, kv_rank=256, window=512, layers=6, q_rank=384),
+    "w2048-d128": dict(width=2048, ff=8192, heads=16, kv_heads=4, dim=128, chunk=4096, lat_heads=16, lat_dim=64, rot_dim=64,
+                       lat_vdim=64, kv_rank=256, window=2048, layers=6, q_rank=512),
+}
+
+
+def _zafilix_kernel_work(cfg: dict, rows: int, batch: int, context: int) -> dict:
+    """What a step's launches of the design's own kernels have to move (bytes) or compute (flops), by entry point; the
+    rows of a sequence are its last ones, ending at `context`."""
+    W = cfg["width"]
+    by = {"leb_outnorm_residual": 0, "leb_activation": 0, "leb_qk_row_norm_rope_store": 0, "leb_attention_decode_prep": 0,
+          "leb_latent_rows": 0, "leb_heads_to_rows": 0, "leb_latent_attention": 0, "leb_softcap": batch * cfg["vocab"] * 8}
+    att = lat = 0
+    per_seq = rows // batch
+    for l in cfg["layers"]:
+        m = l["mixer"]
+        by["leb_outnorm_residual"] += (2 if l["mlp"] else 1) * rows * W * (4 + 4 + 4 + 2)     # x and y read, x and its copy written
+        if l["mlp"]:
+            by["leb_activation"] += rows * l["mlp"]["ff"] * (4 + 2)
+        size = m["mask"]["size"]
+        if l["type"] == "attention":
+            nh, nkv, hd, vd = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            by["leb_qk_row_norm_rope_store"] += rows * ((nh + nkv) * hd + nkv * vd) * 4
+            by["leb_attention_decode_prep"] += batch * ((context - 1) % size + 1) * nkv * (hd + vd) * 2
+            att += 2 * nh * (hd + vd) * batch * sum(i % size + 1 for i in range(context - per_seq, context))
+        else:
+            H, dk = m["heads"], m["kv_rank"] + m["rot_dim"]
+            by["leb_latent_rows"] += rows * (H * (m["dim"] + m["rot_dim"]) + dk) * 4
+            by["leb_heads_to_rows"] += rows * H * m["vdim"] * 4
+            by["leb_latent_attention"] += batch * min(context, size + per_seq - 1) * dk * 2 + rows * H * (dk + m["kv_rank"]) * 2
+            lat += 2 * H * (dk + m["kv_rank"]) * batch * sum(min(i + 1, size) for i in range(context - per_seq, context))
+    return {"bytes": by, "attention_flops": att, "latent_flops": lat}
+
+
 def compare_designs(which: str, steps: int, warmup: int) -> int:
     import numpy as np
     import torch
@@ -528,8 +593,14 @@ def compare_designs(which: str, steps: int, warmup: int) -> int:
     results = {}
     other = "zekivik" if which == "kisilix" else ("kisilix" if which == "tevilix" else "lfm3")
     for size_name, sz in {"zekivik": COMPARE_SIZES, "lenesun": LENESUN_SIZES, "kisilix": KISILIX_SIZES,
-                          "tevilix": KISILIX_SIZES}[which].items():
-        if which == "tevilix":
+                          "tevilix": KISILIX_SIZES, "zafilix": ZAFILIX_SIZES}[which].items():
+        more = []
+        if which == "zafilix":
+            zc = zafilix_config(vocab=32768, **sz)
+            lc = lfm3_attention_like(sz["width"], sz["ff"], sz["heads"], sz["kv_heads"], sz["dim"], sz["layers"], 32768)
+            more = [("lenesun", lenesun_latent_like(sz["width"], sz["lat_heads"], sz["lat_dim"], sz["rot_dim"], sz["lat_vdim"],
+                                                    sz["q_rank"], sz["kv_rank"], sz["layers"], 32768))]
+        elif which == "tevilix":
             zc = tevilix_config(vocab=32768, **sz)
             lc = kisilix_config(vocab=32768, **sz)
         elif which == "kisilix":
@@ -543,14 +614,19 @@ def compare_designs(which: str, steps: int, warmup: int) -> int:
             zc = lenesun_config(vocab=32768, **sz)
             lc = lfm3_moe_like(sz["width"], sz["heads"], sz["dim"], sz["experts"], sz["top"], sz["ff"], sz["layers"], 32768)
         row = {}
-        for label, cfg in ((which, zc), (other, lc)):
+        for label, cfg in [(which, zc), (other, lc)] + more:
             eng = Engine.from_config(cfg, seed=0, dtype="bfloat16", max_tokens=8 * 2304 + 4096, max_seqs=16)
             nums = model_numbers(eng)
             r = {"weights_gb": round(nums["weight_bytes"] / 1e9, 3)}
             print(f"[bench] {size_name} {label}: {r['weights_gb']} GB of weights", file=sys.stderr, flush=True)
             pre_ms = time_prefill(eng, PREFILL_TOKENS, 3, 5, rng)
             print(f"[bench] {size_name} {label}: prompt of {PREFILL_TOKENS} tokens {pre_ms:.3f} ms", file=sys.stderr, flush=True)
-            if label == "tevilix":      # a position sees its window
+            if label == "zafilix":      # a position sees its chunk or its window
+                work = _zafilix_kernel_work(cfg, PREFILL_TOKENS, 1, PREFILL_TOKENS)
+                attn_flops = work["attention_flops"] + work["latent_flops"]
+                w1 = _zafilix_kernel_work(cfg, 1, 1, 2048)["bytes"]
+                kv_seen = [w1["leb_attention_decode_prep"] + w1["leb_latent_attention"]]
+            elif label == "tevilix":      # a position sees its window
                 attn_flops = _tevilix_kernel_work(cfg, PREFILL_TOKENS, 1, PREFILL_TOKENS)["flops"]["leb_attention_mixed"]
                 kv_seen = [sum(min(2048, l["mixer"]["left"]["mask"]["size"]) * l["mixer"]["left"]["kv_heads"]
                                * (l["mixer"]["left"]["dim"] + l["mixer"]["left"]["vdim"]) * 2
@@ -594,7 +670,13 @@ def compare_designs(which: str, steps: int, warmup: int) -> int:
             eng.release(seqs)
             dec_k = t.summary()
             by, fl = {}, {}
-            if label == "tevilix":
+            if label == "zafilix":
+                wp, wd = _zafilix_kernel_work(cfg, PREFILL_TOKENS, 1, PREFILL_TOKENS), _zafilix_kernel_work(cfg, 8, 8, 2048)
+                by = {"prefill": {k: v for k, v in wp["bytes"].items() if k not in ("leb_latent_attention", "leb_attention_decode_prep")},
+                      "decode_b8": dict(wd["bytes"], leb_attention_decode=wd["bytes"]["leb_attention_decode_prep"])}
+                fl = {"prefill": {"leb_latent_attention": wp["latent_flops"], "leb_attention_prefill_tc": wp["attention_flops"],
+                                  "leb_attention_prefill": wp["attention_flops"]}}
+            elif label == "tevilix":
                 wp, wd = _tevilix_kernel_work(cfg, PREFILL_TOKENS, 1, PREFILL_TOKENS), _tevilix_kernel_work(cfg, 8, 8, 2048)
                 by = {"prefill": wp["bytes"], "decode_b8": wd["bytes"]}
                 fl = {"prefill": dict(wp["flops"], leb_attention_mixed_mma=wp["flops"]["leb_attention_mixed"])}
@@ -612,7 +694,7 @@ def compare_designs(which: str, steps: int, warmup: int) -> int:
                     for name in ("leb_attention_decode", "leb_attention_decode_prep", "leb_attention_general"):
                         by["decode_b8"][name] = 8 * 2048 * nums["kv_bytes_per_token"]
             elif label == "lenesun":
-                wp, wd = _lenesun_kernel_work(zc, PREFILL_TOKENS, 1, PREFILL_TOKENS), _lenesun_kernel_work(zc, 8, 8, 2048)
+                wp, wd = _lenesun_kernel_work(cfg, PREFILL_TOKENS, 1, PREFILL_TOKENS), _lenesun_kernel_work(cfg, 8, 8, 2048)
                 by = {"prefill": {k: v for k, v in wp["bytes"].items() if k != "leb_latent_attention"}, "decode_b8": wd["bytes"]}
                 fl = {"prefill": {"leb_latent_attention": wp["attention_flops"]}}
             else:     # the other design's attention, for the comparison: flops of a prompt, cache bytes of a decode step
@@ -640,6 +722,7 @@ def compare_designs(which: str, steps: int, warmup: int) -> int:
         results[size_name] = {"sizes": sz, **row}
     against = {"zekivik": "lfm3 hybrid at equal layer sizes", "kisilix": "zekivik hybrid at equal layer sizes",
                "tevilix": "kisilix at equal layer sizes",
+               "zafilix": "lfm3 with attention in every layer, and lenesun with latent attention alone, at equal layer sizes",
                "lenesun": "lfm3 with attention and experts in every layer at equal layer sizes"}[which]
     print(json.dumps({"compare": which, "against": against, "dtype": "bf16",
                       "data": "synthetic (random weights, uniform random token ids)", "peaks": pk_src,
@@ -666,7 +749,7 @@ def main() -> int:
     ap.add_argument("--unequal", type=int, default=0, metavar="N",
                     help="instead of the default run: N requests with prompts of U[64, 2048] tokens generate "
                          "--steps tokens each in one batch through the Python entry point (prints its own JSON line)")
-    ap.add_argument("--compare", default="", choices=["", "zekivik", "lenesun", "kisilix", "tevilix"],
+    ap.add_argument("--compare", default="", choices=["", "zekivik", "lenesun", "kisilix", "tevilix", "zafilix"],
                     help="instead of the default run: prefill and decode of that design at a few layer sizes beside "
                          "the closest other design at equal sizes, with every kernel's time (prints its own JSON line)")
     args = ap.parse_args()

@@ -88,8 +88,8 @@ __device__ __forceinline__ float gate_mul(float g, float u, int act) {
   }
   return silu_mul<T>(g, u);
 }
-// An activation without a gate in a storing epilogue (code 0) of the products that take it (the weight stream of a
-// decode step, dense and grouped): code LEB_PLAIN_ACT_BASE + a in the place of the gated activation, a as
+// An activation without a gate in a storing epilogue (code 0) of the bfloat16 products that take it (the weight
+// stream of a decode step and the tcgen05 products, dense and grouped): code LEB_PLAIN_ACT_BASE + a in the place of the gated activation, a as
 // leb_activation counts them (0 the erf form of gelu, 1 the square of relu, 2 the tanh form of gelu, 3 silu).  The
 // exact functions, as the activation kernel uses them: a row gives the same numbers through either.
 #define LEB_PLAIN_ACT_BASE 16

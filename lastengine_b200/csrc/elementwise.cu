@@ -575,7 +575,6 @@ __global__ void __launch_bounds__(256)
 outnorm_residual_vec_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ w, float eps,
                             TH* __restrict__ h, int D) {
   __shared__ float red[33];
-  pdl_trigger();   // the kernel after this one may start and wait (see common.cuh)
   pdl_wait();
   const size_t m = blockIdx.x;
   const float4* y4 = reinterpret_cast<const float4*>(y + m * D);
@@ -620,7 +619,6 @@ __global__ void __launch_bounds__(256)
 outnorm_residual_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ w, float eps,
                         TH* __restrict__ h, int D) {
   __shared__ float red[33];
-  pdl_trigger();   // the kernel after this one may start and wait (see common.cuh)
   pdl_wait();
   const size_t m = blockIdx.x;
   float s = 0.f;
@@ -640,6 +638,7 @@ LEB_API int leb_outnorm_residual(float* x, const float* y, const float* w, float
   const bool b16 = h && h_dtype == LEB_BF16;
   const bool vec = D % 4 == 0 && D <= 4096 && ((((uintptr_t)x | (uintptr_t)y | (uintptr_t)w) & 15) == 0) &&
                    ((uintptr_t)h & 15) == 0;
+  LebPlainLaunches plain(true);
   const dim3 grid(M), block(256);
 #define LEB_ONR(CH_)                                                                                                       \
   (b16 ? leb_launch(outnorm_residual_vec_kernel<bf16, CH_>, grid, block, 0, st, x, y, w, eps, (bf16*)h, D)               \
@@ -661,7 +660,6 @@ LEB_API int leb_outnorm_residual(float* x, const float* y, const float* w, float
 
 // z -> cap tanh(scale z / cap) in place (cap <= 0: z -> scale z); four numbers a thread.
 __global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ z, float scale, float cap, size_t n) {
-  pdl_trigger();   // the kernel after this one may start and wait (see common.cuh)
   pdl_wait();
   const size_t i0 = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 4;
   if (i0 + 4 <= n && ((uintptr_t)z & 15) == 0) {
@@ -684,6 +682,7 @@ __global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ z, flo
 
 LEB_API int leb_softcap(float* z, float scale, float cap, size_t n, cudaStream_t st) {
   if (n == 0) return 0;
+  LebPlainLaunches plain(true);
   leb_launch(softcap_kernel, dim3((unsigned)((n + 1023) / 1024)), dim3(256), 0, st, z, scale, cap, n);
   LEB_CHECK_LAUNCH("leb_softcap");
   return 0;

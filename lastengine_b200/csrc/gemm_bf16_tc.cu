@@ -39,7 +39,7 @@ __global__ void __launch_bounds__(TC_THREADS)
 gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                     TC* __restrict__ C_all, int M, int N, int K, int ldc, int epilogue, int* __restrict__ status,
                     const int* __restrict__ group_offsets, int n_groups) {
-  const int act = epilogue >> 8;   // the gated epilogue's activation rides in the upper bits
+  const int act = epilogue >> 8;   // the epilogue's activation rides in the upper bits
   epilogue &= 255;
   __shared__ int g_cum[GROUPED ? TC_MAX_GROUPS + 1 : 1], g_off[GROUPED ? TC_MAX_GROUPS + 1 : 1];
   extern __shared__ uint8_t smem_raw[];
@@ -269,6 +269,10 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
           const int row = row_base + rr;
           if (row >= m_end || col >= n_out) continue;
           float4 f = *reinterpret_cast<const float4*>(stg + rr * 36 + lc);
+          if (sizeof(TC) == 2 && LEB_PLAIN_ACT_OK(act, epilogue)) {
+            f.x = plain_act(f.x, act); f.y = plain_act(f.y, act);
+            f.z = plain_act(f.z, act); f.w = plain_act(f.w, act);
+          }
           TC* o = C + (size_t)row * ldc + col;
           if (vec && col + 3 < n_out) {
             if (sizeof(TC) == 4) {
@@ -341,13 +345,14 @@ LEB_API int leb_gemm_bf16_tc_supported(const void* A, const void* W, int K, int 
   return K > 0 && K % 8 == 0 && lda % 8 == 0 && ((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0;
 }
 
-// epilogue: 0 store, 1 add into float C, 2 SwiGLU over 16/16 interleaved gate/up rows (C has N/2 columns).
+// epilogue: 0 store (bfloat16 C: with an activation without a gate, LEB_PLAIN_ACT_BASE), 1 add into float C, 2 SwiGLU over 16/16 interleaved gate/up rows (C has N/2 columns).
 // status: device int, set non-zero by a block whose bounded wait gave up.
 LEB_API int leb_gemm_bf16_tc(void* C, int c_dtype, const void* A, const void* W, int M, int N, int K, int lda,
                              int ldc, int epilogue, int* status, cudaStream_t st) {
   const int act_ = epilogue >> 8;
   epilogue &= 255;
-  LEB_REQUIRE(LEB_GATE_ACT_OK(act_, epilogue), "leb_gemm_bf16_tc: activation %d goes with the gated epilogue only", act_);
+  LEB_REQUIRE(LEB_GATE_ACT_OK(act_, epilogue) || (LEB_PLAIN_ACT_OK(act_, epilogue) && c_dtype == LEB_BF16),
+              "leb_gemm_bf16_tc: activation %d does not go with epilogue %d", act_, epilogue);
   g_leb_gate_act = act_;
   if (M <= 0 || N <= 0) return 0;
   LEB_REQUIRE(leb_gemm_bf16_tc_supported(A, W, K, lda), "leb_gemm_bf16_tc: operands not aligned for TMA (K %d, lda %d)", K, lda);
@@ -405,7 +410,8 @@ LEB_API int leb_gemm_bf16_tc_sliced(void* C, int c_dtype, const void* A, const v
                                     int ldc, int epilogue, float* part, int n_slices, int* status, cudaStream_t st) {
   const int act_ = epilogue >> 8;
   epilogue &= 255;
-  LEB_REQUIRE(LEB_GATE_ACT_OK(act_, epilogue), "leb_gemm_bf16_tc_sliced: activation %d goes with the gated epilogue only", act_);
+  LEB_REQUIRE(LEB_GATE_ACT_OK(act_, epilogue) || (LEB_PLAIN_ACT_OK(act_, epilogue) && c_dtype == LEB_BF16),
+              "leb_gemm_bf16_tc_sliced: activation %d does not go with epilogue %d", act_, epilogue);
   g_leb_gate_act = act_;
   if (M <= 0 || N <= 0) return 0;
   LEB_REQUIRE(leb_gemm_bf16_tc_supported(A, W, K, lda), "leb_gemm_bf16_tc_sliced: operands not aligned for TMA (K %d, lda %d)", K, lda);
@@ -420,6 +426,7 @@ LEB_API int leb_gemm_bf16_tc_sliced(void* C, int c_dtype, const void* A, const v
   CUtensorMap ma, mw;
   if (tensor_map(&ma, A, M, K, lda, TC_BM)) return 1;
   if (tensor_map(&mw, W, N, K, K, 256)) return 1;
+  // (the partial tiles are float: their plain store applies no activation, the second kernel does)
   if (launch_tc<float, 256, 4>(part, ma, mw, M, N, K, N, 0, status, st, nullptr, n_slices)) return 1;
   return leb_slices_finish(C, c_dtype, part, M, N, ldc, epilogue, n_slices, st);
 }
@@ -432,7 +439,8 @@ LEB_API int leb_gemm_bf16_tc_grouped(void* C, int c_dtype, const void* A, const 
                                      cudaStream_t st) {
   const int act_ = epilogue >> 8;
   epilogue &= 255;
-  LEB_REQUIRE(LEB_GATE_ACT_OK(act_, epilogue), "leb_gemm_bf16_tc_grouped: activation %d goes with the gated epilogue only", act_);
+  LEB_REQUIRE(LEB_GATE_ACT_OK(act_, epilogue) || (LEB_PLAIN_ACT_OK(act_, epilogue) && c_dtype == LEB_BF16),
+              "leb_gemm_bf16_tc_grouped: activation %d does not go with epilogue %d", act_, epilogue);
   g_leb_gate_act = act_;
   if (P <= 0 || N <= 0 || n_groups <= 0) return 0;
   LEB_REQUIRE(n_groups <= TC_MAX_GROUPS, "leb_gemm_bf16_tc_grouped: %d groups; at most %d", n_groups, TC_MAX_GROUPS);

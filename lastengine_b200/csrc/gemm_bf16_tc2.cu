@@ -68,7 +68,7 @@ template <typename TC>
 __global__ void __launch_bounds__(T2_THREADS)
 gemm_bf16_tc2_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                      TC* __restrict__ C, int M, int N, int K, int ldc, int epilogue, int* __restrict__ status) {
-  const int act = epilogue >> 8;   // the gated epilogue's activation rides in the upper bits
+  const int act = epilogue >> 8;   // the epilogue's activation rides in the upper bits
   epilogue &= 255;
   constexpr int BN = T2_BN, STAGES = T2_STAGES;
   constexpr int A_BYTES = 128 * TC_BK * 2, B_BYTES = 128 * TC_BK * 2;   // this block's halves
@@ -240,6 +240,10 @@ gemm_bf16_tc2_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
             const int row = row_base + rr;
             if (row >= M || col >= n_out) continue;
             float4 f = *reinterpret_cast<const float4*>(stg + rr * 36 + lc);
+            if (sizeof(TC) == 2 && LEB_PLAIN_ACT_OK(act, epilogue)) {
+              f.x = plain_act(f.x, act); f.y = plain_act(f.y, act);
+              f.z = plain_act(f.z, act); f.w = plain_act(f.w, act);
+            }
             TC* o = C + (size_t)row * ldc + col;
             if (vec && col + 3 < n_out) {
               if (sizeof(TC) == 4) {
@@ -325,7 +329,8 @@ LEB_API int leb_gemm_bf16_tc2(void* C, int c_dtype, const void* A, const void* W
                               int ldc, int epilogue, int* status, cudaStream_t st) {
   const int act_ = epilogue >> 8;
   epilogue &= 255;
-  LEB_REQUIRE(LEB_GATE_ACT_OK(act_, epilogue), "leb_gemm_bf16_tc2: activation %d goes with the gated epilogue only", act_);
+  LEB_REQUIRE(LEB_GATE_ACT_OK(act_, epilogue) || (LEB_PLAIN_ACT_OK(act_, epilogue) && c_dtype == LEB_BF16),
+              "leb_gemm_bf16_tc2: activation %d does not go with epilogue %d", act_, epilogue);
   g_leb_gate_act = act_;
   if (M <= 0 || N <= 0) return 0;
   LEB_REQUIRE(K > 0 && K % 8 == 0 && lda % 8 == 0 && ((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0,

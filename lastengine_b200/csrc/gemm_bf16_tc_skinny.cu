@@ -205,7 +205,11 @@ gemm_tc_skinny_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
           bf16* o = (bf16*)C + (size_t)c0 * ldc + n;
 #pragma unroll
           for (int i = 0; i < 32; i++)
-            if (c0 + i < M) o[(size_t)i * ldc] = __float2bfloat16_rn(__uint_as_float(v[i]) * row_scale[c0 + i]);
+            if (c0 + i < M) {
+              float a = __uint_as_float(v[i]) * row_scale[c0 + i];
+              if (LEB_PLAIN_ACT_OK(act, epilogue)) a = plain_act(a, act);
+              o[(size_t)i * ldc] = __float2bfloat16_rn(a);
+            }
         }
       }
     }
@@ -317,6 +321,7 @@ skinny_finish_kernel(TC* __restrict__ C, const float* __restrict__ part, int M, 
     a = sum_slices(part + (size_t)m * N + j, slab, n_slices) * r;
     TC* o = C + (size_t)m * ldc + j;
     if (epilogue == 1) a += to_f32(*o);
+    if (sizeof(TC) == 2 && LEB_PLAIN_ACT_OK(act, epilogue)) a = plain_act(a, act);
     *o = from_f32<TC>(a);
   }
   if (nm.emit_vals) {   // the new residual, for the norm that follows: bf16(x * g) and the sum of x^2 per 16 columns
@@ -428,7 +433,8 @@ LEB_API int leb_gemm_bf16_skinny(void* C, int c_dtype, const void* A, const void
                                  cudaStream_t st) {
   const int act_ = epilogue >> 8;
   epilogue &= 255;
-  LEB_REQUIRE(LEB_GATE_ACT_OK(act_, epilogue), "leb_gemm_bf16_skinny: activation %d goes with the gated epilogue only", act_);
+  LEB_REQUIRE(LEB_GATE_ACT_OK(act_, epilogue) || (LEB_PLAIN_ACT_OK(act_, epilogue) && c_dtype == LEB_BF16),
+              "leb_gemm_bf16_skinny: activation %d does not go with epilogue %d", act_, epilogue);
   g_leb_gate_act = act_;
   if (M <= 0 || N <= 0) return 0;
   LEB_REQUIRE(leb_gemm_bf16_skinny_supported(A, W, M, K, lda), "leb_gemm_bf16_skinny: takes 1..128 rows and TMA-aligned operands (M %d, K %d, lda %d)", M, K, lda);

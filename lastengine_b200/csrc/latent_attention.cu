@@ -148,7 +148,6 @@ latent_rows_kernel(T* __restrict__ qn, T* __restrict__ qr, const T* __restrict__
                    const float* __restrict__ inv_freq, int rot_dims, int neox, int M, int H, int dim, int dim_p, int rank,
                    int rot, int page_size, int wide) {
   __shared__ float red[33];
-  pdl_trigger();   // the kernel after this one may start and wait (see common.cuh)
   pdl_wait();
   const int m = blockIdx.x;
   const T* row = in + (size_t)m * ld_in;
@@ -382,6 +381,7 @@ LEB_API int leb_latent_rows(void* qn, void* qr, const void* in, int ld_in, int d
               "leb_latent_rows: %d rotated dimensions of %d", rot_dims, rot);
   LEB_REQUIRE(dtype == LEB_F32 || dtype == LEB_BF16, "leb_latent_rows: unknown dtype %d", dtype);
   const int wide = latent_wide(dtype, dim, dim_p, dim + rot, (uintptr_t)in | (uintptr_t)qn) && ld_in % (dtype == LEB_BF16 ? 8 : 4) == 0;
+  LebPlainLaunches plain(true);
   const dim3 grid(M, pool ? 2 : 1), block(256);
   if (dtype == LEB_F32)
     leb_launch(latent_rows_kernel<float>, grid, block, 0, st, (float*)qn, (float*)qr, (const float*)in, ld_in, (float*)pool,

@@ -271,7 +271,6 @@ __global__ void __launch_bounds__(256) qk_row_norm_rope_store_kernel(
     int page_size, int vd, int hin, int vin) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[33];
-  pdl_trigger();   // the kernel after this one may start and wait (see common.cuh)
   pdl_wait();
   if ((int)blockIdx.x >= M) {
     if (blockIdx.y == 0)
@@ -393,6 +392,7 @@ LEB_API int leb_qk_row_norm_rope_store(void* q_out, const void* q_in, int q_stri
   LEB_REQUIRE(q_norm_w && (!k_in || k_norm_w), "leb_qk_row_norm_rope_store: the rows' norm weights are required");
   LEB_REQUIRE(dtype == LEB_F32 || dtype == LEB_BF16, "leb_qk_row_norm_rope_store: unknown dtype %d", dtype);
   const int tiles = k_in ? ceil_div(M, VT_ROWS) * nkv : 0;
+  LebPlainLaunches plain(true);
   const dim3 grid(M + tiles, k_in ? 2 : 1), block(256);
   const int wide = (nh > nkv ? nh : nkv) * hin;
   const uintptr_t al = (uintptr_t)q_out | (uintptr_t)q_in | (uintptr_t)k_in | (uintptr_t)k_pool | (uintptr_t)q_norm_w | (uintptr_t)k_norm_w;

@@ -592,22 +592,19 @@ PLAIN_ACT_BASE = 16      # a storing epilogue with an activation without a gate:
 
 
 def plain_act_epilogue(act: int) -> int:
-    """The epilogue code of a product that stores act(x . w^T); only for steps `stream_takes_plain_act` accepts."""
+    """The epilogue code of a product that stores act(x . w^T); only for operands `takes_plain_act` accepts."""
     return (PLAIN_ACT_BASE + int(act)) << 8
 
 
-def stream_takes_plain_act(x: torch.Tensor, w: torch.Tensor, rows: int, n_groups: int = 0) -> bool:
-    """Whether `linear` would run these rows through the weight stream of a decode step (dense: up to SMALL_M
-    rows; grouped: up to 16 rows an expert), the products whose storing epilogue takes an activation without a
-    gate.  Every other product leaves float results for `activation`."""
-    if x.dtype != torch.bfloat16 or not w.is_contiguous():
+def takes_plain_act(x: torch.Tensor, w: torch.Tensor, n_groups: int = 0) -> bool:
+    """Whether `linear` runs these rows through a bfloat16 product whose storing epilogue takes an activation
+    without a gate: the weight stream and the tcgen05 products, which fetch 16 bytes at a time.  Every other
+    product leaves float results for `activation`."""
+    if x.dtype != torch.bfloat16 or not w.is_contiguous() or _OPTIONAL_TC[0] is None:
         return False
-    K = x.shape[1]
-    if K % 8 != 0 or x.stride(0) % 8 != 0 or x.data_ptr() % 16 != 0 or w.data_ptr() % 16 != 0:
+    if not _tma_ok(x, w, x.shape[1]):
         return False
-    if n_groups:
-        return n_groups <= 256 and rows <= 16 * n_groups and (w.shape[1] * w.shape[2] * 2) % 16 == 0
-    return rows <= SMALL_M
+    return not n_groups or (n_groups <= 256 and (w.shape[1] * w.shape[2] * 2) % 16 == 0)
 
 
 def activation(out: torch.Tensor, x: torch.Tensor, act: int) -> None:

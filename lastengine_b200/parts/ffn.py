@@ -94,7 +94,7 @@ class SwiGLU(FeedForward):
 class DenseFeedForward(FeedForward):
     """f = W_down act(W_up h) without a gate; act is the erf form of gelu unless `activation` names another
     ("relu_squared": max(z, 0)^2; "gelu_tanh"; "silu").  The up projection's float sums go through the
-    activation in float: in the product's epilogue in a decode step, in a launch of its own otherwise.
+    activation in float: in the product's epilogue in bfloat16, in a launch of its own otherwise.
     `names`: (up, down)."""
 
     def __init__(self, hidden_size: int, intermediate_size: int, activation: str = "gelu",
@@ -117,8 +117,8 @@ class DenseFeedForward(FeedForward):
         M = h.shape[0]
         ws = env.workspace
         a = ws.get("ffn.a", (M, self.F), env.dtype)
-        if kernels.stream_takes_plain_act(h, self.w1, M):
-            # a decode step: the weight stream applies the activation to its float sums before it stores
+        if kernels.takes_plain_act(h, self.w1):
+            # the product applies the activation to its float sums before it stores
             kernels.linear(a, h, self.w1, kernels.plain_act_epilogue(self.act))
         else:
             u = ws.get("ffn.u", (M, self.F), torch.float32)
@@ -258,7 +258,7 @@ class SigmoidTopKMoE(FeedForward):
         xs = ws.get("moe.xs", (P, self.D), env.dtype)
         kernels.gather_rows(xs, h, sorted_pair, div=self.k)
         a = ws.get("moe.a", (P, self.Fe), env.dtype)
-        if not self.gated and kernels.stream_takes_plain_act(xs, self.w13, P, n_groups=self.E):
+        if not self.gated and kernels.takes_plain_act(xs, self.w13, n_groups=self.E):
             kernels.linear(a, xs, self.w13, kernels.plain_act_epilogue(self.act), group_offsets=offsets, rows_hint=P)
         elif not self.gated:
             u = ws.get("moe.gu", (P, self.Fe), torch.float32)
