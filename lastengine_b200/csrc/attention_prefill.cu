@@ -78,7 +78,7 @@ attention_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ q,
   if (row0 >= nrows) return;
 
   // rows of this lane: tile mt, halves 0 (row r) and 1 (row r + 8)
-  int rpos[MT][2], rhead[MT][2], rlo[MT][2];
+  int rpos[MT][2], rhead[MT][2];
   bool rok[MT][2];
 #pragma unroll
   for (int mt = 0; mt < MT; mt++)
@@ -88,7 +88,6 @@ attention_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ q,
       rok[mt][hh] = row < nrows;
       rpos[mt][hh] = p_lo + row / G;       // position within this step's rows of the sequence
       rhead[mt][hh] = row % G;
-      rlo[mt][hh] = first_key(pos0 + rpos[mt][hh], window, chunk);
     }
 
   if (slot < 0) {   // padding sequence: zeros
@@ -195,6 +194,7 @@ attention_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ q,
       }
       float tmax[2] = {ATP_NEG, ATP_NEG};
       if (need_mask) {
+        const int rlo[2] = {first_key(pos0 + rpos[mt][0], window, chunk), first_key(pos0 + rpos[mt][1], window, chunk)};
 #pragma unroll
         for (int t = 0; t < 4; t++)
 #pragma unroll
@@ -202,7 +202,7 @@ attention_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ q,
             const int hh = e >> 1;
             const int kp = key0 + 8 * c + 2 * t + (e & 1);
             const int qp = pos0 + rpos[mt][hh];
-            const bool valid = kp <= qp && kp >= rlo[mt][hh];
+            const bool valid = kp <= qp && kp >= rlo[hh];
             s[t][e] = valid ? s[t][e] * scale2 : ATP_NEG;
             tmax[hh] = fmaxf(tmax[hh], s[t][e]);
           }

@@ -340,25 +340,44 @@ latent_attention_kernel(T* __restrict__ out, int ld_out, float* __restrict__ par
 
 // Merge of the key-range splits of one (row, head), with the sink as one more term of the
 // denominator: out = sum_s acc_s e^(m_s - m) / (sum_s l_s e^(m_s - m) + e^(sink - m)).
+// The first warp turns the splits' maxima and sums into one factor each; then a thread per number of the latent adds the
+// splits' sums, eight loads at a time (n_splits <= 64).
 template <typename T>
-__global__ void latent_merge_kernel(T* __restrict__ out, int ld_out, const float* __restrict__ part,
-                                    const float* __restrict__ sink, int M, int H, int rank, int n_splits) {
+__global__ void __launch_bounds__(128)
+latent_merge_kernel(T* __restrict__ out, int ld_out, const float* __restrict__ part, const float* __restrict__ sink, int M,
+                    int H, int rank, int n_splits) {
+  __shared__ float f_s[64];
   pdl_wait();
   const size_t m = blockIdx.x;
   const int h = blockIdx.y;
   const size_t step = rank + 2;
   const float* pp = part + ((m * H + h) * n_splits) * step;
-  float mn = sink ? sink[h] : LAT_NEG;
-  for (int s = 0; s < n_splits; s++) mn = fmaxf(mn, pp[s * step]);
-  float den = sink ? expf(sink[h] - mn) : 0.f;
-  for (int s = 0; s < n_splits; s++) den += pp[s * step + 1] * expf(pp[s * step] - mn);
-  const float inv = den > 0.f ? 1.0f / den : 0.f;
+  if (threadIdx.x < 32) {
+    const int s0 = threadIdx.x, s1 = threadIdx.x + 32;
+    const float m0 = s0 < n_splits ? pp[s0 * step] : LAT_NEG, m1 = s1 < n_splits ? pp[s1 * step] : LAT_NEG;
+    const float l0 = s0 < n_splits ? pp[s0 * step + 1] : 0.f, l1 = s1 < n_splits ? pp[s1 * step + 1] : 0.f;
+    const float sk = sink ? sink[h] : LAT_NEG;
+    const float mn = fmaxf(sk, warp_max(fmaxf(m0, m1)));
+    const float e0 = expf(m0 - mn), e1 = expf(m1 - mn);
+    const float den = warp_sum(l0 * e0 + l1 * e1) + (sink ? expf(sk - mn) : 0.f);
+    const float inv = den > 0.f ? 1.0f / den : 0.f;
+    f_s[s0] = e0 * inv;
+    f_s[s1] = e1 * inv;
+  }
+  __syncthreads();
   T* o = out + ((size_t)h * M + m) * ld_out;
   for (int d = threadIdx.x; d < ld_out; d += blockDim.x) {
     float a = 0.f;
-    if (d < rank)
-      for (int s = 0; s < n_splits; s++) a += pp[s * step + 2 + d] * expf(pp[s * step] - mn);
-    o[d] = from_f32<T>(a * inv);
+    if (d < rank) {
+      for (int s0 = 0; s0 < n_splits; s0 += 8) {
+        float v[8];
+#pragma unroll
+        for (int q = 0; q < 8; q++) v[q] = s0 + q < n_splits ? pp[(s0 + q) * step + 2 + d] : 0.f;
+#pragma unroll
+        for (int q = 0; q < 8; q++) a += s0 + q < n_splits ? v[q] * f_s[s0 + q] : 0.f;
+      }
+    }
+    o[d] = from_f32<T>(a);
   }
 }
 
@@ -513,8 +532,8 @@ LEB_API int leb_latent_attention(void* out, int ld_out, float* part, const void*
   LEB_REQUIRE(rot >= 0 && rot <= 256, "leb_latent_attention: %d rotated dimensions outside 0..256", rot);
   LEB_REQUIRE(ld_out >= rank, "leb_latent_attention: result rows of %d for a latent of %d", ld_out, rank);
   LEB_REQUIRE(page_size % 32 == 0, "leb_latent_attention: page size %d is not a multiple of 32", page_size);
-  LEB_REQUIRE(n_splits >= 1 && (n_splits == 1 || (max_qlen == 1 && part)),
-              "leb_latent_attention: splits need single-row sequences and scratch");
+  LEB_REQUIRE(n_splits >= 1 && n_splits <= 64 && (n_splits == 1 || (max_qlen == 1 && part)),
+              "leb_latent_attention: up to 64 splits, and they need single-row sequences and scratch");
   LebPlainLaunches plain(true);
   int rc;
   const bool mma = g_latent_mma && dtype == LEB_BF16 && ld_out == rank && leb_latent_attention_mma_supported(rank, rot, page_size) &&

@@ -591,14 +591,24 @@ LEB_API int leb_embed_positions(float* x, void* h, int h_dtype, const void* tabl
 template <typename T>
 __global__ void cast_rows_kernel(T* __restrict__ out, const float* __restrict__ x, size_t n) {
   pdl_wait();
-  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-  if (i < n) out[i] = from_f32<T>(x[i]);
+  const size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (i + 4 <= n && (((uintptr_t)x | (uintptr_t)out) & 15) == 0) {     // four numbers a thread
+    const float4 v = *reinterpret_cast<const float4*>(x + i);
+    if (sizeof(T) == 2) {
+      __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+      *reinterpret_cast<uint2*>(out + i) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+    } else {
+      *reinterpret_cast<float4*>(out + i) = v;
+    }
+    return;
+  }
+  for (size_t k = i; k < n && k < i + 4; k++) out[k] = from_f32<T>(x[k]);
 }
 
 LEB_API int leb_cast_rows(void* out, int dtype, const float* x, size_t n, cudaStream_t st) {
   if (n == 0) return 0;
   LebPlainLaunches plain(true);
-  const dim3 grid((unsigned)((n + 255) / 256)), block(256);
+  const dim3 grid((unsigned)((n + 1023) / 1024)), block(256);
   if (dtype == LEB_F32) leb_launch(cast_rows_kernel<float>, grid, block, 0, st, (float*)out, x, n);
   else if (dtype == LEB_BF16) leb_launch(cast_rows_kernel<bf16>, grid, block, 0, st, (bf16*)out, x, n);
   else return leb_fail("leb_cast_rows: unknown dtype %d", dtype);
