@@ -341,9 +341,9 @@ latent_attention_kernel(T* __restrict__ out, int ld_out, float* __restrict__ par
 // Merge of the key-range splits of one (row, head), with the sink as one more term of the
 // denominator: out = sum_s acc_s e^(m_s - m) / (sum_s l_s e^(m_s - m) + e^(sink - m)).
 // The first warp turns the splits' maxima and sums into one factor each; then a thread per number of the latent adds the
-// splits' sums, eight loads at a time (n_splits <= 64).
+// splits' sums, sixteen loads at a time (n_splits <= 64).
 template <typename T>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(512)
 latent_merge_kernel(T* __restrict__ out, int ld_out, const float* __restrict__ part, const float* __restrict__ sink, int M,
                     int H, int rank, int n_splits) {
   __shared__ float f_s[64];
@@ -369,12 +369,12 @@ latent_merge_kernel(T* __restrict__ out, int ld_out, const float* __restrict__ p
   for (int d = threadIdx.x; d < ld_out; d += blockDim.x) {
     float a = 0.f;
     if (d < rank) {
-      for (int s0 = 0; s0 < n_splits; s0 += 8) {
-        float v[8];
+      for (int s0 = 0; s0 < n_splits; s0 += 16) {
+        float v[16];
 #pragma unroll
-        for (int q = 0; q < 8; q++) v[q] = s0 + q < n_splits ? pp[(s0 + q) * step + 2 + d] : 0.f;
+        for (int q = 0; q < 16; q++) v[q] = s0 + q < n_splits ? pp[(s0 + q) * step + 2 + d] : 0.f;
 #pragma unroll
-        for (int q = 0; q < 8; q++) a += s0 + q < n_splits ? v[q] * f_s[s0 + q] : 0.f;
+        for (int q = 0; q < 16; q++) a += s0 + q < n_splits ? v[q] * f_s[s0 + q] : 0.f;
       }
     }
     o[d] = from_f32<T>(a);
@@ -553,11 +553,11 @@ LEB_API int leb_latent_attention(void* out, int ld_out, float* part, const void*
 #undef LEB_LAT
   if (rc) return rc;
   if (n_splits > 1) {
-    dim3 grid(M, H);
+    dim3 grid(M, H), block(ld_out >= 512 ? 512 : ceil_div(ld_out, 32) * 32);
     if (dtype == LEB_F32)
-      leb_launch(latent_merge_kernel<float>, grid, dim3(128), 0, st, (float*)out, ld_out, part, sink, M, H, rank, n_splits);
+      leb_launch(latent_merge_kernel<float>, grid, block, 0, st, (float*)out, ld_out, part, sink, M, H, rank, n_splits);
     else
-      leb_launch(latent_merge_kernel<bf16>, grid, dim3(128), 0, st, (bf16*)out, ld_out, part, sink, M, H, rank, n_splits);
+      leb_launch(latent_merge_kernel<bf16>, grid, block, 0, st, (bf16*)out, ld_out, part, sink, M, H, rank, n_splits);
     LEB_CHECK_LAUNCH("leb_latent_attention merge");
   }
   return 0;
