@@ -10,7 +10,8 @@
 // window and pos+1 > window, else 0; softmax with the maximum subtracted; o = sum_t p_t v_t.
 // An optional per-head gate multiplies the head's output by sigmoid(gate) (src/dense.rs:147-150); it may also be
 // given per dimension of the head.  Instead of a window a layer may cut its positions into chunks (t0 = the start
-// of pos's chunk).
+// of pos's chunk).  `slopes` [nh]: slope_h (pos - t) is taken off the score of key t; `sinks` [nh]: one more logit per head in
+// the softmax's denominator, without a key and without a value (each or null).
 // Scores, maximum, exponentials, sums and the value accumulation are float.  The reference's
 // GPU kernels keep the same running (max, sum, acc) per warp and merge them
 // (src/cuda/dense.cu:94-123 whole range, :152-183 split range, :238-247 merge); this kernel lets
@@ -34,7 +35,8 @@ attention_kernel(T* __restrict__ out, float* __restrict__ part, const T* __restr
                  const int* __restrict__ seq_slot, const int* __restrict__ seq_pos0,
                  const int* __restrict__ seq_qstart, const int* __restrict__ seq_qlen,
                  const T* __restrict__ gate, int gate_stride, int gate_elem, int nh, int nkv, int hd, int vd,
-                 int page_size, int window, int chunk, float scale, int QT, int HC, int n_splits) {
+                 int page_size, int window, int chunk, float scale, const float* __restrict__ slopes,
+                 const float* __restrict__ sinks, int QT, int HC, int n_splits) {
   extern __shared__ float sm[];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int G = nh / nkv;
@@ -138,6 +140,7 @@ attention_kernel(T* __restrict__ out, float* __restrict__ part, const T* __restr
       for (int d = 0; d < hd; d++) s += qv[d] * kr[d];
       s *= scale;
       const int kp = key0 + lane;
+      if (slopes) s -= slopes[kvh * G + hc * HC + j] * (float)(qpos - kp);
       const bool valid = kp <= qpos && kp >= lo;
       s = valid ? s : ATT_NEG;
       const float mn = fmaxf(mx[ri], warp_max(s));
@@ -170,7 +173,7 @@ attention_kernel(T* __restrict__ out, float* __restrict__ part, const T* __restr
     const int h = kvh * G + hc * HC + j;
     const size_t m = (size_t)q0 + row_lo + i;
     if (n_splits == 1) {
-      const float inv = l[ri] > 0.f ? 1.0f / l[ri] : 0.f;
+      const float inv = sinks ? sink_quotient(mx[ri], l[ri], sinks[h]) : (l[ri] > 0.f ? 1.0f / l[ri] : 0.f);
 #pragma unroll
       for (int jj = 0; jj < HDL; jj++) {
         const int d = lane + 32 * jj;
@@ -197,8 +200,8 @@ attention_kernel(T* __restrict__ out, float* __restrict__ part, const T* __restr
 // (with more, the running sums are rescaled to the new maximum from group to group).
 template <typename T>
 __global__ void attention_merge_kernel(T* __restrict__ out, const float* __restrict__ part,
-                                       const T* __restrict__ gate, int gate_stride, int gate_elem, int nh,
-                                       int hd, int n_splits) {
+                                       const T* __restrict__ gate, int gate_stride, int gate_elem,
+                                       const float* __restrict__ sinks, int nh, int hd, int n_splits) {
   pdl_trigger();   // the kernel after this one may start and wait (see common.cuh)
   pdl_wait();
   const size_t m = blockIdx.x;
@@ -232,7 +235,8 @@ __global__ void attention_merge_kernel(T* __restrict__ out, const float* __restr
       M = cm;
     }
     const float g = gate ? head_gate(gate, m, gate_stride, h, d, hd, gate_elem) : 1.f;
-    out[(m * nh + h) * hd + d] = from_f32<T>(a * (L > 0.f ? 1.0f / L : 0.f) * g);
+    const float inv = sinks ? sink_quotient(M, L, sinks[h]) : (L > 0.f ? 1.0f / L : 0.f);
+    out[(m * nh + h) * hd + d] = from_f32<T>(a * inv * g);
   }
 }
 
@@ -241,8 +245,8 @@ static int launch_attention(void* out, float* part, const void* q, const void* k
                             const void* v_pool, const int* block_table, int bt_width,
                             const int* seq_slot, const int* seq_pos0, const int* seq_qstart,
                             const int* seq_qlen, const void* gate, int gate_stride, int gate_elem, int B, int nh,
-                            int nkv, int hd, int vd, int page_size, int window, int chunk, float scale, int max_qlen,
-                            int n_splits, cudaStream_t st) {
+                            int nkv, int hd, int vd, int page_size, int window, int chunk, float scale,
+                            const float* slopes, const float* sinks, int max_qlen, int n_splits, cudaStream_t st) {
   const int G = nh / nkv;
   const int HC = G < 8 ? G : 8;
   int QT = 32 / HC;
@@ -262,7 +266,7 @@ static int launch_attention(void* out, float* part, const void* q, const void* k
   kern<<<grid, 32 * ATT_WARPS, smem, st>>>(
       (T*)out, part, (const T*)q, (const CT*)k_pool, (const CT*)v_pool, block_table, bt_width,
       seq_slot, seq_pos0, seq_qstart, seq_qlen, (const T*)gate, gate_stride, gate_elem, nh, nkv, hd, vd, page_size,
-      window, chunk, scale, QT, HC, n_splits);
+      window, chunk, scale, slopes, sinks, QT, HC, n_splits);
   LEB_CHECK_LAUNCH("leb_attention");
   return 0;
 }
@@ -275,7 +279,7 @@ LEB_API int leb_attention(void* out, float* part, const void* q, const void* k_p
                           const int* seq_slot, const int* seq_pos0, const int* seq_qstart,
                           const int* seq_qlen, const void* gate, int gate_stride, int gate_elem, int M, int B,
                           int nh, int nkv, int hd, int page_size, int window, int chunk, float scale,
-                          int max_qlen, int n_splits, int vd, cudaStream_t st) {
+                          const float* slopes, const float* sinks, int max_qlen, int n_splits, int vd, cudaStream_t st) {
   if (M <= 0 || B <= 0) return 0;
   if (vd <= 0) vd = hd;
   LEB_REQUIRE(vd <= 256, "leb_attention: value head size %d outside 1..256", vd);
@@ -287,7 +291,7 @@ LEB_API int leb_attention(void* out, float* part, const void* q, const void* k_p
 #define LEB_ATT_W(T, CT, HDL)                                                                                           \
   launch_attention<T, CT, HDL>(out, part, q, k_pool, v_pool, block_table, bt_width, seq_slot, seq_pos0, seq_qstart,      \
                                seq_qlen, gate, gate_stride, gate_elem, B, nh, nkv, hd, vd, page_size, window, chunk, scale, \
-                               max_qlen, n_splits, st)
+                               slopes, sinks, max_qlen, n_splits, st)
 #define LEB_ATT(T, CT) \
   (vd <= 32 ? LEB_ATT_W(T, CT, 1) : vd <= 64 ? LEB_ATT_W(T, CT, 2) : vd <= 128 ? LEB_ATT_W(T, CT, 4) : LEB_ATT_W(T, CT, 8))
   if (dtype == LEB_F32)
@@ -302,9 +306,9 @@ LEB_API int leb_attention(void* out, float* part, const void* q, const void* k_p
   if (n_splits > 1) {
     dim3 grid(M, nh);
     if (dtype == LEB_F32)
-      attention_merge_kernel<float><<<grid, 64, 0, st>>>((float*)out, part, (const float*)gate, gate_stride, gate_elem, nh, vd, n_splits);
+      attention_merge_kernel<float><<<grid, 64, 0, st>>>((float*)out, part, (const float*)gate, gate_stride, gate_elem, sinks, nh, vd, n_splits);
     else
-      attention_merge_kernel<bf16><<<grid, 64, 0, st>>>((bf16*)out, part, (const bf16*)gate, gate_stride, gate_elem, nh, vd, n_splits);
+      attention_merge_kernel<bf16><<<grid, 64, 0, st>>>((bf16*)out, part, (const bf16*)gate, gate_stride, gate_elem, sinks, nh, vd, n_splits);
     LEB_CHECK_LAUNCH("leb_attention merge");
   }
   return 0;
@@ -312,13 +316,14 @@ LEB_API int leb_attention(void* out, float* part, const void* q, const void* k_p
 
 // Merge of split partial results on its own (for kernels that write the same partial layout).
 LEB_API int leb_attention_merge(void* out, const float* part, int dtype, const void* gate,
-                                int gate_stride, int gate_elem, int M, int nh, int hd, int n_splits, cudaStream_t st) {
+                                int gate_stride, int gate_elem, const float* sinks, int M, int nh, int hd, int n_splits,
+                                cudaStream_t st) {
   if (M <= 0) return 0;
   dim3 grid(M, nh);
   if (dtype == LEB_F32)
-    attention_merge_kernel<float><<<grid, 64, 0, st>>>((float*)out, part, (const float*)gate, gate_stride, gate_elem, nh, hd, n_splits);
+    attention_merge_kernel<float><<<grid, 64, 0, st>>>((float*)out, part, (const float*)gate, gate_stride, gate_elem, sinks, nh, hd, n_splits);
   else if (dtype == LEB_BF16)
-    leb_launch(attention_merge_kernel<bf16>, grid, dim3(64), 0, st, (bf16*)out, part, (const bf16*)gate, gate_stride, gate_elem, nh, hd, n_splits);
+    leb_launch(attention_merge_kernel<bf16>, grid, dim3(64), 0, st, (bf16*)out, part, (const bf16*)gate, gate_stride, gate_elem, sinks, nh, hd, n_splits);
   else
     return leb_fail("leb_attention_merge: unknown dtype %d", dtype);
   LEB_CHECK_LAUNCH("leb_attention_merge");

@@ -22,7 +22,8 @@
 //    ends up with the probabilities of positions 8c..8c+7, exactly the 8 positions of its value
 //    piece, so S feeds the second product without any exchange between lanes.
 // Scores, maxima, exponentials and sums are float; P is rounded to bfloat16 for the second
-// product, as keys and values are.
+// product, as keys and values are.  `slopes` [nh]: slope_h (pos - t) is taken off the score of key t; `sinks` [nh]: one more
+// logit per head in the softmax's denominator (each or null).
 #include "common.cuh"
 
 #define ATD_WARPS 4
@@ -92,10 +93,11 @@ struct AtdPrep {
   bf16* v_store;
   const float* q_norm_w;  // [HD] or null
   const float* k_norm_w;
-  const float* inv_freq;  // [HD / 2]
+  const float* inv_freq;  // [HD / 2], or null: no rotation
   float eps;
   bool neox;              // pairs (i, i + HD/2), else (2i, 2i + 1)
   bool row_norm;          // the root mean square of the whole row of heads, weights over the row ([nh HD], [nkv HD])
+  float temp_coef, temp_every;   // q times query_temperature(position) (common.cuh); coef 0: as it is
 };
 
 // Sum of squares of n bfloat16 numbers by the whole block (n a multiple of 8, src on a 16-byte boundary or read one by
@@ -125,7 +127,7 @@ __device__ __forceinline__ float atd_row_ss(const bf16* __restrict__ src, int n,
 template <int HD>
 __device__ __forceinline__ void atd_prep_head(const bf16* __restrict__ src, const float* __restrict__ nw, float eps,
                                               const float* cs, const float* sn, bf16* dst, int lane, bool neox,
-                                              float row_r) {
+                                              float row_r, float factor = 1.f) {
   constexpr int EPL = HD / 32, NP = EPL / 2;
   float x[EPL];
 #pragma unroll
@@ -157,7 +159,7 @@ __device__ __forceinline__ void atd_prep_head(const bf16* __restrict__ src, cons
     }
   }
 #pragma unroll
-  for (int e = 0; e < EPL; e++) dst[lane + 32 * e] = __float2bfloat16_rn(x[e]);
+  for (int e = 0; e < EPL; e++) dst[lane + 32 * e] = __float2bfloat16_rn(x[e] * factor);
 }
 
 // HD: head_dim, a multiple of 32; S: stages of a warp's ring; WIDE: the softmax weights enter the second product as two
@@ -170,7 +172,8 @@ attention_decode_kernel(bf16* __restrict__ out, float* __restrict__ part, const 
                         const int* __restrict__ seq_slot, const int* __restrict__ seq_pos0,
                         const int* __restrict__ seq_qstart, const bf16* __restrict__ gate,
                         int gate_stride, int gate_elem, int nh, int nkv, int page_size, int window, int chunk,
-                        float scale, int n_splits, AtdPrep prep) {
+                        float scale, const float* __restrict__ slopes, const float* __restrict__ sinks, int n_splits,
+                        AtdPrep prep) {
   constexpr int KB = HD / 32;  // 32-wide pieces of head_dim
   constexpr int NT = HD / 8;   // 8-wide output tiles over head_dim
   constexpr int KBYTES = 32 * HD * 2, STAGE = 2 * KBYTES;   // keys, then values
@@ -279,7 +282,7 @@ attention_decode_kernel(bf16* __restrict__ out, float* __restrict__ part, const 
 #pragma unroll
       for (int p = 0; p < 2 * NP; p++) {
         if (prep.neox && p >= NP) break;
-        const float th = (float)qpos * prep.inv_freq[prep.neox ? lane + 32 * p : (lane + 32 * p) >> 1];
+        const float th = prep.inv_freq ? (float)qpos * prep.inv_freq[prep.neox ? lane + 32 * p : (lane + 32 * p) >> 1] : 0.f;
         cs[p] = cosf(th);
         sn[p] = sinf(th);
       }
@@ -293,7 +296,7 @@ attention_decode_kernel(bf16* __restrict__ out, float* __restrict__ part, const 
       for (int hh = warp; hh < G; hh += ATD_WARPS)
         atd_prep_head<HD>(prep.q_raw + m_row * prep.q_stride + (size_t)(h0 + hh) * HD,
                           prep.q_norm_w && prep.row_norm ? prep.q_norm_w + (size_t)(h0 + hh) * HD : prep.q_norm_w, prep.eps,
-                          cs, sn, q_s + hh * HD, lane, prep.neox, rq);
+                          cs, sn, q_s + hh * HD, lane, prep.neox, rq, query_temperature(qpos, prep.temp_coef, prep.temp_every));
       // the new key and value: the block whose range holds the last block of positions stores them
       // (before it asks for that block's copy, so that the copy finds them in the cache)
       if (prep.k_raw && has_new) {
@@ -330,6 +333,8 @@ attention_decode_kernel(bf16* __restrict__ out, float* __restrict__ part, const 
   // scores are kept times log2(e), so that the exponentials are single exp2 steps
   const float scale2 = scale * 1.4426950408889634f;
   const bool upper = G > 8;   // rows 8..15 of the tiles hold heads at all
+  const float slope2[2] = {slopes && r < G ? slopes[h0 + r] * 1.4426950408889634f : 0.f,
+                           slopes && r + 8 < G ? slopes[h0 + r + 8] * 1.4426950408889634f : 0.f};
   float mx[2] = {ATD_NEG, ATD_NEG}, l[2] = {0.f, 0.f};
   float acc[NT][4];
 #pragma unroll
@@ -383,7 +388,7 @@ attention_decode_kernel(bf16* __restrict__ out, float* __restrict__ part, const 
       for (int e = 0; e < 4; e++) {
         const int kp = key0 + 8 * c + 2 * t + (e & 1);
         const bool valid = kp >= key_lo && kp < kv_len;
-        s[t][e] = valid ? s[t][e] * scale2 : ATD_NEG;
+        s[t][e] = valid ? fmaf(s[t][e], scale2, slope2[e >> 1] * (float)(kp - qpos)) : ATD_NEG;
         tmax[e >> 1] = fmaxf(tmax[e >> 1], s[t][e]);
       }
     float corr[2];
@@ -466,7 +471,8 @@ attention_decode_kernel(bf16* __restrict__ out, float* __restrict__ part, const 
     if (n_splits == 1) {
       float g = 1.f;
       if (gate) g = head_gate(gate, m_row, gate_stride, h, d, HD, gate_elem);
-      out[(m_row * nh + h) * HD + d] = __float2bfloat16_rn(L > 0.f ? a / L * g : 0.f);
+      const float o = sinks ? a * sink_quotient(M * 0.6931471805599453f, L, sinks[h]) : (L > 0.f ? a / L : 0.f);
+      out[(m_row * nh + h) * HD + d] = __float2bfloat16_rn(o * g);
     } else {
       float* pp = part + ((m_row * nh + h) * n_splits + split) * (size_t)(HD + 2);
       if (d == 0) { pp[0] = M * 0.6931471805599453f; pp[1] = L; }   // the merge works with natural exponents
@@ -489,8 +495,8 @@ static int attention_decode_launch(void* out, float* part, const void* q, const 
                                    const void* v_pool, const int* block_table, int bt_width,
                                    const int* seq_slot, const int* seq_pos0, const int* seq_qstart,
                                    const void* gate, int gate_stride, int gate_elem, int B, int nh, int nkv, int hd,
-                                   int page_size, int window, int chunk, int wide, float scale, int n_splits,
-                                   AtdPrep prep, cudaStream_t st) {
+                                   int page_size, int window, int chunk, int wide, float scale, const float* slopes,
+                                   const float* sinks, int n_splits, AtdPrep prep, cudaStream_t st) {
   if (B <= 0) return 0;
   LEB_REQUIRE(leb_attention_decode_supported(nh, nkv, hd, page_size),
               "leb_attention_decode: sizes not taken (heads %d, kv heads %d, head_dim %d, page %d)", nh, nkv, hd, page_size);
@@ -509,7 +515,7 @@ static int attention_decode_launch(void* out, float* part, const void* q, const 
     leb_launch(attention_decode_kernel<HD_, S_, W_>, grid, dim3(32 * ATD_WARPS), smem, st,             \
         (bf16*)out, part, (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, block_table,  \
         bt_width, seq_slot, seq_pos0, seq_qstart, (const bf16*)gate, gate_stride, gate_elem, nh, nkv, \
-        page_size, window, chunk, scale, n_splits, prep);                                         \
+        page_size, window, chunk, scale, slopes, sinks, n_splits, prep);                          \
   }
 #define LEB_ATD(HD_, S_)                    \
   {                                         \
@@ -533,17 +539,17 @@ LEB_API int leb_attention_decode(void* out, float* part, const void* q, const vo
                                  const void* v_pool, const int* block_table, int bt_width,
                                  const int* seq_slot, const int* seq_pos0, const int* seq_qstart,
                                  const void* gate, int gate_stride, int gate_elem, int B, int nh, int nkv, int hd,
-                                 int page_size, int window, int chunk, int wide, float scale, int n_splits,
-                                 cudaStream_t st) {
+                                 int page_size, int window, int chunk, int wide, float scale, const float* slopes,
+                                 const float* sinks, int n_splits, cudaStream_t st) {
   return attention_decode_launch(out, part, q, k_pool, v_pool, block_table, bt_width, seq_slot, seq_pos0, seq_qstart, gate,
-                                 gate_stride, gate_elem, B, nh, nkv, hd, page_size, window, chunk, wide, scale, n_splits,
-                                 AtdPrep{}, st);
+                                 gate_stride, gate_elem, B, nh, nkv, hd, page_size, window, chunk, wide, scale, slopes, sinks,
+                                 n_splits, AtdPrep{}, st);
 }
 
 // Returns 1 when the kernel can norm, rotate and store the step's q, k and v itself: head size 64 or
-// 128 and a rotation over the whole head (split-half or adjacent pairs).
+// 128 and a rotation over the whole head (split-half or adjacent pairs) or none (rope_dim 0).
 LEB_API int leb_attention_decode_prep_supported(int nh, int nkv, int hd, int page_size, int rope_dim, int neox) {
-  return leb_attention_decode_supported(nh, nkv, hd, page_size) && (hd == 64 || hd == 128) && rope_dim == hd;
+  return leb_attention_decode_supported(nh, nkv, hd, page_size) && (hd == 64 || hd == 128) && (rope_dim == hd || rope_dim == 0);
 }
 
 // The same with the step's q, k and v as the projection left them (rows of q_stride / kv_stride
@@ -556,24 +562,26 @@ LEB_API int leb_attention_decode_prep(void* out, float* part, const void* q_raw,
                                       const int* seq_pos0, const int* seq_qstart, const float* q_norm_w,
                                       const float* k_norm_w, float eps, const float* inv_freq, int rope_dim,
                                       int neox, int row_norm, const void* gate, int gate_stride, int gate_elem, int B, int nh, int nkv,
-                                      int hd, int page_size, int window, int chunk, int wide, float scale, int n_splits,
-                                      cudaStream_t st) {
+                                      int hd, int page_size, int window, int chunk, int wide, float scale, const float* slopes,
+                                      const float* sinks, float temp_coef, float temp_every, int n_splits, cudaStream_t st) {
   LEB_REQUIRE(leb_attention_decode_prep_supported(nh, nkv, hd, page_size, rope_dim, neox),
               "leb_attention_decode_prep: sizes not taken (head_dim %d, rope_dim %d, split-half %d)", hd, rope_dim, neox);
-  LEB_REQUIRE(q_raw && inv_freq, "leb_attention_decode_prep: q and the frequencies are required");
+  LEB_REQUIRE(q_raw && (inv_freq || rope_dim == 0), "leb_attention_decode_prep: q and the frequencies are required");
+  LEB_REQUIRE(temp_coef == 0.f || temp_every > 0.f, "leb_attention_decode_prep: a temperature that rises every %g positions", temp_every);
   LEB_REQUIRE((k_raw == nullptr) == (v_raw == nullptr), "leb_attention_decode_prep: keys and values come together");
   AtdPrep prep{(const bf16*)q_raw, (const bf16*)k_raw, (const bf16*)v_raw, q_stride, kv_stride, (bf16*)k_pool,
-               (bf16*)v_pool, q_norm_w, k_norm_w, inv_freq, eps, neox != 0, row_norm != 0};
+               (bf16*)v_pool, q_norm_w, k_norm_w, rope_dim ? inv_freq : nullptr, eps, neox != 0, row_norm != 0, temp_coef,
+               temp_every};
   return attention_decode_launch(out, part, nullptr, k_pool, v_pool, block_table, bt_width, seq_slot, seq_pos0, seq_qstart,
-                                 gate, gate_stride, gate_elem, B, nh, nkv, hd, page_size, window, chunk, wide, scale, n_splits,
-                                 prep, st);
+                                 gate, gate_stride, gate_elem, B, nh, nkv, hd, page_size, window, chunk, wide, scale, slopes, sinks,
+                                 n_splits, prep, st);
 }
 
 // ---- the same step for callers that cannot allocate (see leb_no_alloc.h) ---------------------------
 #include "leb_no_alloc.h"
 
 extern "C" int leb_attention_merge(void* out, const float* part, int dtype, const void* gate, int gate_stride,
-                                   int gate_elem, int M, int nh, int hd, int n_splits, cudaStream_t st);
+                                   int gate_elem, const float* sinks, int M, int nh, int hd, int n_splits, cudaStream_t st);
 
 // The split partial results of leb_attention_decode_static.  In host code this name is only a
 // handle for cudaGetSymbolAddress, not a device address.
@@ -610,9 +618,10 @@ LEB_API int leb_attention_decode_static(void* out, const void* q, const void* k_
     scratch = g_static_scratch_ptr[dev];
   }
   int rc = leb_attention_decode(out, scratch, q, k_pool, v_pool, block_table, bt_width, seq_slot, seq_pos0,
-                                seq_qstart, gate, gate_stride, 0, B, nh, nkv, hd, page_size, window, 0, 0, scale, n_splits, st);
+                                seq_qstart, gate, gate_stride, 0, B, nh, nkv, hd, page_size, window, 0, 0, scale, nullptr, nullptr,
+                                n_splits, st);
   if (rc) return rc;
   if (n_splits > 1)
-    return leb_attention_merge(out, scratch, LEB_BF16, gate, gate_stride, 0, B, nh, hd, n_splits, st);
+    return leb_attention_merge(out, scratch, LEB_BF16, gate, gate_stride, 0, nullptr, B, nh, hd, n_splits, st);
   return 0;
 }

@@ -14,7 +14,8 @@
 // the window, with a running (max, sum, acc) per row; the fragments of the next block are
 // loaded while the current one is multiplied, exponentials are 2^x on scores pre-multiplied by
 // log2(e), and blocks wholly below the diagonal skip the mask.  Keys and values come from the cache
-// only, which already holds this step's rows.
+// only, which already holds this step's rows.  `slopes` [nh]: slope_h (pos - t) is taken off the score of key t; `sinks`
+// [nh]: one more logit per head in the softmax's denominator (each or null).
 #include "common.cuh"
 
 #define ATP_WARPS 4
@@ -57,7 +58,8 @@ attention_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ q,
                          const int* __restrict__ seq_slot, const int* __restrict__ seq_pos0,
                          const int* __restrict__ seq_qstart, const int* __restrict__ seq_qlen,
                          const bf16* __restrict__ gate, int gate_stride, int gate_elem, int nh, int nkv,
-                         int page_size, int window, int chunk, float scale, int QT) {
+                         int page_size, int window, int chunk, float scale, const float* __restrict__ slopes,
+                         const float* __restrict__ sinks, int QT) {
   constexpr int KB = HD / 32, NT = HD / 8;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int r = lane >> 2, c = lane & 3;
@@ -139,6 +141,11 @@ attention_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ q,
   const int* table = block_table + (size_t)b * bt_width;
   // Scores are kept in base 2: s2 = (q.k) * scale * log2(e), p = 2^(s2 - max2) = e^(s - max).
   const float scale2 = scale * 1.4426950408889634f;
+  float slope2[MT][2];
+#pragma unroll
+  for (int mt = 0; mt < MT; mt++)
+#pragma unroll
+    for (int hh = 0; hh < 2; hh++) slope2[mt][hh] = slopes ? slopes[h0 + rhead[mt][hh]] * 1.4426950408889634f : 0.f;
   // the lowest query position among this lane's rows: blocks wholly at or below it need no mask
   int qmin = 0x7fffffff;
 #pragma unroll
@@ -203,7 +210,16 @@ attention_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ q,
             const int kp = key0 + 8 * c + 2 * t + (e & 1);
             const int qp = pos0 + rpos[mt][hh];
             const bool valid = kp <= qp && kp >= rlo[hh];
-            s[t][e] = valid ? s[t][e] * scale2 : ATP_NEG;
+            s[t][e] = valid ? fmaf(s[t][e], scale2, slope2[mt][hh] * (float)(kp - qp)) : ATP_NEG;
+            tmax[hh] = fmaxf(tmax[hh], s[t][e]);
+          }
+      } else if (slopes) {
+#pragma unroll
+        for (int t = 0; t < 4; t++)
+#pragma unroll
+          for (int e = 0; e < 4; e++) {
+            const int hh = e >> 1, kp = key0 + 8 * c + 2 * t + (e & 1);
+            s[t][e] = fmaf(s[t][e], scale2, slope2[mt][hh] * (float)(kp - pos0 - rpos[mt][hh]));
             tmax[hh] = fmaxf(tmax[hh], s[t][e]);
           }
       } else {
@@ -293,7 +309,8 @@ attention_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ q,
       const size_t m = q0 + rpos[mt][hh];
       const int h = h0 + rhead[mt][hh];
       const float g = gate && !gate_elem ? head_gate(gate, m, gate_stride, h, 0, HD, 0) : 1.f;
-      const float inv = l[mt][hh] > 0.f ? g / l[mt][hh] : 0.f;
+      const float inv = sinks ? g * sink_quotient(mx[mt][hh] * 0.6931471805599453f, l[mt][hh], sinks[h])
+                              : (l[mt][hh] > 0.f ? g / l[mt][hh] : 0.f);
       bf16* o = out + (m * nh + h) * HD;
 #pragma unroll
       for (int n = 0; n < NT; n++) {
@@ -318,8 +335,8 @@ LEB_API int leb_attention_prefill(void* out, const void* q, const void* k_pool, 
                                   const int* block_table, int bt_width, const int* seq_slot,
                                   const int* seq_pos0, const int* seq_qstart, const int* seq_qlen,
                                   const void* gate, int gate_stride, int gate_elem, int B, int nh, int nkv, int hd,
-                                  int page_size, int window, int chunk, int wide, float scale, int max_qlen,
-                                  cudaStream_t st) {
+                                  int page_size, int window, int chunk, int wide, float scale, const float* slopes,
+                                  const float* sinks, int max_qlen, cudaStream_t st) {
   if (B <= 0 || max_qlen <= 0) return 0;
   LEB_REQUIRE(leb_attention_prefill_supported(nh, nkv, hd, page_size),
               "leb_attention_prefill: sizes not taken (heads %d, kv heads %d, head_dim %d, page %d)", nh, nkv, hd, page_size);
@@ -334,7 +351,7 @@ LEB_API int leb_attention_prefill(void* out, const void* q, const void* k_pool, 
   attention_prefill_kernel<HD_, MT_, W_><<<grid, 32 * ATP_WARPS, 0, st>>>(                               \
       (bf16*)out, (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, block_table, bt_width,   \
       seq_slot, seq_pos0, seq_qstart, seq_qlen, (const bf16*)gate, gate_stride, gate_elem, nh, nkv,  \
-      page_size, window, chunk, scale, QT)
+      page_size, window, chunk, scale, slopes, sinks, QT)
 #define LEB_ATP(HD_, MT_)                \
   if (wide) LEB_ATP_W(HD_, MT_, true);   \
   else LEB_ATP_W(HD_, MT_, false)

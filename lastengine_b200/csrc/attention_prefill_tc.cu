@@ -91,7 +91,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             const int* __restrict__ seq_pos0, const int* __restrict__ seq_qstart,
                             const int* __restrict__ seq_qlen, const bf16* __restrict__ gate, int gate_stride, int gate_elem,
                             int nh, int nkv, int window, int chunk, int pool, float scale, const float* __restrict__ head_scale,
-                            const float* __restrict__ freq_v, int* __restrict__ status) {
+                            const float* __restrict__ freq_v, const float* __restrict__ slopes,
+                            const float* __restrict__ sinks, int* __restrict__ status) {
   constexpr int HD = 64, PAGE = 64, TP = 128 / GS, NS = ATC_STAGES;
   constexpr int Q_BYTES = 128 * HD * 2, KV_BYTES = PAGE * HD * 2, V_BYTES = VD * PAGE * 2;
   extern __shared__ uint8_t atc_raw[];
@@ -238,6 +239,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const uint32_t lane_base = (uint32_t)(warp * 32) << 16;
     const float scale2 = (head_scale ? head_scale[h0 + g] : scale) * 1.4426950408889634f;
     const int nb_row = POOLED ? atc_blocks_seen(qpos, window, pool) : 0;
+    // With slopes the scores are finished (scaled, less slope (qpos - key), times log2 e) as they come out of tensor memory,
+    // and what follows multiplies them by one.
+    const bool sloped = !POOLED && slopes != nullptr;
+    const float slope2 = sloped ? slopes[h0 + g] * 1.4426950408889634f : 0.f;
+    const float scale_after = sloped ? 1.f : scale2;
     float m_used = ATC_NEG, l = 0.f;
     for (int i = 0; i < n_it && ok; i++) {
       const bool pooled = POOLED && i < npp;
@@ -248,6 +254,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       tmem_ld32(t_s0 + 64 * bsel + lane_base, v);
       tmem_ld32(t_s0 + 64 * bsel + lane_base + 32, v + 32);
       tmem_ld_wait();
+      if (sloped) {
+        const float at0 = slope2 * (float)(key0 - qpos);
+#pragma unroll
+        for (int c = 0; c < PAGE; c++)
+          v[c] = __float_as_uint(fmaf(__uint_as_float(v[c]), scale2, fmaf(slope2, (float)c, at0)));
+      }
       // columns [c_lo, c_hi] of this page are keys this row may see
       const int c_lo = pooled ? 0 : max(0, key_lo_row - key0);
       const int c_hi = row_valid ? min(PAGE - 1, (pooled ? nb_row - 1 : qpos) - key0) : -1;
@@ -266,7 +278,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       }
       const float rmax = fmaxf(fmaxf(rm[0], rm[1]), fmaxf(rm[2], rm[3]));
       // maxima are kept times scale * log2(e); a row with no key in this page keeps what it had
-      const float m_new = rmax > 0.5f * ATC_NEG ? fmaxf(m_used, rmax * scale2) : m_used;
+      const float m_new = rmax > 0.5f * ATC_NEG ? fmaxf(m_used, rmax * scale_after) : m_used;
       bool move = false;
       if (l == 0.f) m_used = m_new;                 // nothing accumulated for this row yet: O's row is zero
       else if (m_new > m_used + 8.f) move = true;   // the reference maximum has to follow
@@ -294,7 +306,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
       for (int c = 0; c < PAGE; c += 2) {
         // a masked score is -1e30: 2^(that * scale - m_ref) is exactly zero
-        const float p0 = ex2(fmaf(__uint_as_float(v[c]), scale2, -m_ref)), p1 = ex2(fmaf(__uint_as_float(v[c + 1]), scale2, -m_ref));
+        const float p0 = ex2(fmaf(__uint_as_float(v[c]), scale_after, -m_ref)), p1 = ex2(fmaf(__uint_as_float(v[c + 1]), scale_after, -m_ref));
         ps[(c >> 1) & 3] += p0 + p1;
         __nv_bfloat162 pp = __floats2bfloat162_rn(p0, p1);
         pk[c >> 1] = *reinterpret_cast<uint32_t*>(&pp);
@@ -338,6 +350,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     if (ok) {
       tc_fence_after();
       float inv = l > 0.f ? 1.0f / l : 0.f;
+      if (!POOLED && sinks) inv = sink_quotient(m_used * 0.6931471805599453f, l, sinks[h0 + g]);
       if (gate && !gate_elem && row_valid) inv *= head_gate(gate, m_base + pi, gate_stride, h0 + g, 0, VD, 0);
       uint4* orow = reinterpret_cast<uint4*>(out + ((m_base + pi) * nh + h0 + g) * VD);
       uint32_t o[VD];
@@ -408,7 +421,8 @@ static int launch_attention_prefill_tc(const char* who, void* out, const void* q
                                        int pt_width, const int* seq_slot, const int* seq_pos0, const int* seq_qstart,
                                        const int* seq_qlen, const void* gate, int gate_stride, int gate_elem, int B, int nh, int nkv,
                                        int hd, int page_size, int window, int chunk, int pool, float scale, const float* head_scale,
-                                       const float* freq_v, int max_qlen, int* status, cudaStream_t st) {
+                                       const float* freq_v, const float* slopes, const float* sinks, int max_qlen, int* status,
+                                       cudaStream_t st) {
   if (B <= 0 || max_qlen <= 0 || M <= 0) return 0;
   LEB_REQUIRE(leb_attention_prefill_tc_supported(nh, nkv, hd, page_size),
               "%s: sizes not taken (heads %d, kv heads %d, head_dim %d, page %d)", who, nh, nkv, hd, page_size);
@@ -443,7 +457,8 @@ static int launch_attention_prefill_tc(const char* who, void* out, const void* q
     }                                                                                                             \
     leb_launch(attention_prefill_tc_kernel<GS_, POOLED, WIDE, VD>, grid, dim3(ATC_THREADS), smem, st,                       \
         mq, mk, mv, mpk, mpv, (bf16*)out, block_table, bt_width, pool_table, pt_width, seq_slot, seq_pos0, seq_qstart, \
-        seq_qlen, (const bf16*)gate, gate_stride, gate_elem, nh, nkv, window, chunk, pooled ? pool : 0, scale, head_scale, freq_v, status); \
+        seq_qlen, (const bf16*)gate, gate_stride, gate_elem, nh, nkv, window, chunk, pooled ? pool : 0, scale, head_scale, freq_v, slopes, \
+        sinks, status); \
   }
   switch (G) {
     case 1: LEB_ATC(1); break;
@@ -459,16 +474,17 @@ static int launch_attention_prefill_tc(const char* who, void* out, const void* q
 // Prompt attention of the step's rows over the paged cache (which already holds their keys and
 // values).  q: [M, nh*64] with row stride q_stride; k_pool [n_pages][nkv][64][64], v_pool
 // [n_pages][nkv][64 dims][64 positions]; out [M, nh*64].  status: device int, set non-zero by a
-// block whose bounded wait gave up.
+// block whose bounded wait gave up.  slopes, sinks [nh] or null: slope_h (pos - t) taken off the score of key t, and one more
+// logit per head in the softmax's denominator.
 LEB_API int leb_attention_prefill_tc(void* out, const void* q, int q_stride, int M, const void* k_pool,
                                      const void* v_pool, int n_pages, const int* block_table, int bt_width,
                                      const int* seq_slot, const int* seq_pos0, const int* seq_qstart,
                                      const int* seq_qlen, const void* gate, int gate_stride, int gate_elem, int B, int nh,
                                      int nkv, int hd, int page_size, int window, int chunk, int wide, float scale,
-                                     int max_qlen, int* status, cudaStream_t st) {
+                                     const float* slopes, const float* sinks, int max_qlen, int* status, cudaStream_t st) {
 #define LEB_ATC_ARGS "leb_attention_prefill_tc", out, q, q_stride, M, k_pool, v_pool, n_pages, block_table, bt_width, nullptr, \
                      nullptr, 0, nullptr, 0, seq_slot, seq_pos0, seq_qstart, seq_qlen, gate, gate_stride, gate_elem, B, nh, nkv, \
-                     hd, page_size, window, chunk, 0, scale, nullptr, nullptr, max_qlen, status, st
+                     hd, page_size, window, chunk, 0, scale, nullptr, nullptr, slopes, sinks, max_qlen, status, st
   return wide ? launch_attention_prefill_tc<false, true, 64>(LEB_ATC_ARGS) : launch_attention_prefill_tc<false, false, 64>(LEB_ATC_ARGS);
 #undef LEB_ATC_ARGS
 }
@@ -487,7 +503,7 @@ LEB_API int leb_attention_pooled_tc(void* out, const void* q, int q_stride, int 
   LEB_REQUIRE(vd == 64 || vd == 32, "leb_attention_pooled_tc: value heads of %d numbers (64 or 32)", vd);
 #define LEB_APT_ARGS "leb_attention_pooled_tc", out, q, q_stride, M, k_pool, v_pool, n_pages, block_table, bt_width, pk_pool, \
                      pv_pool, n_pooled_pages, pool_table, pt_width, seq_slot, seq_pos0, seq_qstart, seq_qlen, nullptr, 0, 0, B, nh, \
-                     nkv, hd, page_size, window, 0, pool, 1.0f, head_scale, freq_v, max_qlen, status, st
+                     nkv, hd, page_size, window, 0, pool, 1.0f, head_scale, freq_v, nullptr, nullptr, max_qlen, status, st
   const int rc = vd == 64 ? launch_attention_prefill_tc<true, true, 64>(LEB_APT_ARGS) : launch_attention_prefill_tc<true, true, 32>(LEB_APT_ARGS);
 #undef LEB_APT_ARGS
   return rc;

@@ -127,6 +127,20 @@ template <typename T> __device__ __forceinline__ T from_f32(float v);
 template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <> __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat16_rn(v); }
 
+// Four neighbouring numbers as floats (16 bytes of float, 8 of bfloat16; aligned to that).
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const bf16* p) {
+  const uint2 r = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x));
+  const float2 c = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+  return make_float4(a.x, a.y, c.x, c.y);
+}
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(bf16* p, float4 v) {
+  __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -168,6 +182,18 @@ template <typename T>
 __device__ __forceinline__ float head_gate(const T* gate, size_t row, int stride, int h, int d, int width, int elem) {
   const float z = to_f32(gate[row * stride + (elem ? h * width + d : h)]);
   return 1.0f / (1.0f + expf(-z));
+}
+
+// The factor on a query at position p: 1 + coef ln(floor((p + 1) / every) + 1).
+__device__ __forceinline__ float query_temperature(int p, float coef, float every) {
+  return coef != 0.f ? 1.0f + coef * logf(floorf((float)(p + 1) / every) + 1.0f) : 1.0f;
+}
+
+// A softmax row summed as (m, l) = (reference maximum, sum of e^(s - m)) takes one more logit `sink` into its denominator
+// (a logit without a key or a value): returns what the row's weighted sum of values is multiplied by.
+__device__ __forceinline__ float sink_quotient(float m, float l, float sink) {
+  const float top = fmaxf(m, sink), f = expf(m - top);
+  return f / (l * f + expf(sink - top));
 }
 
 static inline int ceil_div(int a, int b) { return (a + b - 1) / b; }

@@ -180,16 +180,29 @@ LEB_API int leb_swiglu(void* a, int out_dtype, const void* gu, int in_dtype, int
 }
 
 // ---------------------------------------------------------------------------------------------
-// out[p, :] = in[rows[p] / div, :]   (expert-sorted copies of token rows; div = experts per token)
+// out[p, :] = in[rows[p] / div, :]   (expert-sorted copies of token rows; div = experts per token), times w[rows[p]] where
+// weights are given (experts that are weighted at their input)
 template <typename T>
 __global__ void gather_rows_kernel(T* __restrict__ out, const T* __restrict__ in,
-                                   const int* __restrict__ rows, int div, int D) {
+                                   const int* __restrict__ rows, const float* __restrict__ w, int div, int D) {
   pdl_trigger();   // the kernel after this one may start and wait (see common.cuh)
   pdl_wait();
   int p = blockIdx.x;
   int src = rows[p] / div;
   const T* a = in + (size_t)src * D;
   T* o = out + (size_t)p * D;
+  if (w) {
+    const float f = w[rows[p]];
+    if (D % 4 == 0 && (((uintptr_t)a | (uintptr_t)o) & 15) == 0) {
+      for (int i = threadIdx.x * 4; i < D; i += blockDim.x * 4) {
+        const float4 v = load4(a + i);
+        store4(o + i, make_float4(v.x * f, v.y * f, v.z * f, v.w * f));
+      }
+    } else {
+      for (int i = threadIdx.x; i < D; i += blockDim.x) o[i] = from_f32<T>(to_f32(a[i]) * f);
+    }
+    return;
+  }
   if ((((uintptr_t)a | (uintptr_t)o) & 15) == 0 && (D * sizeof(T)) % 16 == 0) {
     const int n = D * (int)sizeof(T) / 16;
     for (int i = threadIdx.x; i < n; i += blockDim.x) reinterpret_cast<uint4*>(o)[i] = reinterpret_cast<const uint4*>(a)[i];
@@ -198,14 +211,14 @@ __global__ void gather_rows_kernel(T* __restrict__ out, const T* __restrict__ in
   }
 }
 
-LEB_API int leb_gather_rows(void* out, const void* in, int dtype, const int* rows, int div, int P,
+LEB_API int leb_gather_rows(void* out, const void* in, int dtype, const int* rows, const float* w, int div, int P,
                             int D, cudaStream_t st) {
   if (P <= 0) return 0;
   LEB_REQUIRE(div >= 1, "leb_gather_rows: div must be positive");
   if (dtype == LEB_F32)
-    leb_launch(gather_rows_kernel<float>, dim3(P), dim3(128), 0, st, (float*)out, (const float*)in, rows, div, D);
+    leb_launch(gather_rows_kernel<float>, dim3(P), dim3(128), 0, st, (float*)out, (const float*)in, rows, w, div, D);
   else if (dtype == LEB_BF16)
-    leb_launch(gather_rows_kernel<bf16>, dim3(P), dim3(128), 0, st, (bf16*)out, (const bf16*)in, rows, div, D);
+    leb_launch(gather_rows_kernel<bf16>, dim3(P), dim3(128), 0, st, (bf16*)out, (const bf16*)in, rows, w, div, D);
   else
     return leb_fail("leb_gather_rows: unknown dtype %d", dtype);
   LEB_CHECK_LAUNCH("leb_gather_rows");
@@ -306,18 +319,6 @@ __global__ void __launch_bounds__(256) gated_residual_kernel(
 // The same with 16-byte accesses for rows of up to CH * 512 * 4 elements: a thread keeps its pieces of the
 // new row in registers between the sum and the norm, so a row is read once and a decode step's few
 // rows are not a chain of dependent loads.
-__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 load4(const bf16* p) {
-  const uint2 r = *reinterpret_cast<const uint2*>(p);
-  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x));
-  const float2 c = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
-  return make_float4(a.x, a.y, c.x, c.y);
-}
-__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-__device__ __forceinline__ void store4(bf16* p, float4 v) {
-  __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
-  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
-}
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 
 template <typename TZ, typename TH, int CH>

@@ -460,7 +460,7 @@ LEB_API int leb_moe_align(int* offsets, int* sorted_pair, int* pair_row, const i
   return 0;
 }
 
-// x[m, :] (+)= sum_j w[m, j] * ys[pair_row[m*k + j], :]   in the order j = 0..k-1, float.
+// x[m, :] (+)= sum_j w[m, j] * ys[pair_row[m*k + j], :]   in the order j = 0..k-1, float (topk_w null: weights of one).
 // A thread owns VEC consecutive columns of one token; the token's k rows and weights are read
 // first and then all k pieces of ys are asked for before any is used, so the kernel costs two
 // trips to memory whatever k is.
@@ -478,7 +478,7 @@ moe_combine_kernel(float* __restrict__ x, const float* __restrict__ ys, const in
 #pragma unroll
   for (int j = 0; j < KMAX; j++) {
     row[j] = j < k ? pair_row[m * k + j] : 0;
-    w[j] = j < k ? topk_w[m * k + j] : 0.f;
+    w[j] = j < k ? (topk_w ? topk_w[m * k + j] : 1.f) : 0.f;
   }
   float* o = x + m * D + i;
   if (VEC == 4) {

@@ -10,8 +10,9 @@
 //     u  = w_t (v_t - S^T k_t)        delta form (the write replaces what the key already reads)
 //     S <- S + k_t u^T
 //     o_t = S^T q_t (+ skip_h v_t)
-// in this order: the read-out sees the row's own write.  Several heads may share one key/query head
-// (head h reads key head h / (H / Gk)).
+// in this order: the read-out sees the row's own write.  The bonus form reads first: with a weight b per key channel
+//     o_t = (S + diag(b) k_t u^T)^T q_t,  then  S <- diag(a_t) S + k_t u^T,  u = w_t v_t
+// Several heads may share one key/query head (head h reads key head h / (H / Gk)).
 //
 // The columns of S never mix, so eight lanes own one column and walk the sequence's rows of the step in
 // order; k, q, a, v and w of the rows come through shared memory.  The state is kept [slot][head][column][row] so that a warp's column is
@@ -50,13 +51,15 @@ __device__ __forceinline__ float sum8(float x) {      // over the eight lanes of
 // come in through shared memory, REC_ROWS rows at a time in two buffers: the copies of the next rows are in
 // flight while these are computed, and the walk over the rows never waits on global memory.  A staged row is
 // padded with zeros to 32 NV numbers, so the walk has no bounds to test.
-template <int NV, bool DELTA, bool ROW_DECAY>
+constexpr int REC_PLAIN = 0, REC_DELTA = 1, REC_BONUS = 2;
+template <int NV, int FORM, bool ROW_DECAY>
 __global__ void __launch_bounds__(32 * REC_WARPS)
 gated_recurrence_kernel(float* __restrict__ out, int ldo, const float* __restrict__ k, const float* __restrict__ q, int ldk,
                         const float* __restrict__ v, int ldv, const float* __restrict__ wr, int ldw,
-                        const float* __restrict__ decay, int ldd, const float* __restrict__ skip,
+                        const float* __restrict__ decay, int ldd, const float* __restrict__ skip, const float* __restrict__ bonus,
                         float* __restrict__ state, const int* __restrict__ seq_slot, const int* __restrict__ seq_qstart,
                         const int* __restrict__ seq_qlen, int H, int Gk, int d, int e, int ev, int wide) {
+  constexpr bool DELTA = FORM == REC_DELTA, BONUS = FORM == REC_BONUS;
   extern __shared__ __align__(16) float rec_sm[];
   constexpr int DP = 32 * NV;                   // a staged row of k, q or the decay
   constexpr int DA = ROW_DECAY ? DP : 1;
@@ -80,6 +83,14 @@ gated_recurrence_kernel(float* __restrict__ out, int ldo, const float* __restric
       const int r = 4 * (j8 + 8 * i) + x;
       s[4 * i + x] = (sp && r < d) ? sp[r] : 0.f;
     }
+  float ub[BONUS ? 4 * NV : 1];
+  if (BONUS) {
+#pragma unroll
+    for (int i = 0; i < 4 * NV; i++) {
+      const int r = 4 * (j8 + 8 * (i / 4)) + (i & 3);
+      ub[i] = r < d ? bonus[(size_t)h * d + r] : 0.f;
+    }
+  }
   const float sk = skip ? skip[h] : 0.f;
   // one buffer: k [REC_ROWS][DP] | q [REC_ROWS][DP] | v [REC_ROWS][REC_COLS] | decay [REC_ROWS][DA] | write [REC_ROWS]
   for (int idx = threadIdx.x; idx < 2 * REC_ROWS * (DP - d); idx += blockDim.x) {      // the padding, once
@@ -120,7 +131,8 @@ gated_recurrence_kernel(float* __restrict__ out, int ldo, const float* __restric
         if (c0 + jj < ev) rec_copy4(vs + t * REC_COLS + jj, v + (m + t) * ldv + h * ev + c0 + jj);
         else if (c0 + jj < e) vs[t * REC_COLS + jj] = 1.0f;      // columns past the values' width hold a constant one
       } else if (jj == REC_COLS) {
-        rec_copy4(ws + t, wr + (m + t) * ldw + h);
+        if (wr) rec_copy4(ws + t, wr + (m + t) * ldw + h);
+        else ws[t] = 1.0f;
       } else if (!ROW_DECAY) {
         rec_copy4(as + t, decay + (m + t) * ldd + h);
       }
@@ -165,6 +177,19 @@ gated_recurrence_kernel(float* __restrict__ out, int ldo, const float* __restric
           qv[i] = q4[j8 + 8 * i];
           float4 av = make_float4(a1, a1, a1, a1);
           if (ROW_DECAY) av = a4[j8 + 8 * i];
+          if (BONUS) {       // the read-out of the state before the row and of the row's weighted write, then both steps of the state
+            const float u = wc * vc;
+            const float x0 = kv[i].x * u, x1 = kv[i].y * u, x2 = kv[i].z * u, x3 = kv[i].w * u;
+            dp[0] = fmaf(fmaf(ub[4 * i + 0], x0, s[4 * i + 0]), qv[i].x, dp[0]);
+            dp[1] = fmaf(fmaf(ub[4 * i + 1], x1, s[4 * i + 1]), qv[i].y, dp[1]);
+            dp[2] = fmaf(fmaf(ub[4 * i + 2], x2, s[4 * i + 2]), qv[i].z, dp[2]);
+            dp[3] = fmaf(fmaf(ub[4 * i + 3], x3, s[4 * i + 3]), qv[i].w, dp[3]);
+            s[4 * i + 0] = fmaf(s[4 * i + 0], av.x, x0);
+            s[4 * i + 1] = fmaf(s[4 * i + 1], av.y, x1);
+            s[4 * i + 2] = fmaf(s[4 * i + 2], av.z, x2);
+            s[4 * i + 3] = fmaf(s[4 * i + 3], av.w, x3);
+            continue;
+          }
           s[4 * i + 0] *= av.x;
           s[4 * i + 1] *= av.y;
           s[4 * i + 2] *= av.z;
@@ -175,6 +200,10 @@ gated_recurrence_kernel(float* __restrict__ out, int ldo, const float* __restric
             dp[2] = fmaf(s[4 * i + 2], kv[i].z, dp[2]);
             dp[3] = fmaf(s[4 * i + 3], kv[i].w, dp[3]);
           }
+        }
+        if (BONUS) {
+          o_part[t] = (dp[0] + dp[1]) + (dp[2] + dp[3]);
+          continue;
         }
         float u = wc * vc;
         if (DELTA) u = wc * (vc - sum8((dp[0] + dp[1]) + (dp[2] + dp[3])));
@@ -217,16 +246,19 @@ gated_recurrence_kernel(float* __restrict__ out, int ldo, const float* __restric
 // row_decay, else [M, H]; skip [H] or null; state [slots][H][e][d].  seq_qlen null: one row per sequence.
 // ev < e: a head's value has ev numbers and the state's columns ev .. e-1 are written with the value one, so
 // that column accumulates the keys alone (decayed and weighted like the rest) and its read-out is the
-// product of that sum with the query: the normaliser of a memory whose result is divided by it.
+// product of that sum with the query: the normaliser of a memory whose result is divided by it.  write null: 1.
+// form: 0 plain, 1 delta, 2 bonus (bonus [H*d], a decay per key channel).
 LEB_API int leb_gated_recurrence(float* out, int ldo, const float* k, const float* q, int ldk, const float* v, int ldv,
-                                 const float* write, int ldw, const float* decay, int ldd, int row_decay, int delta,
-                                 const float* skip, float* state, const int* seq_slot, const int* seq_qstart,
+                                 const float* write, int ldw, const float* decay, int ldd, int row_decay, int form,
+                                 const float* skip, const float* bonus, float* state, const int* seq_slot, const int* seq_qstart,
                                  const int* seq_qlen, int B, int H, int Gk, int d, int e, int ev, cudaStream_t st) {
   if (B <= 0) return 0;
   LEB_REQUIRE(ev >= 0 && ev <= e, "leb_gated_recurrence: %d value columns for a state of %d", ev, e);
   LEB_REQUIRE(H >= 1 && Gk >= 1 && H % Gk == 0, "leb_gated_recurrence: %d heads do not divide into %d key heads", H, Gk);
   LEB_REQUIRE(d >= 1 && d <= 256 && e >= 1, "leb_gated_recurrence: a state of %d x %d (rows 1..256)", d, e);
   LEB_REQUIRE(H <= 65535 && B <= 65535, "leb_gated_recurrence: step too large");
+  LEB_REQUIRE(form >= 0 && form <= 2 && (form != 2 || (bonus && row_decay)),
+              "leb_gated_recurrence: form %d (0 plain, 1 delta, 2 bonus: with its weights and a decay per key channel)", form);
   const dim3 grid(ceil_div(e, REC_COLS), H, B), block(32 * REC_WARPS);
   const int nv = d <= 32 ? 1 : d <= 64 ? 2 : d <= 128 ? 4 : 8, dp = 32 * nv;
   const size_t smem = (size_t)2 * (REC_ROWS * (2 * dp + REC_COLS) + ((REC_ROWS * ((row_decay ? dp : 1) + 1) + 3) & ~3)) * sizeof(float);
@@ -243,14 +275,15 @@ LEB_API int leb_gated_recurrence(float* out, int ldo, const float* k, const floa
       set = smem;                                                                                                        \
     }                                                                                                                    \
     leb_launch(gated_recurrence_kernel<NV_, D_, R_>, grid, block, smem, st, out, ldo, k, q, ldk, v, ldv, write, ldw, decay, \
-               ldd, skip, state, seq_slot, seq_qstart, seq_qlen, H, Gk, d, e, ev, wide);                                     \
+               ldd, skip, bonus, state, seq_slot, seq_qstart, seq_qlen, H, Gk, d, e, ev, wide);                              \
   }
 #define LEB_REC2(NV_)                                     \
   {                                                       \
-    if (delta && row_decay) LEB_REC3(NV_, true, true)     \
-    else if (delta) LEB_REC3(NV_, true, false)            \
-    else if (row_decay) LEB_REC3(NV_, false, true)        \
-    else LEB_REC3(NV_, false, false)                      \
+    if (form == 2) LEB_REC3(NV_, REC_BONUS, true)         \
+    else if (form == 1 && row_decay) LEB_REC3(NV_, REC_DELTA, true) \
+    else if (form == 1) LEB_REC3(NV_, REC_DELTA, false)   \
+    else if (row_decay) LEB_REC3(NV_, REC_PLAIN, true)    \
+    else LEB_REC3(NV_, REC_PLAIN, false)                  \
   }
   if (nv == 1) LEB_REC2(1)
   else if (nv == 2) LEB_REC2(2)
@@ -360,14 +393,14 @@ LEB_API int leb_ssm_prep(float* xbc, int ldx, int C, const float* conv_bias, flo
 // A recurrent mixer's result on its way to the output projection: groups of `gs` neighbouring numbers of a
 // row are divided by their root mean square (eps inside the root) and multiplied by a weight
 // (w[j % wlen]: one weight for every group, or one per column), and the row is gated by a second
-// row z: sigmoid(z) after the norm (gate_first = 0), or silu(z) before it (gate_first = 1).
+// row z: sigmoid(z) after the norm (gate = 0), silu(z) before it (1), or silu(z) after it (2).
 // y, z float; out in the activation type.  A team takes a group: a warp (four groups a block, blockIdx.y counts
 // blocks of groups), or for groups wider than GNG_WARP_MAX the whole block (blockIdx.y is the group).
 constexpr int GNG_WARP_MAX = 256;
 template <typename T>
 __global__ void __launch_bounds__(128)
 group_norm_gate_kernel(T* __restrict__ out, const float* __restrict__ y, const float* __restrict__ z, int ldz,
-                       const float* __restrict__ w, int C, int gs, int wlen, float eps, int gate_first) {
+                       const float* __restrict__ w, int C, int gs, int wlen, float eps, int gate) {
   __shared__ float red[4];
   pdl_wait();
   const size_t m = blockIdx.x;
@@ -381,7 +414,7 @@ group_norm_gate_kernel(T* __restrict__ out, const float* __restrict__ y, const f
   float ss = 0.f;
   if (live)
     for (int i = t0; i < gs; i += nt) {
-      const float x = gate_first ? yr[i] * silu_f(zr[i]) : yr[i];
+      const float x = gate == 1 ? yr[i] * silu_f(zr[i]) : yr[i];
       ss += x * x;
     }
   ss = warp_sum(ss);
@@ -395,15 +428,16 @@ group_norm_gate_kernel(T* __restrict__ out, const float* __restrict__ y, const f
   const float r = 1.0f / sqrtf(ss / (float)gs + eps);
   for (int i = t0; i < gs; i += nt) {
     const int j = gidx * gs + i;
-    const float x = gate_first ? yr[i] * silu_f(zr[i]) : yr[i];
+    const float x = gate == 1 ? yr[i] * silu_f(zr[i]) : yr[i];
     float val = x * r * w[j % wlen];
-    if (!gate_first) val *= sigmoid_f(zr[i]);
+    if (gate == 0) val *= sigmoid_f(zr[i]);
+    if (gate == 2) val *= silu_f(zr[i]);
     out[m * C + j] = from_f32<T>(val);
   }
 }
 
 LEB_API int leb_group_norm_gate(void* out, int dtype, const float* y, const float* z, int ldz, const float* w, int M, int C,
-                                int gs, int wlen, float eps, int gate_first, cudaStream_t st) {
+                                int gs, int wlen, float eps, int gate, cudaStream_t st) {
   if (M <= 0) return 0;
   LEB_REQUIRE(gs >= 1 && C % gs == 0 && wlen >= 1, "leb_group_norm_gate: %d columns in groups of %d", C, gs);
   LebPlainLaunches plain(true);
@@ -411,9 +445,9 @@ LEB_API int leb_group_norm_gate(void* out, int dtype, const float* y, const floa
   const dim3 grid(M, gs > GNG_WARP_MAX ? groups : ceil_div(groups, 4));
   LEB_REQUIRE(grid.y <= 65535, "leb_group_norm_gate: %d groups in a row", groups);
   if (dtype == LEB_F32)
-    leb_launch(group_norm_gate_kernel<float>, grid, dim3(128), 0, st, (float*)out, y, z, ldz, w, C, gs, wlen, eps, gate_first);
+    leb_launch(group_norm_gate_kernel<float>, grid, dim3(128), 0, st, (float*)out, y, z, ldz, w, C, gs, wlen, eps, gate);
   else if (dtype == LEB_BF16)
-    leb_launch(group_norm_gate_kernel<bf16>, grid, dim3(128), 0, st, (bf16*)out, y, z, ldz, w, C, gs, wlen, eps, gate_first);
+    leb_launch(group_norm_gate_kernel<bf16>, grid, dim3(128), 0, st, (bf16*)out, y, z, ldz, w, C, gs, wlen, eps, gate);
   else
     return leb_fail("leb_group_norm_gate: unknown dtype %d", dtype);
   LEB_CHECK_LAUNCH("leb_group_norm_gate");

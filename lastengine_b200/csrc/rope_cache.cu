@@ -87,7 +87,8 @@ __global__ void __launch_bounds__(ROPE_WARPS * 32) qk_rope_store_kernel(
     const int* __restrict__ row_pos, const int* __restrict__ seq_slot,
     const float* __restrict__ q_norm_w, const float* __restrict__ k_norm_w, float eps,
     const float* __restrict__ inv_freq, int rope_dim, int neox, int M, int nh, int nkv, int hd,
-    int page_size, int vd, int v_norm, int hin, int vin) {   // hin <= hd, vin <= vd: a head's width in q_in/k_in and v_in
+    int page_size, int vd, int v_norm, int hin, int vin,     // hin <= hd, vin <= vd: a head's width in q_in/k_in and v_in
+    float temp_coef, float temp_every) {                     // q times query_temperature(position) (coef 0: as it is)
   extern __shared__ float sm[];
   pdl_trigger();   // the kernel after this one may start and wait (see common.cuh)
   pdl_wait();
@@ -152,7 +153,8 @@ __global__ void __launch_bounds__(ROPE_WARPS * 32) qk_rope_store_kernel(
     __syncwarp();
     if (is_q) {
       T* o = q_out + ((size_t)m * nh + head) * hd;
-      for (int i = lane; i < hd; i += 32) o[i] = from_f32<T>(v[i]);
+      const float factor = query_temperature(pos, temp_coef, temp_every);
+      for (int i = lane; i < hd; i += 32) o[i] = from_f32<T>(v[i] * factor);
     } else {
       CT* o = k_pool + kdst + (size_t)(head - nh) * page_size * hd;
       for (int i = lane; i < hd; i += 32) o[i] = from_f32<CT>(v[i]);
@@ -172,7 +174,8 @@ __global__ void __launch_bounds__(ROPE_WARPS * 32) qk_rope_store_lanes_kernel(
     const int* __restrict__ block_table, int bt_width,
     const int* __restrict__ row_seq, const int* __restrict__ row_pos, const int* __restrict__ seq_slot,
     const float* __restrict__ q_norm_w, const float* __restrict__ k_norm_w, float eps,
-    const float* __restrict__ inv_freq, int M, int nh, int nkv, int page_size, int per_warp, int vd, int v_norm, int vin) {
+    const float* __restrict__ inv_freq, int M, int nh, int nkv, int page_size, int per_warp, int vd, int v_norm, int vin,
+    float temp_coef, float temp_every) {
   constexpr int HD = EPL * 32, NP = EPL / 2, U = 4;
   pdl_trigger();   // the kernel after this one may start and wait (see common.cuh)
   pdl_wait();
@@ -197,7 +200,7 @@ __global__ void __launch_bounds__(ROPE_WARPS * 32) qk_rope_store_lanes_kernel(
   float c[NP], sn[NP], wq[EPL], wk[EPL];
 #pragma unroll
   for (int p = 0; p < NP; p++) {
-    const float th = (float)pos * inv_freq[lane + 32 * p];
+    const float th = inv_freq ? (float)pos * inv_freq[lane + 32 * p] : 0.f;     // no rotation: turned by zero
     c[p] = cosf(th);
     sn[p] = sinf(th);
   }
@@ -206,6 +209,7 @@ __global__ void __launch_bounds__(ROPE_WARPS * 32) qk_rope_store_lanes_kernel(
     wq[e] = q_norm_w ? q_norm_w[lane + 32 * e] : 1.f;
     wk[e] = k_norm_w ? k_norm_w[lane + 32 * e] : 1.f;
   }
+  const float factor = query_temperature(pos, temp_coef, temp_every);
   for (int hb = h0; hb < h1; hb += U) {
     float x[U][EPL];
 #pragma unroll
@@ -245,7 +249,7 @@ __global__ void __launch_bounds__(ROPE_WARPS * 32) qk_rope_store_lanes_kernel(
       if (is_q) {
         T* o = q_out + ((size_t)m * nh + head) * HD;
 #pragma unroll
-        for (int e = 0; e < EPL; e++) o[lane + 32 * e] = from_f32<T>(x[u][e]);
+        for (int e = 0; e < EPL; e++) o[lane + 32 * e] = from_f32<T>(x[u][e] * factor);
       } else {
         CT* o = k_pool + kdst + (size_t)(head - nh) * page_size * HD;
 #pragma unroll
@@ -431,8 +435,10 @@ LEB_API int leb_qk_rope_store(void* q_out, const void* q_in, int q_stride, const
                               const int* row_pos, const int* seq_slot, const float* q_norm_w,
                               const float* k_norm_w, float eps, const float* inv_freq, int rope_dim,
                               int neox, int M, int nh, int nkv, int hd, int page_size, int vd, int v_norm,
-                              int hin, int vin, cudaStream_t st) {
+                              int hin, int vin, float temp_coef, float temp_every, cudaStream_t st) {
   if (M <= 0) return 0;
+  if (!inv_freq) rope_dim = 0;
+  LEB_REQUIRE(temp_coef == 0.f || temp_every > 0.f, "leb_qk_rope_store: a temperature that rises every %g positions", temp_every);
   LEB_REQUIRE(hd >= 2 && hd <= 512, "leb_qk_rope_store: head_dim %d outside 2..512", hd);
   LEB_REQUIRE(rope_dim <= hd && rope_dim % 2 == 0, "leb_qk_rope_store: rope_dim %d does not fit head_dim %d", rope_dim, hd);
   if (vd <= 0) vd = hd;      // values as wide as keys
@@ -442,7 +448,7 @@ LEB_API int leb_qk_rope_store(void* q_out, const void* q_in, int q_stride, const
   int tiles = k_in ? ceil_div(M, VT_ROWS) * nkv : 0;
   int total = nh + (k_in ? nkv : 0);
   dim3 block(32 * ROPE_WARPS);
-  if (dtype == LEB_BF16 && inv_freq && neox && rope_dim == hd && hin == hd && (hd == 64 || hd == 128)) {
+  if (dtype == LEB_BF16 && (inv_freq ? neox && rope_dim == hd : temp_coef != 0.f) && hin == hd && (hd == 64 || hd == 128)) {
     // heads per warp: one while the launch is small, up to all of a row's over 8 warps
     int per_warp = 1;
     const long long n_sm = sm_count();
@@ -452,12 +458,12 @@ LEB_API int leb_qk_rope_store(void* q_out, const void* q_in, int q_stride, const
       leb_launch(qk_rope_store_lanes_kernel<bf16, bf16, 2>, grid, block, 0, st,
           (bf16*)q_out, (const bf16*)q_in, q_stride, (const bf16*)k_in, (const bf16*)v_in, kv_stride,
           (bf16*)k_pool, (bf16*)v_pool, block_table, bt_width, row_seq, row_pos, seq_slot, q_norm_w,
-          k_norm_w, eps, inv_freq, M, nh, nkv, page_size, per_warp, vd, v_norm, vin);
+          k_norm_w, eps, inv_freq, M, nh, nkv, page_size, per_warp, vd, v_norm, vin, temp_coef, temp_every);
     else
       leb_launch(qk_rope_store_lanes_kernel<bf16, bf16, 4>, grid, block, 0, st,
           (bf16*)q_out, (const bf16*)q_in, q_stride, (const bf16*)k_in, (const bf16*)v_in, kv_stride,
           (bf16*)k_pool, (bf16*)v_pool, block_table, bt_width, row_seq, row_pos, seq_slot, q_norm_w,
-          k_norm_w, eps, inv_freq, M, nh, nkv, page_size, per_warp, vd, v_norm, vin);
+          k_norm_w, eps, inv_freq, M, nh, nkv, page_size, per_warp, vd, v_norm, vin, temp_coef, temp_every);
     LEB_CHECK_LAUNCH("leb_qk_rope_store");
     return 0;
   }
@@ -467,12 +473,14 @@ LEB_API int leb_qk_rope_store(void* q_out, const void* q_in, int q_stride, const
     leb_launch(qk_rope_store_kernel<float, float>, grid, block, smem, st,
         (float*)q_out, (const float*)q_in, q_stride, (const float*)k_in, (const float*)v_in,
         kv_stride, (float*)k_pool, (float*)v_pool, block_table, bt_width, row_seq, row_pos,
-        seq_slot, q_norm_w, k_norm_w, eps, inv_freq, rope_dim, neox, M, nh, nkv, hd, page_size, vd, v_norm, hin, vin);
+        seq_slot, q_norm_w, k_norm_w, eps, inv_freq, rope_dim, neox, M, nh, nkv, hd, page_size, vd, v_norm, hin, vin,
+        temp_coef, temp_every);
   else if (dtype == LEB_BF16)
     leb_launch(qk_rope_store_kernel<bf16, bf16>, grid, block, smem, st,
         (bf16*)q_out, (const bf16*)q_in, q_stride, (const bf16*)k_in, (const bf16*)v_in, kv_stride,
         (bf16*)k_pool, (bf16*)v_pool, block_table, bt_width, row_seq, row_pos, seq_slot, q_norm_w,
-        k_norm_w, eps, inv_freq, rope_dim, neox, M, nh, nkv, hd, page_size, vd, v_norm, hin, vin);
+        k_norm_w, eps, inv_freq, rope_dim, neox, M, nh, nkv, hd, page_size, vd, v_norm, hin, vin,
+        temp_coef, temp_every);
   else
     return leb_fail("leb_qk_rope_store: unknown dtype %d", dtype);
   LEB_CHECK_LAUNCH("leb_qk_rope_store");

@@ -301,6 +301,9 @@ class Engine:
             blk = self.model.blocks[e.layer]
             layer_flops += sum(p.flops_per_row() for p in blk.parts().values())
             pair_flops += blk.mixer.flops_per_query_key()
+        for a in self.plan.stream_adds:
+            if a.matrix is not None:
+                layer_flops += 2 * self.model.stream_matrices[a.matrix].numel()
         specs = []
         for spec in self.model.cache_specs().values():
             specs += list(spec) if isinstance(spec, (tuple, list)) else [spec]
@@ -340,4 +343,4 @@ class Engine:
                     walk(v)
         for _, part in self.model.named_parts():
             walk(part)
-        return n
+        return n + sum(t.numel() * t.element_size() for t in self.model.stream_matrices.values())

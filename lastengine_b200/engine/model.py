@@ -11,8 +11,12 @@ import torch
 from .. import parts as _parts  # noqa: F401  (registers the built-in parts)
 from ..parts.base import BuildEnv, ModelPlan, TensorSpec
 from ..ops import kernels
-from ..parts.base import VECTOR
+from ..parts.base import MATRIX, VECTOR
 from ..registry import BLOCKS, EMBEDDINGS, FEED_FORWARDS, GATES, HEADS, MIXERS, NORMS
+
+
+# the cache entry of an embedding that keeps state per sequence (the schedule's entries count from 0)
+EMBEDDING_ENTRY = -1
 
 
 class Model:
@@ -36,7 +40,10 @@ class Model:
         for a in plan.stream_adds:
             self.stream_adds.setdefault(a.before, []).append(a)
         self.keeps_embedding = any(a.embedding for a in plan.stream_adds)
+        self.projects_stream = any(a.matrix is not None for a in plan.stream_adds)
         self.stream_tables: dict[str, torch.Tensor] = {}
+        self.stream_matrices: dict[str, torch.Tensor] = {}
+        self.embedding_spec = self.embedding.cache_spec() if hasattr(self.embedding, "cache_spec") else None
 
     # ---- tensors ------------------------------------------------------------------------
     def named_parts(self) -> list[tuple[str, object]]:
@@ -65,6 +72,8 @@ class Model:
                 specs[name] = spec
         for name, shape in self.plan.stream_tables.items():
             specs[name] = TensorSpec(tuple(shape), VECTOR)
+        for name, shape in self.plan.stream_matrices.items():
+            specs[name] = TensorSpec(tuple(shape), MATRIX)
         return specs
 
     def load(self, tensors: dict[str, torch.Tensor]) -> None:
@@ -77,12 +86,15 @@ class Model:
                     own[rel] = tensors[name]
             part.load(own, self.env)
         self.stream_tables = {n: tensors[n].contiguous() for n in self.plan.stream_tables if n in tensors}
+        self.stream_matrices = {n: tensors[n].contiguous() for n in self.plan.stream_matrices if n in tensors}
         if getattr(self.head, "tied", False):
             self.head.tie(self.embedding)
 
     def cache_specs(self) -> dict[int, object]:
         """cache entry id -> spec, for the entries that own storage."""
         specs = {}
+        if self.embedding_spec is not None:
+            specs[EMBEDDING_ENTRY] = self.embedding_spec
         for i, e in enumerate(self.plan.schedule):
             if e.cache is None or e.cache == i:
                 specs[i] = self.blocks[e.layer].mixer.cache_spec()
@@ -95,11 +107,17 @@ class Model:
         env, ws = self.env, self.env.workspace
         M, D = batch.n_rows, self.hidden_size
         x = ws.get("model.x", (M, D), torch.float32)
-        self.embedding.forward(x, batch.tokens, batch=batch)
-        x0 = None
+        if self.embedding_spec is not None:
+            self.embedding.forward(x, batch.tokens, batch=batch, cache=cache.view(EMBEDDING_ENTRY, True, batch.tables))
+        else:
+            self.embedding.forward(x, batch.tokens, batch=batch)
+        x0 = pair = None
         if self.keeps_embedding:      # the embedding output is added to the stream again later
             x0 = ws.get("model.x0", (M, D), torch.float32)
-            self.embedding.forward(x0, batch.tokens, batch=batch)
+            kernels.stream_columns(x0, x)
+        if self.projects_stream:      # or enters a product beside the stream: [stream | embedding output] in one row
+            pair = ws.get("model.pair", (M, 2 * D), env.dtype)
+            kernels.stream_columns(pair[:, D:], x)
         sched = self.plan.schedule
         pending = None      # the half of the next block's first norm that the last block left (decode steps)
         for i, e in enumerate(sched):
@@ -107,6 +125,13 @@ class Model:
             view = cache.view(entry, e.writes_cache and entry == i, batch.tables)
             block = self.blocks[e.layer]
             for a in self.stream_adds.get(i, ()):
+                if a.matrix is not None:
+                    # the stream's columns take their place in the rows, the stream becomes the table's row, and the product is added
+                    kernels.stream_columns(pair[:, :D], x, self.stream_tables[a.table][a.row] if a.table is not None else None,
+                                           fill=True)
+                    kernels.linear(x, pair, self.stream_matrices[a.matrix], kernels.ACCUMULATE)
+                    pending = None
+                    continue
                 kernels.stream_add(x, x0 if a.embedding else None,
                                    self.stream_tables[a.table][a.row] if a.table is not None else None)
                 pending = None      # a norm half left for this block was taken from the stream as it was before

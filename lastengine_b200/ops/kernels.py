@@ -90,16 +90,16 @@ class KernelTimer:
 
 
 def _declare(L) -> None:
-    P, I, F, S = c_void_p, c_int, c_float, c_size_t
+    P, I, F, S, LL = c_void_p, c_int, c_float, c_size_t, ctypes.c_longlong
     sig = {
         "leb_embed": [P, P, I, P, I, I, I, F, P],
         "leb_rmsnorm": [P, I, P, P, P, I, I, F, I, P],
         "leb_swiglu": [P, I, P, I, I, I, P],
-        "leb_gather_rows": [P, P, I, P, I, I, I, P],
+        "leb_gather_rows": [P, P, I, P, P, I, I, I, P],
         "leb_add": [P, P, S, P],
         "leb_shortconv": [P, P, I, P, P, P, P, P, P, P, I, I, I, I, P],
-        "leb_qk_rope_store": [P, P, I, P, P, I, P, P, I, P, I, P, P, P, P, P, F, P, I, I, I, I, I, I, I, I, I, I, I, P],
-        "leb_attention": [P, P, P, P, P, I, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, I, I, P],
+        "leb_qk_rope_store": [P, P, I, P, P, I, P, P, I, P, I, P, P, P, P, P, F, P, I, I, I, I, I, I, I, I, I, I, I, F, F, P],
+        "leb_attention": [P, P, P, P, P, I, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, P, P, I, I, I, P],
         "leb_gated_act": [P, I, P, I, I, I, I, F, F, P],
         "leb_layernorm": [P, I, P, P, P, I, I, F, P],
         "leb_scaled_residual": [P, P, F, P, I, P, F, I, I, P],
@@ -134,16 +134,16 @@ def _declare(L) -> None:
         "leb_penalties_slots": [P, P, P, P, I, I, I, F, F, P],
         "leb_history_append": [P, P, P, P, I, I, P],
         "leb_attention_decode_supported": [I, I, I, I],
-        "leb_attention_decode": [P, P, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P],
-        "leb_attention_merge": [P, P, I, P, I, I, I, I, I, I, P],
+        "leb_attention_decode": [P, P, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, P, P, I, P],
+        "leb_attention_merge": [P, P, I, P, I, I, P, I, I, I, I, P],
         "leb_attention_decode_prep_supported": [I, I, I, I, I, I],
-        "leb_attention_decode_prep": [P, P, P, I, P, P, I, P, P, P, I, P, P, P, P, P, F, P, I, I, I, P, I, I, I, I, I, I, I, I, I, I, F, I, P],
+        "leb_attention_decode_prep": [P, P, P, I, P, P, I, P, P, P, I, P, P, P, P, P, F, P, I, I, I, P, I, I, I, I, I, I, I, I, I, I, F, P, P, F, F, I, P],
         "leb_attention_prefill_supported": [I, I, I, I],
         "leb_attention_prefill_tc_supported": [I, I, I, I],
-        "leb_attention_prefill_tc": [P, P, I, I, P, P, I, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, P],
+        "leb_attention_prefill_tc": [P, P, I, I, P, P, I, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, P, P, I, P, P],
         "leb_attention_pooled_tc": [P, P, I, I, P, P, I, P, I, P, P, I, P, I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P, P],
         "leb_attention_pooled_tc_value_dim": [I],
-        "leb_attention_prefill": [P, P, P, P, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P],
+        "leb_attention_prefill": [P, P, P, P, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, P, P, I, P],
         "leb_gemm_bf16_skinny_slices": [I, I],
         "leb_gemm_bf16_skinny_supported": [P, P, I, I, I],
         "leb_gemm_bf16_skinny": [P, I, P, P, I, I, I, I, I, I, P, I, P, I, I, F, P, P, P, P, P],
@@ -153,7 +153,7 @@ def _declare(L) -> None:
         "leb_selftest_bounded_wait": [P, I, I, P],
         "leb_gemm_bf16_tc_slices": [I, I, I],
         "leb_gemm_bf16_tc_sliced": [P, I, P, P, I, I, I, I, I, I, P, I, P, P],
-        "leb_gated_recurrence": [P, I, P, P, I, P, I, P, I, P, I, I, I, P, P, P, P, P, I, I, I, I, I, I, P],
+        "leb_gated_recurrence": [P, I, P, P, I, P, I, P, I, P, I, I, I, P, P, P, P, P, P, I, I, I, I, I, I, P],
         "leb_min_gru": [P, I, P, P, P, I, P, P, P, P, P, P, I, I, I, P, P],
         "leb_exp_gates": [P, P, P, P, P, I, P, P, F, P, P, P, P, I, I, I, P],
         "leb_exp_gates_finish": [P, I, P, P, P, I, P, F, F, I, I, I, P],
@@ -172,6 +172,12 @@ def _declare(L) -> None:
         "leb_qk_row_norm_rope_store": [P, P, I, P, P, I, P, P, I, P, I, P, P, P, P, P, F, P, I, I, I, I, I, I, I, I, I, I, P],
         "leb_outnorm_residual": [P, P, P, F, P, I, I, I, P],
         "leb_softcap": [P, F, F, S, P],
+        "leb_pointwise_norm": [P, I, P, P, F, P, P, I, I, I, P],
+        "leb_pointwise_norm_sum": [P, P, F, P, F, F, P, P, P, I, F, P, P, I, I, P],
+        "leb_stream_columns": [P, I, I, P, P, I, I, I, P],
+        "leb_embed_pairs": [P, P, P, I, P, P, P, P, P, P, P, I, I, I, I, LL, LL, F, P],
+        "leb_row_shift_mix": [P, P, I, P, P, P, P, P, P, I, I, I, P],
+        "leb_low_rank_decay": [P, P, I, P, P, I, I, I, P],
         "leb_cast_rows": [P, I, P, S, P],
         "leb_pooled_attn_prep": [P, P, P, I, P, I, P, P, P, F, P, I, P, P, I, P, P, P, I, I, I, I, I, I, P],
         "leb_pool_blocks": [P, P, P, P, I, P, I, P, I, P, P, P, I, I, I, I, I, I, I, P],
@@ -356,6 +362,121 @@ def softcap(z: torch.Tensor, scale: float, cap: float) -> None:
     _check(lib().leb_softcap(_ptr(z), float(scale), float(cap), z.numel(), _stream()))
 
 
+def pointwise_norm(out: torch.Tensor, x: torch.Tensor, alpha: float, w: torch.Tensor, b: torch.Tensor,
+                   rows: torch.Tensor | None = None, add: bool = False) -> None:
+    """out = tanh(alpha x[rows]) * w + b element by element (out += ... with add, out float then); x float."""
+    _cuda(out, "pointwise_norm.out")
+    _cuda(x, "pointwise_norm.x", torch.float32)
+    _cuda(w, "pointwise_norm.w", torch.float32)
+    _cuda(b, "pointwise_norm.b", torch.float32)
+    M, D = out.shape
+    assert x.shape[1] == D and w.numel() == D and b.numel() == D
+    if rows is not None:
+        _cuda(rows, "pointwise_norm.rows", torch.int32)
+        assert rows.numel() >= M
+    else:
+        assert x.shape[0] >= M
+    _check(lib().leb_pointwise_norm(_ptr(out), _dt(out, "pointwise_norm.out"), _ptr(x), _ptr(rows), float(alpha), _ptr(w), _ptr(b),
+                                    M, D, 1 if add else 0, _stream()))
+
+
+def pointwise_norm_sum(x: torch.Tensor, y: torch.Tensor, norm: tuple, h: torch.Tensor | None = None, next_norm: tuple | None = None,
+                       weighted: tuple | None = None) -> None:
+    """x += norm(y) element by element (x, y float [M, D]; a norm is (alpha, w, b)); with `h` the launch also leaves
+    next_norm(x) of the new rows there in h's type.  `weighted` = (c1, y2, c2): c1 y + c2 y2 stands in y's place."""
+    _cuda(x, "pointwise_norm_sum.x", torch.float32)
+    _cuda(y, "pointwise_norm_sum.y", torch.float32)
+    M, D = x.shape
+    assert y.shape == (M, D)
+    for _, w, b in [norm] + ([next_norm] if next_norm is not None else []):
+        _cuda(w, "pointwise_norm_sum.w", torch.float32)
+        _cuda(b, "pointwise_norm_sum.b", torch.float32)
+        assert w.numel() == D and b.numel() == D
+    c1, y2, c2 = weighted if weighted is not None else (1.0, None, 0.0)
+    if y2 is not None:
+        _cuda(y2, "pointwise_norm_sum.y2", torch.float32)
+        assert y2.shape == (M, D)
+    a2, w2, b2 = next_norm if h is not None else (0.0, None, None)
+    if h is not None:
+        _cuda(h, "pointwise_norm_sum.h")
+        assert h.shape == (M, D)
+    _check(lib().leb_pointwise_norm_sum(_ptr(x), _ptr(y), float(c1), _ptr(y2), float(c2), float(norm[0]), _ptr(norm[1]),
+                                        _ptr(norm[2]), _ptr(h), _dt(h, "pointwise_norm_sum.h") if h is not None else F32,
+                                        float(a2), _ptr(w2), _ptr(b2), M, D, _stream()))
+
+
+def stream_columns(out: torch.Tensor, x: torch.Tensor, vec: torch.Tensor | None = None, fill: bool = False) -> None:
+    """out = x in out's type (out [M, D] may be a column range of a wider tensor); with `fill`, x <- vec in every row
+    (None: zeros) afterwards."""
+    _cuda(out, "stream_columns.out", contiguous=False)
+    _cuda(x, "stream_columns.x", torch.float32)
+    M, D = x.shape
+    assert out.shape == (M, D) and out.stride(1) == 1
+    if vec is not None:
+        _cuda(vec, "stream_columns.vec", torch.float32)
+        assert vec.numel() == D
+    _check(lib().leb_stream_columns(_ptr(out), out.stride(0), _dt(out, "stream_columns.out"), _ptr(x), _ptr(vec), 1 if fill else 0,
+                                    M, D, _stream()))
+
+
+def embed_pairs(x: torch.Tensor, table: torch.Tensor, pairs: torch.Tensor, tokens: torch.Tensor, state: torch.Tensor, batch,
+                mul_prev: int, mul_cur: int, scale: float = 1.0) -> None:
+    """x[m] = table[token] * scale + pairs[(previous token * mul_prev + token * mul_cur) mod (rows - 1)] as float, the last
+    row of `pairs` for a sequence's first token.  `state` int32 [slots, 1]: every sequence's last token, moved on."""
+    _cuda(x, "embed_pairs.x", torch.float32)
+    _cuda(table, "embed_pairs.table")
+    _cuda(pairs, "embed_pairs.pairs", table.dtype)
+    _cuda(tokens, "embed_pairs.tokens", torch.int32)
+    _cuda(state, "embed_pairs.state", torch.int32)
+    M, D = x.shape
+    assert table.shape[1] == D and pairs.shape[1] == D and tokens.numel() >= M and state.shape[1:] == (1,)
+    single = batch.max_qlen == 1 and M == batch.n_seqs
+    _check(lib().leb_embed_pairs(_ptr(x), _ptr(table), _ptr(pairs), _dt(table, "embed_pairs.table"), _ptr(tokens),
+                                 _ptr(batch.row_seq), _ptr(batch.row_pos), _ptr(batch.seq_slot), _ptr(batch.seq_qstart),
+                                 None if single else _ptr(batch.seq_qlen), _ptr(state), M, D, table.shape[0], pairs.shape[0] - 1,
+                                 int(mul_prev), int(mul_cur), float(scale), _stream()))
+
+
+def row_shift_mix(mix: torch.Tensor, h: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, batch) -> None:
+    """mix[s, m] = h[m] + (row before - h[m]) * mu[s] (mu float [n, D]); the row before a sequence's first is zeros, and
+    `state` float [slots, D] carries every sequence's last row to its next step."""
+    _cuda(mix, "row_shift_mix.mix")
+    _cuda(h, "row_shift_mix.h", mix.dtype)
+    _cuda(mu, "row_shift_mix.mu", torch.float32)
+    _cuda(state, "row_shift_mix.state", torch.float32)
+    n, M, D = mix.shape
+    assert h.shape == (M, D) and mu.shape == (n, D) and state.shape[1:] == (D,)
+    single = batch.max_qlen == 1 and M == batch.n_seqs
+    _check(lib().leb_row_shift_mix(_ptr(mix), _ptr(h), _dt(mix, "row_shift_mix"), _ptr(mu), _ptr(state), _ptr(batch.row_seq),
+                                   _ptr(batch.seq_slot), _ptr(batch.seq_qstart), None if single else _ptr(batch.seq_qlen),
+                                   M, D, n, _stream()))
+
+
+def low_rank_decay(out: torch.Tensor, low: torch.Tensor, w2: torch.Tensor, w0: torch.Tensor) -> None:
+    """out = exp(-exp(tanh(low) . w2 + w0)), all float: low [M, rank] (a column range is fine), w2 [rank, C], w0 [C]."""
+    _cuda(out, "low_rank_decay.out", torch.float32)
+    M, C = out.shape
+    _cuda(w2, "low_rank_decay.w2", torch.float32)
+    _cuda(w0, "low_rank_decay.w0", torch.float32)
+    rank = w2.shape[0]
+    ldl = _f32_rows(low, "low_rank_decay.low", M, rank)
+    assert w2.shape == (rank, C) and w0.numel() == C
+    _check(lib().leb_low_rank_decay(_ptr(out), _ptr(low), ldl, _ptr(w2), _ptr(w0), M, C, rank, _stream()))
+
+
+_GROUP_OFFSETS: dict[tuple, torch.Tensor] = {}
+
+
+def equal_group_offsets(n: int, M: int, device) -> torch.Tensor:
+    """Row ranges for a grouped product over n buffers of M rows each, one behind the other: buffer i owns rows [i M, (i + 1) M).
+    Made once per (n, M) and kept for good (a few bytes each): captured steps hold their addresses."""
+    key = (int(n), int(M), str(device))
+    t = _GROUP_OFFSETS.get(key)
+    if t is None:
+        t = _GROUP_OFFSETS[key] = (torch.arange(n + 1, dtype=torch.int64) * M).to(torch.int32).to(device)
+    return t
+
+
 def embed_positions(x: torch.Tensor, h: torch.Tensor | None, table: torch.Tensor, tokens: torch.Tensor,
                     positions: torch.Tensor, row_pos: torch.Tensor, scale: float = 1.0) -> None:
     """x[m] = table[tokens[m]] * scale + positions[row_pos[m]] as float; with `h`, the rows in h's type too."""
@@ -432,26 +553,30 @@ def ssm_prep(xbc: torch.Tensor, conv_bias: torch.Tensor | None, dt: torch.Tensor
 RECURRENCE_MAX_ROWS = 256     # rows of a head's state the recurrence kernel takes
 
 
-def gated_recurrence(out: torch.Tensor, k: torch.Tensor, q: torch.Tensor, v: torch.Tensor, write: torch.Tensor,
+def gated_recurrence(out: torch.Tensor, k: torch.Tensor, q: torch.Tensor, v: torch.Tensor, write: torch.Tensor | None,
                      decay: torch.Tensor, state: torch.Tensor, batch, H: int, Gk: int, d: int, e: int,
-                     delta: bool, skip: torch.Tensor | None = None, ones_columns: int = 0) -> None:
+                     delta: bool, skip: torch.Tensor | None = None, ones_columns: int = 0,
+                     bonus: torch.Tensor | None = None) -> None:
     """The linear recurrence of the step's rows with a state per sequence and head (all float):
         S <- diag(decay) S;  u = write * v (delta: write * (v - S^T k));  S <- S + k u^T;  o = S^T q (+ skip_h v)
     k, q [M, Gk*d] (one row stride), v [M, H*e], write [M, H], decay [M, H*d] (per key channel) or [M, H];
     head h reads key head h // (H // Gk); state [slots, H, e, d] (a column of S is contiguous); out [M, H*e].
     `ones_columns` n > 0: v has e - n columns per head and the state's last n columns are written with ones, so
-    they hold the (decayed, weighted) sum of the keys and their read-out is that sum's product with q."""
+    they hold the (decayed, weighted) sum of the keys and their read-out is that sum's product with q.
+    `bonus` [H*d] (decay per key channel): the read-out sees the state before the row and the row's own write weighted
+    per key channel, o = (S + diag(bonus) k u^T)^T q, and then S <- diag(decay) S + k u^T.  `write` None: ones."""
     M = out.shape[0]
     ev = e - int(ones_columns)
-    assert 0 <= ev <= e and not (delta and ones_columns)
+    assert 0 <= ev <= e and not (delta and ones_columns) and not (delta and bonus is not None)
     ldo = _f32_rows(out, "gated_recurrence.out", M, H * e)
     ldk = _f32_rows(k, "gated_recurrence.k", M, Gk * d)
     assert _f32_rows(q, "gated_recurrence.q", M, Gk * d) == ldk
     ldv = _f32_rows(v, "gated_recurrence.v", M, H * ev)
-    ldw = _f32_rows(write, "gated_recurrence.write", M, H)
-    row_decay = decay.shape[1] == H * d and not (d == 1 and decay.shape[1] == H and False)
-    if decay.shape[1] != H * d:
-        row_decay = False
+    ldw = _f32_rows(write, "gated_recurrence.write", M, H) if write is not None else 0
+    row_decay = decay.shape[1] == H * d
+    if bonus is not None:
+        _cuda(bonus, "gated_recurrence.bonus", torch.float32)
+        assert bonus.numel() == H * d and row_decay
     ldd = _f32_rows(decay, "gated_recurrence.decay", M, H * d if row_decay else H)
     _cuda(state, "gated_recurrence.state", torch.float32)
     assert state.shape[1:] == (H, e, d)
@@ -460,16 +585,17 @@ def gated_recurrence(out: torch.Tensor, k: torch.Tensor, q: torch.Tensor, v: tor
         assert skip.numel() == H
     single = batch.max_qlen == 1 and M == batch.n_seqs
     _check(lib().leb_gated_recurrence(_ptr(out), ldo, _ptr(k), _ptr(q), ldk, _ptr(v), ldv, _ptr(write), ldw, _ptr(decay), ldd,
-                                      1 if row_decay else 0, 1 if delta else 0, _ptr(skip), _ptr(state), _ptr(batch.seq_slot),
+                                      1 if row_decay else 0, 2 if bonus is not None else (1 if delta else 0), _ptr(skip),
+                                      _ptr(bonus), _ptr(state), _ptr(batch.seq_slot),
                                       _ptr(batch.seq_qstart), None if single else _ptr(batch.seq_qlen), batch.n_seqs,
                                       H, Gk, d, e, ev, _stream()))
 
 
 def group_norm_gate(out: torch.Tensor, y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, group_size: int, eps: float,
-                    gate_first: bool) -> None:
+                    gate_first: bool, silu_after: bool = False) -> None:
     """Groups of `group_size` neighbouring numbers of a row of y (float [M, C]) divided by their root mean square,
-    times w[j % len(w)], gated by z (float [M, C], a column slice is fine): times sigmoid(z) after the norm, or
-    (gate_first) y silu(z) before it.  out [M, C] in the activation type."""
+    times w[j % len(w)], gated by z (float [M, C], a column slice is fine): times sigmoid(z) after the norm (silu(z) with
+    `silu_after`), or (gate_first) y silu(z) before it.  out [M, C] in the activation type."""
     _cuda(out, "group_norm_gate.out")
     M, C = out.shape
     _cuda(y, "group_norm_gate.y", torch.float32)
@@ -477,7 +603,8 @@ def group_norm_gate(out: torch.Tensor, y: torch.Tensor, z: torch.Tensor, w: torc
     ldz = _f32_rows(z, "group_norm_gate.z", M, C)
     _cuda(w, "group_norm_gate.w", torch.float32)
     _check(lib().leb_group_norm_gate(_ptr(out), _dt(out, "group_norm_gate.out"), _ptr(y), _ptr(z), ldz, _ptr(w), M, C,
-                                     int(group_size), w.numel(), float(eps), 1 if gate_first else 0, _stream()))
+                                     int(group_size), w.numel(), float(eps), 2 if silu_after else (1 if gate_first else 0),
+                                     _stream()))
 
 
 def min_gru(out: torch.Tensor, pz: torch.Tensor, px: torch.Tensor, pg: torch.Tensor, bz: torch.Tensor | None,
@@ -924,14 +1051,19 @@ def retention(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tens
                                M, batch.n_seqs, H, d, e, _stream()))
 
 
-def gather_rows(out: torch.Tensor, src: torch.Tensor, rows: torch.Tensor, div: int = 1) -> None:
-    """out[p] = src[rows[p] // div]."""
+def gather_rows(out: torch.Tensor, src: torch.Tensor, rows: torch.Tensor, div: int = 1,
+                weights: torch.Tensor | None = None) -> None:
+    """out[p] = src[rows[p] // div], times weights[rows[p]] (float) where they are given."""
     _cuda(out, "gather_rows.out")
     _cuda(src, "gather_rows.src", out.dtype)
     _cuda(rows, "gather_rows.rows", torch.int32)
     P_, D = out.shape
     assert src.shape[1] == D and rows.numel() >= P_
-    _check(lib().leb_gather_rows(_ptr(out), _ptr(src), _dt(out, "gather_rows"), _ptr(rows), div, P_, D, _stream()))
+    if weights is not None:
+        _cuda(weights, "gather_rows.weights", torch.float32)
+        assert weights.numel() >= P_
+    _check(lib().leb_gather_rows(_ptr(out), _ptr(src), _dt(out, "gather_rows"), _ptr(rows), _ptr(weights), div, P_, D,
+                                 _stream()))
 
 
 def add_(x: torch.Tensor, y: torch.Tensor) -> None:
@@ -1008,12 +1140,16 @@ def shortconv_decode_fused(y: torch.Tensor, h: torch.Tensor, w_in: torch.Tensor,
     return True
 
 
+def _temperature(t: tuple[float, float] | None) -> tuple[float, float]:
+    return (0.0, 1.0) if t is None else (float(t[0]), float(t[1]))
+
+
 def qk_rope_store(q_out: torch.Tensor, q_in: torch.Tensor, k_in: torch.Tensor | None,
                   v_in: torch.Tensor | None, k_pool: torch.Tensor | None, v_pool: torch.Tensor | None,
                   block_table: torch.Tensor, batch, q_norm_w, k_norm_w, eps: float,
                   inv_freq: torch.Tensor | None, rope_dim: int, neox: bool, nh: int, nkv: int, hd: int,
                   page_size: int, vd: int | None = None, v_norm: bool = False, hd_in: int | None = None,
-                  vd_in: int | None = None) -> None:
+                  vd_in: int | None = None, temperature: tuple[float, float] | None = None) -> None:
     """Per-head norm and rotation of q and k; k and v go to the paged cache, q to q_out.
 
     q_in/k_in/v_in may be column slices of one fused projection (row stride = its width).
@@ -1021,7 +1157,7 @@ def qk_rope_store(q_out: torch.Tensor, q_in: torch.Tensor, k_in: torch.Tensor | 
     divided by its root mean square (with `eps`, no weight) before it is stored.  `hd_in` / `vd_in`:
     width of a head in q_in/k_in and in v_in where heads are stored wider than they are (hd in q_out
     and the key pool, vd in the value pool; the rest of a stored head is zeros, the norms run over the
-    head as it comes).
+    head as it comes).  `temperature` = (coef, every): q at position p times 1 + coef ln(floor((p + 1) / every) + 1).
     """
     vd = hd if vd is None else int(vd)
     hd_in = hd if hd_in is None else int(hd_in)
@@ -1053,7 +1189,7 @@ def qk_rope_store(q_out: torch.Tensor, q_in: torch.Tensor, k_in: torch.Tensor | 
         _dt(q_out, "qk_rope_store"), _ptr(block_table), block_table.shape[1], _ptr(batch.row_seq),
         _ptr(batch.row_pos), _ptr(batch.seq_slot), _ptr(q_norm_w), _ptr(k_norm_w), float(eps),
         _ptr(inv_freq), rope_dim, 1 if neox else 0, M, nh, nkv, hd, page_size, vd, 1 if v_norm else 0, hd_in, vd_in,
-        _stream()))
+        *_temperature(temperature), _stream()))
 
 
 def qk_row_norm_rope_store(q_out: torch.Tensor, q_in: torch.Tensor, k_in: torch.Tensor | None, v_in: torch.Tensor | None,
@@ -1254,7 +1390,7 @@ def sm_count() -> int:
     return n
 
 
-def attention_splits(batch, nkv: int, G: int, sm_count: int | None = None, hd: int = 64, chunk: int = 0) -> int:
+def attention_splits(batch, nkv: int, G: int, sm_count: int | None = None, hd: int = 64, chunk: int = 0, window: int = 0) -> int:
     """How many blocks share one sequence's key range in a decode step (1 for prompts).
 
     Measured on B200 (head size 64, 8 kv heads, times with the merge of the splits): a block has a
@@ -1270,7 +1406,7 @@ def attention_splits(batch, nkv: int, G: int, sm_count: int | None = None, hd: i
         return 1
     if sm_count is None:
         sm_count = globals()["sm_count"]()
-    kv = max(_read_length(int(batch.max_kvlen), 0, chunk), 1)
+    kv = max(_read_length(int(batch.max_kvlen), window, chunk), 1)
     per = max(batch.n_seqs * nkv * ((G + 15) // 16), 1)
     stage_bytes = 2 * 32 * hd * 2 * (3 if hd <= 32 else 2) * 4          # a block's rings: 4 warps, keys and values
     slots = sm_count * max(1, min(3, (227 * 1024) // stage_bytes))      # blocks that run at once
@@ -1287,21 +1423,25 @@ class RawQKV:
     """A decode step's q, k and v as the projection left them, for the decode attention kernel that
     norms, rotates and stores them itself (`decode_attention_takes_raw` says when it can)."""
 
-    def __init__(self, q_in, k_in, v_in, q_norm_w, k_norm_w, eps, inv_freq, rope_dim, neox, row_norm: bool = False):
-        """`row_norm`: q and k are normed over their whole row, with weights over the row."""
+    def __init__(self, q_in, k_in, v_in, q_norm_w, k_norm_w, eps, inv_freq, rope_dim, neox, row_norm: bool = False,
+                 temperature: tuple[float, float] | None = None):
+        """`row_norm`: q and k are normed over their whole row, with weights over the row.  `inv_freq` None: no rotation.
+        `temperature`: as in `qk_rope_store`."""
+        self.temperature = temperature
         self.row_norm = bool(row_norm)
         self.q_in, self.k_in, self.v_in = q_in, k_in, v_in
         self.q_norm_w, self.k_norm_w, self.eps = q_norm_w, k_norm_w, float(eps)
-        self.inv_freq, self.rope_dim, self.neox = inv_freq, int(rope_dim), bool(neox)
+        self.inv_freq, self.rope_dim, self.neox = inv_freq, (int(rope_dim) if inv_freq is not None else 0), bool(neox)
 
 
 def decode_attention_takes_raw(dtype: torch.dtype, batch, M: int, nh: int, nkv: int, hd: int, page_size: int,
                                inv_freq, rope_dim: int, neox: bool) -> bool:
     """Whether `attention(..., raw=...)` will do the per-head norm, the rotation and the cache write
     of this step itself: a bfloat16 decode step (one row per sequence) whose sizes the tensor-core
-    decode kernel takes, with a rotation over the whole head."""
-    return bool(dtype == torch.bfloat16 and batch.max_qlen == 1 and M == batch.n_seqs and inv_freq is not None
-                and lib().leb_attention_decode_prep_supported(nh, nkv, hd, page_size, int(rope_dim), 1 if neox else 0))
+    decode kernel takes, with a rotation over the whole head or none."""
+    rot = int(rope_dim) if inv_freq is not None else 0
+    return bool(dtype == torch.bfloat16 and batch.max_qlen == 1 and M == batch.n_seqs
+                and lib().leb_attention_decode_prep_supported(nh, nkv, hd, page_size, rot, 1 if neox else 0))
 
 
 def _gate_layout(gate: torch.Tensor | None, M: int, nh: int, width: int, dtype: torch.dtype) -> tuple[int, int]:
@@ -1317,20 +1457,27 @@ def attention(out: torch.Tensor, q: torch.Tensor | None, k_pool: torch.Tensor, v
               block_table: torch.Tensor, batch, nh: int, nkv: int, hd: int, page_size: int,
               window: int, scale: float, gate: torch.Tensor | None = None,
               n_splits: int = 1, scratch: torch.Tensor | None = None, raw: RawQKV | None = None,
-              vd: int | None = None, chunk: int = 0, wide: bool = False) -> None:
+              vd: int | None = None, chunk: int = 0, wide: bool = False, slopes: torch.Tensor | None = None,
+              sinks: torch.Tensor | None = None) -> None:
     """Causal attention of the step's rows over the paged cache (which already holds their keys;
     with `raw`, the kernel puts the step's keys and values there itself and `q` is not used).
     `vd`: width of a value head where it differs from the key head's (the general kernel then).
     `gate`: [rows, heads], a factor sigmoid(gate) per head, or [rows, heads * value width], one per number.
     `chunk` > 0: a row reads its own chunk of that many positions only, counted from the sequence's first.
-    `wide`: the softmax weights enter the bfloat16 product with the values as two terms (16 significant bits)."""
+    `wide`: the softmax weights enter the bfloat16 product with the values as two terms (16 significant bits).
+    `slopes` [heads]: slope_h (i - j) is taken off the scaled score of query i and key j.  `sinks` [heads]: one more logit
+    per head in the softmax's denominator, without a key and without a value, not scaled."""
     _cuda(out, "attention.out")
+    for name, t in (("slopes", slopes), ("sinks", sinks)):
+        if t is not None:
+            _cuda(t, f"attention.{name}", torch.float32)
+            assert t.numel() == nh
     if vd is not None and vd != hd:
         return _attention_general(out, q, k_pool, v_pool, block_table, batch, nh, nkv, hd, int(vd), page_size, window,
-                                  scale, gate, n_splits, scratch, chunk)
+                                  scale, gate, n_splits, scratch, chunk, slopes, sinks)
     if raw is not None:
         return _attention_decode_raw(out, raw, k_pool, v_pool, block_table, batch, nh, nkv, hd, page_size, window,
-                                     scale, gate, n_splits, scratch, chunk, wide)
+                                     scale, gate, n_splits, scratch, chunk, wide, slopes, sinks)
     _cuda(q, "attention.q", out.dtype)
     _cuda(k_pool, "attention.k_pool", out.dtype)
     _cuda(v_pool, "attention.v_pool", out.dtype)
@@ -1352,10 +1499,10 @@ def attention(out: torch.Tensor, q: torch.Tensor | None, k_pool: torch.Tensor, v
             _ptr(out), _ptr(scratch), _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(block_table),
             block_table.shape[1], _ptr(batch.seq_slot), _ptr(batch.seq_pos0), _ptr(batch.seq_qstart),
             _ptr(gate), gate_stride, gate_elem, batch.n_seqs, nh, nkv, hd, page_size, window, chunk, int(wide), float(scale),
-            n_splits, _stream()))
+            _ptr(slopes), _ptr(sinks), n_splits, _stream()))
         if n_splits > 1:
-            _check(L.leb_attention_merge(_ptr(out), _ptr(scratch), BF16, _ptr(gate), gate_stride, gate_elem, M, nh, hd,
-                                         n_splits, _stream()))
+            _check(L.leb_attention_merge(_ptr(out), _ptr(scratch), BF16, _ptr(gate), gate_stride, gate_elem, _ptr(sinks), M,
+                                         nh, hd, n_splits, _stream()))
         return
     if (out.dtype == torch.bfloat16 and n_splits == 1 and batch.max_qlen >= TC_ATTENTION_MIN_ROWS
             and q.stride(0) % 8 == 0 and L.leb_attention_prefill_tc_supported(nh, nkv, hd, page_size)):
@@ -1364,7 +1511,7 @@ def attention(out: torch.Tensor, q: torch.Tensor | None, k_pool: torch.Tensor, v
             _ptr(out), _ptr(q), q.stride(0), M, _ptr(k_pool), _ptr(v_pool), k_pool.shape[0], _ptr(block_table),
             block_table.shape[1], _ptr(batch.seq_slot), _ptr(batch.seq_pos0), _ptr(batch.seq_qstart),
             _ptr(batch.seq_qlen), _ptr(gate), gate_stride, gate_elem, batch.n_seqs, nh, nkv, hd, page_size, window, chunk,
-            int(wide), float(scale), batch.max_qlen, _ptr(_status_word(out.device)), _stream()))
+            int(wide), float(scale), _ptr(slopes), _ptr(sinks), batch.max_qlen, _ptr(_status_word(out.device)), _stream()))
         return
     if (out.dtype == torch.bfloat16 and n_splits == 1
             and L.leb_attention_prefill_supported(nh, nkv, hd, page_size)):
@@ -1373,17 +1520,17 @@ def attention(out: torch.Tensor, q: torch.Tensor | None, k_pool: torch.Tensor, v
             _ptr(out), _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(block_table), block_table.shape[1],
             _ptr(batch.seq_slot), _ptr(batch.seq_pos0), _ptr(batch.seq_qstart), _ptr(batch.seq_qlen),
             _ptr(gate), gate_stride, gate_elem, batch.n_seqs, nh, nkv, hd, page_size, window, chunk, int(wide), float(scale),
-            batch.max_qlen, _stream()))
+            _ptr(slopes), _ptr(sinks), batch.max_qlen, _stream()))
         return
     _check(L.leb_attention(
         _ptr(out), _ptr(scratch), _ptr(q), _ptr(k_pool), _ptr(v_pool), _dt(out, "attention"),
         _ptr(block_table), block_table.shape[1], _ptr(batch.seq_slot), _ptr(batch.seq_pos0),
         _ptr(batch.seq_qstart), _ptr(batch.seq_qlen), _ptr(gate), gate_stride, gate_elem, M, batch.n_seqs, nh, nkv,
-        hd, page_size, window, chunk, float(scale), batch.max_qlen, n_splits, hd, _stream()))
+        hd, page_size, window, chunk, float(scale), _ptr(slopes), _ptr(sinks), batch.max_qlen, n_splits, hd, _stream()))
 
 
 def _attention_general(out, q, k_pool, v_pool, block_table, batch, nh, nkv, hd, vd, page_size, window, scale, gate,
-                       n_splits, scratch, chunk=0) -> None:
+                       n_splits, scratch, chunk=0, slopes=None, sinks=None) -> None:
     """The general kernel with value heads of their own width."""
     _cuda(q, "attention.q", out.dtype)
     _cuda(k_pool, "attention.k_pool", out.dtype)
@@ -1401,11 +1548,11 @@ def _attention_general(out, q, k_pool, v_pool, block_table, batch, nh, nkv, hd, 
         _ptr(out), _ptr(scratch), _ptr(q), _ptr(k_pool), _ptr(v_pool), _dt(out, "attention"),
         _ptr(block_table), block_table.shape[1], _ptr(batch.seq_slot), _ptr(batch.seq_pos0),
         _ptr(batch.seq_qstart), _ptr(batch.seq_qlen), _ptr(gate), gate_stride, gate_elem, M, batch.n_seqs, nh, nkv,
-        hd, page_size, window, chunk, float(scale), batch.max_qlen, n_splits, vd, _stream()))
+        hd, page_size, window, chunk, float(scale), _ptr(slopes), _ptr(sinks), batch.max_qlen, n_splits, vd, _stream()))
 
 
 def _attention_decode_raw(out, raw: RawQKV, k_pool, v_pool, block_table, batch, nh, nkv, hd, page_size, window,
-                          scale, gate, n_splits, scratch, chunk=0, wide=False) -> None:
+                          scale, gate, n_splits, scratch, chunk=0, wide=False, slopes=None, sinks=None) -> None:
     M = out.shape[0]
     if not decode_attention_takes_raw(out.dtype, batch, M, nh, nkv, hd, page_size, raw.inv_freq, raw.rope_dim, raw.neox):
         raise KernelError("attention: this step's q, k and v must be normed, rotated and stored before the call")
@@ -1426,7 +1573,7 @@ def _attention_decode_raw(out, raw: RawQKV, k_pool, v_pool, block_table, batch, 
         if t is not None:
             _cuda(t, f"attention.{name}", torch.float32)
             assert not heads or t.numel() == (heads * hd if raw.row_norm else hd)
-    assert raw.inv_freq.numel() == hd // 2
+    assert raw.inv_freq is None or raw.inv_freq.numel() == hd // 2
     gate_stride, gate_elem = _gate_layout(gate, M, nh, hd, out.dtype)
     if n_splits > 1:
         need = M * nh * n_splits * (hd + 2)
@@ -1438,10 +1585,10 @@ def _attention_decode_raw(out, raw: RawQKV, k_pool, v_pool, block_table, batch, 
         _ptr(k_pool), _ptr(v_pool), _ptr(block_table), block_table.shape[1], _ptr(batch.seq_slot), _ptr(batch.seq_pos0),
         _ptr(batch.seq_qstart), _ptr(raw.q_norm_w), _ptr(raw.k_norm_w), raw.eps, _ptr(raw.inv_freq), raw.rope_dim,
         1 if raw.neox else 0, int(raw.row_norm), _ptr(gate), gate_stride, gate_elem, batch.n_seqs, nh, nkv, hd, page_size, window,
-        chunk, int(wide), float(scale), n_splits, _stream()))
+        chunk, int(wide), float(scale), _ptr(slopes), _ptr(sinks), *_temperature(raw.temperature), n_splits, _stream()))
     if n_splits > 1:
-        _check(L.leb_attention_merge(_ptr(out), _ptr(scratch), BF16, _ptr(gate), gate_stride, gate_elem, M, nh, hd, n_splits,
-                                     _stream()))
+        _check(L.leb_attention_merge(_ptr(out), _ptr(scratch), BF16, _ptr(gate), gate_stride, gate_elem, _ptr(sinks), M, nh, hd,
+                                     n_splits, _stream()))
 
 
 # ----------------------------------------------------------------------------------------------
@@ -1665,15 +1812,18 @@ def moe_align(offsets: torch.Tensor, sorted_pair: torch.Tensor, pair_row: torch.
     _check(lib().leb_moe_align(_ptr(offsets), _ptr(sorted_pair), _ptr(pair_row), _ptr(topk_ids), P_, E, _stream()))
 
 
-def moe_combine(x: torch.Tensor, ys: torch.Tensor, pair_row: torch.Tensor, topk_w: torch.Tensor,
-                accumulate: bool) -> None:
+def moe_combine(x: torch.Tensor, ys: torch.Tensor, pair_row: torch.Tensor, topk_w: torch.Tensor | None,
+                accumulate: bool, k: int | None = None) -> None:
+    """x (+)= the weighted sum of every row's k expert results; `topk_w` None (with `k`): their plain sum."""
     _cuda(x, "moe_combine.x", torch.float32)
     _cuda(ys, "moe_combine.ys", torch.float32)
     _cuda(pair_row, "moe_combine.pair_row", torch.int32)
-    _cuda(topk_w, "moe_combine.topk_w", torch.float32)
     M, D = x.shape
-    k = topk_w.shape[1]
-    assert ys.shape[1] == D and ys.shape[0] >= M * k and topk_w.shape[0] == M
+    if topk_w is not None:
+        _cuda(topk_w, "moe_combine.topk_w", torch.float32)
+        assert topk_w.shape[0] == M
+        k = topk_w.shape[1]
+    assert k is not None and ys.shape[1] == D and ys.shape[0] >= M * k and pair_row.numel() >= M * k
     _check(lib().leb_moe_combine(_ptr(x), _ptr(ys), _ptr(pair_row), _ptr(topk_w), M, D, k,
                                  1 if accumulate else 0, _stream()))
 

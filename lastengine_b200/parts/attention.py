@@ -22,11 +22,17 @@ hidden] (`output_gate="numbers"`); instead of a window the positions may be cut 
 sequence's first: a row reads its own chunk up to itself.  `wide_weights`: the softmax weights enter the bfloat16
 product with the values as two bfloat16 terms (16 significant bits) instead of one.
 
+More options: `values="keys"`: there is no value projection, a position's value is its key as it leaves the convolution
+(or the projection), before the norm; `slopes` (a number per head): slope_h (i - j) is taken off the scaled score of query
+i and key j; `sink`: a logit per head that takes its share of the softmax's denominator and stands for no position,
+learned ("learned", tensor `sink`) or a constant zero ("zero"); `query_temperature`
+(coef, every): the normed query at position p times 1 + coef ln(floor((p + 1) / every) + 1).
+
 Key and value heads of different widths are cached at the wider of the two when that is a size the
 tensor-core attention kernels take: the narrower heads are stored with zeros behind them (a zero
 dimension changes no score and adds nothing to a value; the scale is explicit and the norms run over
-the head as it is), and the output projection gets zero columns where the padding is.  Other pairs
-of widths run the general kernel.
+the head as it is), and the output projection gets zero columns where the padding is.  `widen=True` takes the next such size
+for heads of any width up to the largest.  Other widths run the general kernel.
 """
 from __future__ import annotations
 
@@ -47,7 +53,11 @@ class AttentionMixer(Mixer):
                  norm_eps: float, qk_norm: bool | str = True, position: PartSpec | None = None,
                  window: int = 0, output_gate: bool | str = False, own_kv: bool = True,
                  scale: float | None = None, v_head_dim: int | None = None, conv_taps: int = 0,
-                 v_norm: bool = False, names: dict[str, str] | None = None, chunk: int = 0, wide_weights: bool = False):
+                 v_norm: bool = False, names: dict[str, str] | None = None, chunk: int = 0, wide_weights: bool = False,
+                 values: str = "own", slopes: list[float] | None = None, sink: str | None = None,
+                 query_temperature: tuple[float, float] | None = None, widen: bool = False):
+        if values not in ("own", "keys") or sink not in (None, "zero", "learned"):
+            raise ValueError(f"values {values!r} ('own', 'keys') / sink {sink!r} (None, 'zero', 'learned')")
         if qk_norm not in (True, False, "unit", "row") or output_gate not in (True, False, "numbers"):
             raise ValueError(f"qk_norm {qk_norm!r} (True, False, 'unit', 'row') / output_gate {output_gate!r} (True, False, 'numbers')")
         if num_heads % num_kv_heads != 0:
@@ -65,15 +75,28 @@ class AttentionMixer(Mixer):
         # widths in the cache: the wider of the two where the fast kernels take it
         wide = max(self.hd, self.vd)
         self.khd, self.kvd = (wide, wide) if self.hd != self.vd and wide in (32, 64, 96, 128) else (self.hd, self.vd)
+        if widen and wide <= 128:
+            self.khd = self.kvd = -(-wide // 32) * 32
         self.taps = int(conv_taps)
         if not 0 <= self.taps <= 16:
             raise ValueError(f"conv_taps {conv_taps}: 0 (no convolution) or 1..16")
         if self.taps and not own_kv:
             raise ValueError("a layer that reads another layer's cache cannot convolve its own k and v")
         self.v_norm = bool(v_norm)
+        self.values_are_keys = values == "keys"
+        if self.values_are_keys and (self.vd != self.hd or not own_kv):
+            raise ValueError(f"values that are keys have their width ({self.hd}, not {self.vd}) and come with keys of the layer's own")
+        if slopes is not None and len(slopes) != num_heads:
+            raise ValueError(f"{len(slopes)} slopes for {num_heads} heads")
+        self.slope_values = None if slopes is None else [float(s) for s in slopes]
+        self.sink_kind = sink
+        self.temperature = None if query_temperature is None or float(query_temperature[0]) == 0.0 \
+            else (float(query_temperature[0]), float(query_temperature[1]))
+        if self.temperature is not None and not self.temperature[1] > 0:
+            raise ValueError(f"a query temperature rises every so many positions, got {query_temperature[1]}")
         self.n = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "out_proj.weight",
                   "gate": "gate_proj.weight", "q_norm": "q_layernorm.weight", "k_norm": "k_layernorm.weight",
-                  "q_conv": "q_conv.weight", "k_conv": "k_conv.weight", "v_conv": "v_conv.weight"}
+                  "q_conv": "q_conv.weight", "k_conv": "k_conv.weight", "v_conv": "v_conv.weight", "sink": "sink"}
         self.n.update(names or {})
         self.window, self.chunk, self.wide = int(window), int(chunk), bool(wide_weights)
         self.output_gate, self.gate_numbers = bool(output_gate), output_gate == "numbers"
@@ -83,7 +106,9 @@ class AttentionMixer(Mixer):
         self.scale = float(scale) if scale is not None else 1.0 / math.sqrt(self.hd)
         pos = position or PartSpec("none")
         self.position = POSITION_ENCODINGS.get(pos.kind)(**pos.params)
-        self.w_in = self.w_out = self.q_norm_w = self.k_norm_w = None
+        if self.temperature is not None and (self.qk_row or pos.kind not in ("none", "rope")):
+            raise NotImplementedError("a query temperature beside norms over whole rows or an encoding that is no rotation")
+        self.w_in = self.w_out = self.q_norm_w = self.k_norm_w = self.slopes = self.sinks = None
         self.n_extra, self.extra_out = 0, None
 
     def tensors(self) -> dict[str, TensorSpec]:
@@ -92,7 +117,10 @@ class AttentionMixer(Mixer):
              n["o"]: TensorSpec((D, nh * vd), MATRIX)}
         if self.own_kv:
             t[n["k"]] = TensorSpec((nkv * hd, D), MATRIX)
-            t[n["v"]] = TensorSpec((nkv * vd, D), MATRIX)
+            if not self.values_are_keys:
+                t[n["v"]] = TensorSpec((nkv * vd, D), MATRIX)
+        if self.sink_kind == "learned":
+            t[n["sink"]] = TensorSpec((nh,), VECTOR, std=1.0)
         if self.qk_norm:
             t[n["q_norm"]] = TensorSpec((nh * hd if self.qk_row else hd,), NORM)
             if self.own_kv:
@@ -102,7 +130,8 @@ class AttentionMixer(Mixer):
         if self.taps:
             t[n["q_conv"]] = TensorSpec((nh * hd, self.taps), VECTOR, std=0.5)
             t[n["k_conv"]] = TensorSpec((nkv * hd, self.taps), VECTOR, std=0.5)
-            t[n["v_conv"]] = TensorSpec((nkv * vd, self.taps), VECTOR, std=0.5)
+            if not self.values_are_keys:
+                t[n["v_conv"]] = TensorSpec((nkv * vd, self.taps), VECTOR, std=0.5)
         for name, spec in self.position.tensors().items():
             t[f"position.{name}"] = spec
         return t
@@ -112,13 +141,17 @@ class AttentionMixer(Mixer):
         if self.taps <= 1:       # a single tap looks at the current row only
             return kv
         # the convolution's memory: the last taps-1 projected values of every q, k and v channel
-        return kv, StateSpec(((self.nh + self.nkv) * self.hd + self.nkv * self.vd, self.taps - 1), torch.float32)
+        return kv, StateSpec((self._n_qkv(), self.taps - 1), torch.float32)
+
+    def _n_qkv(self) -> int:
+        """Projected numbers of a row: q, k and, where they have a projection, v."""
+        return (self.nh + self.nkv) * self.hd + (0 if self.values_are_keys else self.nkv * self.vd)
 
     def load(self, tensors, env: BuildEnv) -> None:
         n = self.n
         parts = [tensors[n["q"]]]
         if self.own_kv:
-            parts += [tensors[n["k"]], tensors[n["v"]]]
+            parts += [tensors[n["k"]]] + ([] if self.values_are_keys else [tensors[n["v"]]])
         if self.output_gate:
             parts.append(self._cached_width(tensors[n["gate"]], 0) if self.gate_numbers else tensors[n["gate"]])
         self.w_in = torch.cat(parts, dim=0).contiguous() if len(parts) > 1 else parts[0].contiguous()
@@ -132,8 +165,13 @@ class AttentionMixer(Mixer):
             self.q_norm_w = self.k_norm_w = torch.ones(self.hd, dtype=torch.float32, device=env.device)
         self.w_conv = None
         if self.taps:
-            self.w_conv = torch.cat([tensors[n["q_conv"]], tensors[n["k_conv"]], tensors[n["v_conv"]]],
-                                    dim=0).to(torch.float32).contiguous()
+            convs = [tensors[n["q_conv"]], tensors[n["k_conv"]]] + ([] if self.values_are_keys else [tensors[n["v_conv"]]])
+            self.w_conv = torch.cat(convs, dim=0).to(torch.float32).contiguous()
+        if self.slope_values is not None:
+            self.slopes = torch.tensor(self.slope_values, dtype=torch.float32, device=env.device)
+        if self.sink_kind is not None:
+            self.sinks = tensors[n["sink"]].to(torch.float32).contiguous() if self.sink_kind == "learned" \
+                else torch.zeros(self.nh, dtype=torch.float32, device=env.device)
         self.position.load({n[len("position."):]: v for n, v in tensors.items() if n.startswith("position.")}, env)
 
     def _cached_width(self, w: torch.Tensor, dim: int) -> torch.Tensor:
@@ -181,8 +219,8 @@ class AttentionMixer(Mixer):
         col = nh * hd
         if writes:
             k_in = proj[:, col: col + nkv * hd]
-            v_in = proj[:, col + nkv * hd: col + nkv * (hd + vd)]
-            col += nkv * (hd + vd)
+            v_in = k_in if self.values_are_keys else proj[:, col + nkv * hd: col + nkv * (hd + vd)]
+            col = self._n_qkv()
         if self.output_gate:
             gate = proj[:, col: col + self.n_gate]
         if self.n_extra:
@@ -194,7 +232,7 @@ class AttentionMixer(Mixer):
             conv = ws.get("attn.conv", (M, col), env.dtype)
             kernels.causal_conv(conv, proj[:, :col], self.w_conv, cache.state, batch)
             q_in, k_in = conv[:, : nh * hd], conv[:, nh * hd: (nh + nkv) * hd]
-            v_in = conv[:, (nh + nkv) * hd:]
+            v_in = k_in if self.values_are_keys else conv[:, (nh + nkv) * hd:]
         khd, kvd = self.khd, self.kvd
         q = ws.get("attn.q", (M, nh * khd), env.dtype)
         kp, vp = (cache.k, cache.v) if writes else (None, None)
@@ -204,7 +242,7 @@ class AttentionMixer(Mixer):
                 and kernels.decode_attention_takes_raw(env.dtype, batch, M, nh, nkv, hd, cache.page_size, *rotary)):
             # a decode step: the attention kernel norms and rotates q and k and stores k and v itself
             raw = kernels.RawQKV(q_in, k_in, v_in, self.q_norm_w, self.k_norm_w if writes else None, self.eps, *rotary,
-                                 row_norm=self.qk_row)
+                                 row_norm=self.qk_row, temperature=self.temperature)
         elif self.qk_row:
             if rotary is None or not writes:
                 raise NotImplementedError("norms over whole rows with a position encoding that is no rotation, or another layer's cache")
@@ -214,7 +252,7 @@ class AttentionMixer(Mixer):
             # per-head norm, rotation and the cache write in one launch
             kernels.qk_rope_store(q, q_in, k_in, v_in, kp, vp, cache.block_table, batch, self.q_norm_w,
                                   self.k_norm_w if writes else None, self.eps, *rotary, nh, nkv, khd, cache.page_size,
-                                  vd=kvd, v_norm=self.v_norm, hd_in=hd, vd_in=vd)
+                                  vd=kvd, v_norm=self.v_norm, hd_in=hd, vd_in=vd, temperature=self.temperature)
         elif not plain_v:
             raise NotImplementedError("value heads of their own width or norm with a position encoding that is no rotation")
         else:
@@ -234,12 +272,12 @@ class AttentionMixer(Mixer):
             kernels.qk_rope_store(q, qn, kn, vn, kp, vp, cache.block_table, batch, None, None, self.eps,
                                   None, 0, True, nh, nkv, hd, cache.page_size)
         o = ws.get("attn.o", (M, nh * kvd), env.dtype)
-        n_splits = kernels.attention_splits(batch, nkv, nh // nkv, hd=khd, chunk=self.chunk)
+        n_splits = kernels.attention_splits(batch, nkv, nh // nkv, hd=khd, chunk=self.chunk, window=self.window)
         scratch = None
         if n_splits > 1:
             scratch = ws.get("attn.part", (M * nh * n_splits * (max(khd, kvd) + 2),), torch.float32)
         kernels.attention(o, None if raw is not None else q, cache.k, cache.v, cache.block_table, batch, nh, nkv, khd,
                           cache.page_size, self.window, self.scale, gate=gate, n_splits=n_splits, scratch=scratch, raw=raw,
-                          vd=kvd, chunk=self.chunk, wide=self.wide)
+                          vd=kvd, chunk=self.chunk, wide=self.wide, slopes=self.slopes, sinks=self.sinks)
         kernels.linear(out, o, self.w_out, kernels.ACCUMULATE if accumulate else kernels.STORE,
                        emit=emit if accumulate else None)

@@ -22,6 +22,9 @@ FeedForward:
     forward(h, out, accumulate, batch, env)
 Norm:
     forward(out, x, rows=None, add=False)          x float; out in any activation dtype
+Embedding:
+    forward(x, tokens, batch=...)                  x: float [rows, hidden], written.  One that keeps state per sequence has
+                                                   a cache_spec() and gets its view as `cache=`
 PositionEncoding:
     fused_rotary() -> (inv_freq, rope_dim, neox)   a rotation that the mixer's kernel applies itself
                       | None                       while it norms q and k and stores k and v, or
@@ -139,12 +142,14 @@ class LayerSpec:
 
 @dataclass(frozen=True)
 class StreamAdd:
-    """Something added to the residual stream right before a schedule entry runs: the embedding
-    output (the stream as it was before the first entry) and/or one row of a model-wide table."""
+    """What happens to the residual stream right before a schedule entry runs: the embedding output (the stream
+    as it was before the first entry) and/or one row of a model-wide table is added; with `matrix` the stream first
+    becomes W [stream ; embedding output], and the row is added to that."""
     before: int                    # index into the schedule
     embedding: bool = False
     table: str | None = None       # canonical tensor name of a [rows, hidden] table
     row: int = 0
+    matrix: str | None = None      # canonical tensor name of a [hidden, 2 hidden] matrix
 
 
 @dataclass(frozen=True)
@@ -180,6 +185,7 @@ class ModelPlan:
                                            # model has no use for (an optional tensor of a part no layer has): skipped
     stream_adds: tuple[StreamAdd, ...] = ()     # additions to the residual stream between schedule entries
     stream_tables: dict[str, tuple[int, ...]] = field(default_factory=dict)   # canonical name -> shape of their tables
+    stream_matrices: dict[str, tuple[int, ...]] = field(default_factory=dict)   # canonical name -> shape of their matrices
     max_positions: int | None = None   # the longest sequence the model takes (a table of learned positions); None: no limit
     checkpoint_names: Any = None   # callable: canonical name -> name in a checkpoint (the inverse of
                                    # tensor_aliases; None: "model." in front of everything but the head)
@@ -200,6 +206,9 @@ class ModelPlan:
             if a.table is not None and (a.table not in self.stream_tables
                                         or not 0 <= a.row < self.stream_tables[a.table][0]):
                 raise ValueError(f"a stream addition names row {a.row} of '{a.table}', which the plan does not declare")
+            if a.matrix is not None and (a.embedding or self.stream_matrices.get(a.matrix) != (self.hidden_size, 2 * self.hidden_size)):
+                raise ValueError(f"a stream addition names the matrix '{a.matrix}', which the plan does not declare as "
+                                 f"[hidden, 2 hidden] (or adds the embedding output beside it)")
 
 
 @dataclass

@@ -3,8 +3,10 @@
 parallel_residual (further down): x += mult * (Mixer(norm(x)) + FeedForward(norm(x))), with one norm for both
 sublayers or one each.
 
-post_norm_residual and output_norm_residual (at the end): the sublayers read the stream itself, and the norm comes
+post_norm_residual and output_norm_residual: the sublayers read the stream itself, and the norm comes
 after each sum, or on each sublayer's result before its sum.
+
+sandwich_norm_residual (at the end): pointwise norms on what each sublayer reads and on what it gives.
 
 pre_norm_residual (src/dense.rs:178-194):
     x += [post_norm](Mixer(norm(x)));  x += [post_norm](FeedForward(norm(x)))
@@ -365,3 +367,59 @@ class OutputNormResidualBlock(PostNormResidualBlock):
 
     def _sum(self, x, y, norm, h) -> None:
         kernels.outnorm_residual(x, y, norm.weight, norm.eps, h=h)
+
+
+@BLOCKS.register("sandwich_norm_residual")
+class SandwichNormResidualBlock:
+    """x <- x + n1'(Mixer(n1(x)));  x <- x + n2'(FeedForward(n2(x))): a norm on what each sublayer reads and one on what it
+    gives, pointwise norms (parts.norm.DynamicTanh) throughout.  A layer may have no feed-forward: it then ends after
+    the first sum.  The stream, the sums and the norms are float.  One launch norms a sublayer's result, adds it to the
+    stream and leaves the next sublayer's normed input (in this block, or the first of the next block when that is of
+    this arrangement too and nothing happens to the stream in between).  A mixer that ends in a weighted sum of two
+    results (`forward_parts`) leaves that sum to the same launch."""
+
+    def __init__(self, mixer, ffn, mixer_norm, ffn_norm=None, post_mixer_norm=None, post_ffn_norm=None):
+        from .norm import DynamicTanh
+        if post_mixer_norm is None or (ffn is None) != (ffn_norm is None) or (ffn is None) != (post_ffn_norm is None):
+            raise ValueError("every sublayer of the sandwich arrangement comes with two norms")
+        for n in (mixer_norm, ffn_norm, post_mixer_norm, post_ffn_norm):
+            if n is not None and not isinstance(n, DynamicTanh):
+                raise ValueError("the sandwich arrangement takes pointwise norms")
+        self.mixer, self.ffn, self.mixer_norm, self.ffn_norm = mixer, ffn, mixer_norm, ffn_norm
+        self.post_mixer_norm, self.post_ffn_norm = post_mixer_norm, post_ffn_norm
+
+    def parts(self) -> dict[str, object]:
+        p = {"mixer": self.mixer, "mixer_norm": self.mixer_norm, "post_mixer_norm": self.post_mixer_norm}
+        if self.ffn is not None:
+            p["ffn"], p["ffn_norm"], p["post_ffn_norm"] = self.ffn, self.ffn_norm, self.post_ffn_norm
+        return p
+
+    def first_reader(self):
+        return self.mixer_norm, self
+
+    def forward(self, x: torch.Tensor, batch, cache, env, pending=None):
+        M, D = x.shape
+        ws = env.workspace
+        env.split_in = env.split_out = None
+        if isinstance(pending, NormedRows) and pending.norm is self.mixer_norm and pending.values.shape == (M, D):
+            h = pending.values
+        else:
+            h = ws.get("block.h", (M, D), env.dtype)
+            self.mixer_norm.forward(h, x)
+        other = ws.get("block.h2" if h is ws.get("block.h", (M, D), env.dtype) else "block.h", (M, D), env.dtype)
+        nxt = env.next_block_norm
+        after = nxt[0] if nxt is not None and isinstance(nxt[1], SandwichNormResidualBlock) else None
+        follows = self.ffn_norm if self.ffn is not None else after
+        if hasattr(self.mixer, "forward_parts"):
+            y, a, y2, b = self.mixer.forward_parts(h, batch, cache, env)
+            weighted = (a, y2, b)
+        else:
+            y, weighted = ws.get("block.t", (M, D), torch.float32), None
+            self.mixer.forward(h, y, False, batch, cache, env)
+        self.post_mixer_norm.add_into(x, y, follows, other if follows is not None else None, weighted)
+        if self.ffn is None:
+            return NormedRows(other, after) if after is not None else None
+        y = ws.get("block.t", (M, D), torch.float32)
+        self.ffn.forward(other, y, False, batch, env)
+        self.post_ffn_norm.add_into(x, y, after, h if after is not None else None)
+        return NormedRows(h, after) if after is not None else None

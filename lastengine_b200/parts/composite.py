@@ -92,7 +92,18 @@ class ParallelMixers(Mixer):
         return view
 
     def forward(self, h, out, accumulate, batch, cache, env) -> None:
-        M, D = out.shape
+        y1, a, y2, b, bias = self._run(h, batch, cache, env)
+        kernels.weighted_pair_sum(out, y1, a, y2, b, bias1=bias, accumulate=accumulate)
+
+    def forward_parts(self, h, batch, cache, env):
+        """(y1, a, y2, b): the two children's float results and their weights, for whoever forms a y1 + b y2 in a launch of its own."""
+        y1, a, y2, b, bias = self._run(h, batch, cache, env)
+        if bias is not None:
+            kernels.add_row_vector(y1, bias)
+        return y1, a, y2, b
+
+    def _run(self, h, batch, cache, env):
+        M, D = h.shape
         ws = env.workspace
         y1 = ws.get("pair.left", (M, D), torch.float32)
         y2 = ws.get("pair.right", (M, D), torch.float32)
@@ -108,4 +119,4 @@ class ParallelMixers(Mixer):
         self.right.forward(h, y2, False, batch, self._view(cache, 1), env, **kr)
         if getattr(self.right, "output_bias", lambda: None)() is not None:
             raise NotImplementedError("an output bias on the right-hand mixer")
-        kernels.weighted_pair_sum(out, y1, self.a, y2, self.b, bias1=bias, accumulate=accumulate)
+        return y1, self.a, y2, self.b, bias

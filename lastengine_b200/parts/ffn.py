@@ -143,6 +143,8 @@ class SigmoidTopKMoE(FeedForward):
     `router="sigmoid_grouped"` with `groups=(count, keep)` and `group_top`: sigmoid scores, the bias only chooses,
     groups as above but a group's score is the sum of its `group_top` largest choice scores; weights are the
     chosen s over their sum (+ 1e-20), times `scaling`.
+    `router="sigmoid"` with `norm_topk=False`: weights are the chosen sigmoids themselves.
+    `weight_input=True`: y = sum_e expert_e(w_e h), experts that see their weighted rows (default: sum_e w_e expert_e(h)).
     `gated=False`: experts of the plain shape W_down act(W_up h) (no gate tensors) with `activation` one of
     "gelu" (erf form), "relu_squared", "gelu_tanh", "silu".
     `shared_size` > 0: one more expert of that width and the same activation runs for every row and is added
@@ -154,7 +156,7 @@ class SigmoidTopKMoE(FeedForward):
                  bias_std: float = 0.1, router: str = "sigmoid", activation: str = "silu",
                  limit: float = 0.0, alpha: float = 1.0, names: dict[str, str] | None = None,
                  groups: tuple[int, int] | None = None, shared_size: int = 0, gated: bool = True,
-                 group_top: int = 1):
+                 group_top: int = 1, weight_input: bool = False):
         if not 1 <= top_k <= min(num_experts, 16):
             raise ValueError(f"top-{top_k} of {num_experts} experts: the router takes 1..min(experts, 16)")
         if num_experts > 256:
@@ -166,6 +168,7 @@ class SigmoidTopKMoE(FeedForward):
         if not 1 <= self.group_top <= 15:
             raise ValueError(f"a group is ranked by its 1..15 best scores, got {group_top}")
         self.gated = bool(gated)
+        self.weight_input = bool(weight_input)
         if router in ("softmax_grouped", "sigmoid_grouped"):
             count, keep = (int(groups[0]), int(groups[1])) if groups is not None else (1, 1)
             if not (1 <= keep <= count <= 255 and num_experts % count == 0 and keep * (num_experts // count) >= top_k):
@@ -256,7 +259,7 @@ class SigmoidTopKMoE(FeedForward):
         pair_row = ws.get("moe.rows", (P,), torch.int32)
         kernels.moe_align(offsets, sorted_pair, pair_row, ids, self.E)
         xs = ws.get("moe.xs", (P, self.D), env.dtype)
-        kernels.gather_rows(xs, h, sorted_pair, div=self.k)
+        kernels.gather_rows(xs, h, sorted_pair, div=self.k, weights=wts if self.weight_input else None)
         a = ws.get("moe.a", (P, self.Fe), env.dtype)
         if not self.gated and kernels.takes_plain_act(xs, self.w13, n_groups=self.E):
             kernels.linear(a, xs, self.w13, kernels.plain_act_epilogue(self.act), group_offsets=offsets, rows_hint=P)
@@ -275,6 +278,6 @@ class SigmoidTopKMoE(FeedForward):
                 kernels.gated_act(a, gu, self.act, self.limit, self.alpha)
         ys = ws.get("moe.ys", (P, self.D), torch.float32)
         kernels.linear(ys, a, self.w2, group_offsets=offsets, rows_hint=P)
-        kernels.moe_combine(out, ys, pair_row, wts, accumulate)
+        kernels.moe_combine(out, ys, pair_row, None if self.weight_input else wts, accumulate, k=self.k)
         if self.shared is not None:
             self.shared.forward(h, out, True, batch, env)

@@ -37,9 +37,6 @@ from ..registry import MIXERS, POSITION_ENCODINGS
 from .base import MATRIX, NORM, VECTOR, BuildEnv, LatentSpec, Mixer, PartSpec, TensorSpec
 
 
-_HEAD_OFFSETS: dict[tuple, torch.Tensor] = {}
-
-
 def _up8(n: int) -> int:
     return -(-n // 8) * 8
 
@@ -134,15 +131,6 @@ class LatentAttentionMixer(Mixer):
     def flops_per_query_key(self) -> int:
         return 2 * self.H * (2 * self.rank + self.rd)   # a score over the cached row and a weighted sum of its latent
 
-    def _head_offsets(self, M: int, device) -> torch.Tensor:
-        """Row ranges of the head-major buffers for the grouped products: head h owns rows [h M, (h + 1) M).
-        Made once per (heads, rows) and kept for good (a few bytes each): captured steps hold their addresses."""
-        key = (self.H, M, str(device))
-        t = _HEAD_OFFSETS.get(key)
-        if t is None:
-            t = _HEAD_OFFSETS[key] = (torch.arange(self.H + 1, dtype=torch.int64) * M).to(torch.int32).to(device)
-        return t
-
     def forward(self, h, out, accumulate, batch, cache, env) -> None:
         H, hd, rd, vd, rank = self.H, self.hd, self.rd, self.vd, self.rank
         M = h.shape[0]
@@ -167,7 +155,7 @@ class LatentAttentionMixer(Mixer):
         else:
             kernels.latent_rows(qn, qr, proj, pool if writes else None, cache.block_table, batch, self.kv_norm_w, self.eps,
                                 self.inv_freq, self.rot_dims, self.neox, H, hd, rank, rd, cache.page_size)
-        offsets = self._head_offsets(M, h.device)
+        offsets = kernels.equal_group_offsets(H, M, h.device)     # of the head-major buffers
         qt = ws.get("lat.qt", (H, M, rank), env.dtype)
         kernels.linear(qt.view(H * M, rank), qn.view(H * M, self.hd_p), self.w_ukt, group_offsets=offsets, rows_hint=H * M)
         u = ws.get("lat.u", (H, M, self.rank_p), env.dtype)
