@@ -25,7 +25,7 @@ A step is one decode step of the whole batch.  One JSON line goes to stdout:
 
 Weights (1.8 GB) are far larger than L2, so consecutive steps cannot be served from L2.
 
-`--compare zekivik` (or `lenesun`, `kisilix`, `tevilix`, `zafilix`) leaves all of that aside and prints a line of its own: prompt and decode times
+`--compare zekivik` (or `lenesun`, `kisilix`, `tevilix`, `zafilix`, `nolapel`) leaves all of that aside and prints a line of its own: prompt and decode times
 of that design at a few layer sizes beside the closest LFM3 model at equal sizes, with every kernel entry point's time.
 """
 from __future__ import annotations
@@ -445,7 +445,11 @@ def _kisilix_kernel_work(cfg: dict, rows: int, batch: int, context: int) -> dict
         m = l["mixer"]
         n_sub = 2 if l["mlp"] else 1
         by["leb_postnorm_residual"] += n_sub * rows * W * (4 + 4 + 4 + 2)            # x and y read (float), x and its bfloat16 copy written
-        if l["mlp"]:
+        if l["mlp"] and l["mlp"]["kind"] == "moe":
+            top = l["mlp"]["router"]["top"]
+            by["leb_gather_rows"] = by.get("leb_gather_rows", 0) + rows * top * W * 4
+            by["leb_moe_combine"] = by.get("leb_moe_combine", 0) + rows * (top + 1) * W * 4
+        elif l["mlp"]:
             by["leb_gated_act"] += rows * l["mlp"]["ff"] * (8 + 2)
         if l["type"] == "attention":
             nh, nkv, hd, vd = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
@@ -583,6 +587,101 @@ def _zafilix_kernel_work(cfg: dict, rows: int, batch: int, context: int) -> dict
     return {"bytes": by, "attention_flops": att, "latent_flops": lat}
 
 
+# ---- the Nolapel design beside the Kisilix design and LFM3 attention layers (--compare nolapel) -------------------
+def nolapel_config(width: int, heads: int, kv_heads: int, dim: int, window: int, mix_heads: int, mix_dim: int, ssm_heads: int,
+                   ssm_vdim: int, ssm_state: int, ssm_groups: int, experts: int, top: int, ff: int, shared: int, layers: int,
+                   vocab: int) -> dict:
+    """Side-by-side layers (causal attention with a sink beside time mixing), state-space layers and windowed attention
+    layers in turn, every layer with experts; the second half runs as a loop of one pass, so the stream goes through
+    the product with the embedding output once."""
+    par = {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                    "rot": {"dims": dim, "base": 1000000.0}}, "left_scale": 0.75,
+           "right": {"heads": mix_heads, "dim": mix_dim}, "right_scale": 1.25}
+    ssm = {"heads": ssm_heads, "vdim": ssm_vdim, "state": ssm_state, "groups": ssm_groups, "norm_groups": ssm_groups, "conv": 4}
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "conv": 4, "scale": dim ** -0.5, "mask": {"size": window},
+           "q_temp": {"coef": 0.1, "every": 512}}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff}, "shared": {"ff": shared}}
+    kinds = (("parallel", par), ("mamba2", ssm), ("attention", att))
+    return {"architecture": "Nolapel", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 131, "mul_cur": 17}},
+            "loop": {"start": layers // 2, "stop": layers, "times": 1},
+            "layers": [{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1], "mlp": moe} for i in range(layers)]}
+
+
+def kisilix_moe_like(width: int, heads: int, kv_heads: int, dim: int, window: int, mix_heads: int, mix_dim: int, ssm_heads: int,
+                     ssm_vdim: int, ssm_state: int, ssm_groups: int, experts: int, top: int, ff: int, shared: int, layers: int,
+                     vocab: int) -> dict:
+    """The closest design layer for layer: the delta rule where the other has side-by-side mixers (a recurrence with a
+    decay per key channel at the same head sizes), the same state-space layers, windowed attention, the same experts."""
+    dlt = {"heads": mix_heads, "kv_heads": mix_heads, "dim": mix_dim, "vdim": mix_dim, "conv": 4}
+    ssm = {"heads": ssm_heads, "vdim": ssm_vdim, "state": ssm_state, "groups": ssm_groups, "norm_groups": ssm_groups, "conv": 4}
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+           "rot": {"dims": dim, "base": 1000000.0}, "mask": {"size": window, "pool": 4096}}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff}, "shared": {"ff": shared}}
+    kinds = (("channel_delta", dlt), ("mamba2", ssm), ("attention", att))
+    return {"architecture": "Kisilix", "vocab": vocab, "width": width, "max_positions": 4096, "norm": {"eps": 1e-5},
+            "postln_alpha": 1.0, "layers": [{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1], "mlp": moe} for i in range(layers)]}
+
+
+NOLAPEL_SIZES = {
+    "w2048": dict(width=2048, heads=32, kv_heads=8, dim=64, window=1024, mix_heads=32, mix_dim=64, ssm_heads=64, ssm_vdim=64,
+                  ssm_state=128, ssm_groups=8, experts=32, top=4, ff=512, shared=1024, layers=6),
+    "w1024": dict(width=1024, heads=16, kv_heads=4, dim=64, window=512, mix_heads=16, mix_dim=64, ssm_heads=32, ssm_vdim=64,
+                  ssm_state=64, ssm_groups=1, experts=16, top=2, ff=512, shared=512, layers=6),
+    "w2048-d128": dict(width=2048, heads=16, kv_heads=4, dim=128, window=1024, mix_heads=16, mix_dim=128, ssm_heads=32, ssm_vdim=128,
+                       ssm_state=128, ssm_groups=4, experts=32, top=1, ff=1024, shared=2048, layers=6),
+}
+
+
+def _nolapel_kernel_work(cfg: dict, rows: int, batch: int, context: int) -> dict:
+    """What a step's launches of the design's own kernels have to move (bytes) or compute (flops), by entry point; the
+    rows of a sequence are its last ones, ending at `context`."""
+    W = cfg["width"]
+    by = {"leb_embed_pairs": rows * W * (2 + 2 + 4), "leb_pointwise_norm": rows * W * 6, "leb_pointwise_norm_sum": 0,
+          "leb_stream_columns": rows * W * (6 + 10), "leb_row_shift_mix": 0, "leb_low_rank_decay": 0, "leb_gated_recurrence": 0,
+          "leb_group_norm_gate": 0, "leb_causal_conv": 0, "leb_ssm_prep": 0, "leb_qk_rope_store": 0, "leb_gather_rows": 0,
+          "leb_moe_combine": 0, "leb_softcap": batch * cfg["vocab"] * 8, "attention": 0}
+    fl = {"attention": 0, "leb_gated_recurrence": 0}
+    per_seq = rows // batch
+    at = range(context - per_seq, context)
+    for l in cfg["layers"]:
+        m, f = l["mixer"], l["mlp"]
+        by["leb_pointwise_norm_sum"] += 2 * rows * W * (4 + 4 + 4 + 2)         # x and the result read, x and the next norm written
+        by["leb_gather_rows"] += rows * f["router"]["top"] * W * 4
+        by["leb_moe_combine"] += rows * (f["router"]["top"] + 1) * W * 4
+        if l["type"] == "mamba2":
+            H, e, N, G = m["heads"], m["vdim"], m["state"], m["groups"]
+            C = H * e + 2 * G * N
+            by["leb_causal_conv"] += rows * C * 8 + batch * C * (m["conv"] - 1) * 8
+            by["leb_ssm_prep"] += rows * (2 * C + 3 * H) * 4
+            by["leb_gated_recurrence"] += rows * (2 * G * N + 2 * H * e + 2 * H) * 4 + batch * H * N * e * 8
+            fl["leb_gated_recurrence"] += rows * H * N * e * 6
+            by["leb_group_norm_gate"] += rows * H * e * (4 + 4 + 2)
+            continue
+        a = m["left"] if l["type"] == "parallel" else m
+        nh, nkv, hd = a["heads"], a["kv_heads"], a["dim"]
+        win = (a.get("mask") or {}).get("size", context)
+        fl["attention"] += 4 * nh * hd * batch * sum(min(i + 1, win) for i in at)
+        by["attention"] += batch * min(context, win) * nkv * 2 * hd * 2
+        n_in = (nh + nkv) * hd + (0 if l["type"] == "attention" else nkv * hd)
+        by["leb_qk_rope_store"] += rows * (n_in * 2 + (nh + 2 * nkv) * hd * 2)
+        if l["type"] == "attention":
+            by["leb_causal_conv"] += rows * n_in * 4 + batch * n_in * (m["conv"] - 1) * 8
+        else:
+            H, d = m["right"]["heads"], m["right"]["dim"]
+            by["leb_pointwise_norm_sum"] += rows * W * 4                       # the second mixer's result
+            by["leb_row_shift_mix"] += rows * W * (2 + 5 * 2) + batch * W * 8
+            by["leb_low_rank_decay"] += rows * H * d * 4
+            by["leb_gated_recurrence"] += rows * H * d * 5 * 4 + batch * H * d * d * 8
+            fl["leb_gated_recurrence"] += rows * H * d * d * 8
+            by["leb_group_norm_gate"] += rows * H * d * (4 + 4 + 2)
+    for name in ("leb_attention_decode", "leb_attention_decode_prep"):
+        by[name] = by["attention"]
+    for name in ("leb_attention_prefill_tc", "leb_attention_prefill"):
+        fl[name] = fl["attention"]
+    return {"bytes": by, "flops": fl}
+
+
 def compare_designs(which: str, steps: int, warmup: int) -> int:
     import numpy as np
     import torch
@@ -591,11 +690,14 @@ def compare_designs(which: str, steps: int, warmup: int) -> int:
     pk, pk_src = peaks()
     rng = np.random.default_rng(0)
     results = {}
-    other = "zekivik" if which == "kisilix" else ("kisilix" if which == "tevilix" else "lfm3")
+    other = "zekivik" if which == "kisilix" else ("kisilix" if which in ("tevilix", "nolapel") else "lfm3")
     for size_name, sz in {"zekivik": COMPARE_SIZES, "lenesun": LENESUN_SIZES, "kisilix": KISILIX_SIZES,
-                          "tevilix": KISILIX_SIZES, "zafilix": ZAFILIX_SIZES}[which].items():
+                          "tevilix": KISILIX_SIZES, "zafilix": ZAFILIX_SIZES, "nolapel": NOLAPEL_SIZES}[which].items():
         more = []
-        if which == "zafilix":
+        if which == "nolapel":
+            zc, lc = nolapel_config(vocab=32768, **sz), kisilix_moe_like(vocab=32768, **sz)
+            more = [("lfm3", lfm3_attention_like(sz["width"], sz["width"], sz["heads"], sz["kv_heads"], sz["dim"], sz["layers"], 32768))]
+        elif which == "zafilix":
             zc = zafilix_config(vocab=32768, **sz)
             lc = lfm3_attention_like(sz["width"], sz["ff"], sz["heads"], sz["kv_heads"], sz["dim"], sz["layers"], 32768)
             more = [("lenesun", lenesun_latent_like(sz["width"], sz["lat_heads"], sz["lat_dim"], sz["rot_dim"], sz["lat_vdim"],
@@ -621,7 +723,10 @@ def compare_designs(which: str, steps: int, warmup: int) -> int:
             print(f"[bench] {size_name} {label}: {r['weights_gb']} GB of weights", file=sys.stderr, flush=True)
             pre_ms = time_prefill(eng, PREFILL_TOKENS, 3, 5, rng)
             print(f"[bench] {size_name} {label}: prompt of {PREFILL_TOKENS} tokens {pre_ms:.3f} ms", file=sys.stderr, flush=True)
-            if label == "zafilix":      # a position sees its chunk or its window
+            if label == "nolapel":      # a position of the windowed layers sees its window
+                attn_flops = _nolapel_kernel_work(cfg, PREFILL_TOKENS, 1, PREFILL_TOKENS)["flops"]["attention"]
+                kv_seen = [_nolapel_kernel_work(cfg, 1, 1, 2048)["bytes"]["attention"]]
+            elif label == "zafilix":      # a position sees its chunk or its window
                 work = _zafilix_kernel_work(cfg, PREFILL_TOKENS, 1, PREFILL_TOKENS)
                 attn_flops = work["attention_flops"] + work["latent_flops"]
                 w1 = _zafilix_kernel_work(cfg, 1, 1, 2048)["bytes"]
@@ -670,7 +775,12 @@ def compare_designs(which: str, steps: int, warmup: int) -> int:
             eng.release(seqs)
             dec_k = t.summary()
             by, fl = {}, {}
-            if label == "zafilix":
+            if label == "nolapel":
+                wp, wd = _nolapel_kernel_work(cfg, PREFILL_TOKENS, 1, PREFILL_TOKENS), _nolapel_kernel_work(cfg, 8, 8, 2048)
+                by = {"prefill": {k: v for k, v in wp["bytes"].items() if k not in ("leb_attention_decode", "leb_attention_decode_prep")},
+                      "decode_b8": wd["bytes"]}
+                fl = {"prefill": wp["flops"]}
+            elif label == "zafilix":
                 wp, wd = _zafilix_kernel_work(cfg, PREFILL_TOKENS, 1, PREFILL_TOKENS), _zafilix_kernel_work(cfg, 8, 8, 2048)
                 by = {"prefill": {k: v for k, v in wp["bytes"].items() if k not in ("leb_latent_attention", "leb_attention_decode_prep")},
                       "decode_b8": dict(wd["bytes"], leb_attention_decode=wd["bytes"]["leb_attention_decode_prep"])}
@@ -723,6 +833,7 @@ def compare_designs(which: str, steps: int, warmup: int) -> int:
     against = {"zekivik": "lfm3 hybrid at equal layer sizes", "kisilix": "zekivik hybrid at equal layer sizes",
                "tevilix": "kisilix at equal layer sizes",
                "zafilix": "lfm3 with attention in every layer, and lenesun with latent attention alone, at equal layer sizes",
+               "nolapel": "kisilix with experts, and lfm3 with attention in every layer, at equal layer sizes",
                "lenesun": "lfm3 with attention and experts in every layer at equal layer sizes"}[which]
     print(json.dumps({"compare": which, "against": against, "dtype": "bf16",
                       "data": "synthetic (random weights, uniform random token ids)", "peaks": pk_src,
@@ -749,7 +860,7 @@ def main() -> int:
     ap.add_argument("--unequal", type=int, default=0, metavar="N",
                     help="instead of the default run: N requests with prompts of U[64, 2048] tokens generate "
                          "--steps tokens each in one batch through the Python entry point (prints its own JSON line)")
-    ap.add_argument("--compare", default="", choices=["", "zekivik", "lenesun", "kisilix", "tevilix", "zafilix"],
+    ap.add_argument("--compare", default="", choices=["", "zekivik", "lenesun", "kisilix", "tevilix", "zafilix", "nolapel"],
                     help="instead of the default run: prefill and decode of that design at a few layer sizes beside "
                          "the closest other design at equal sizes, with every kernel's time (prints its own JSON line)")
     args = ap.parse_args()
