@@ -126,5 +126,5 @@ def save_file(tensors: dict[str, torch.Tensor], path: str, metadata: dict[str, s
         f.write(blob)
         for name in order:
             t = tensors[name].detach().cpu().contiguous()
-            f.write(t.view(torch.uint8).reshape(-1).numpy().tobytes() if t.numel() else b"")
+            f.write(t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b"")
     os.replace(tmp, path)
