@@ -129,45 +129,72 @@ LEB_API int leb_row_shift_mix(void* mix, const void* h, int dtype, const float* 
 }
 
 // The decay of a recurrence from a low-rank pair: out[m, c] = exp(-exp(sum_j tanh(low[m, j]) w2[j, c] + w0[c])), all
-// float (w2 [rank, C], so that neighbouring threads read neighbouring numbers).  A block takes LRD_ROWS rows x 128
-// channels; the rows' tanh values stay in shared memory, a slab of ranks at a time.
-constexpr int LRD_ROWS = 8, LRD_SLAB = 64;
-template <int R>
+// float (w2 [rank, C], so that neighbouring threads read neighbouring numbers).  A block takes R rows x 128 VEC
+// channels, a thread VEC neighbouring ones; the rows' tanh values stay in shared memory, a slab of ranks at a time.
+constexpr int LRD_SLAB = 64;
+template <int R, int VEC>
 __global__ void __launch_bounds__(128)
 low_rank_decay_kernel(float* __restrict__ out, const float* __restrict__ low, int ldl, const float* __restrict__ w2,
                       const float* __restrict__ w0, int M, int C, int rank) {
-  __shared__ float ts[LRD_SLAB][R];
+  __shared__ __align__(16) float ts[LRD_SLAB][R];
   pdl_wait();
-  const int m0 = blockIdx.x * R, c = blockIdx.y * 128 + threadIdx.x;
-  float acc[R];
+  const int m0 = blockIdx.x * R, c = (blockIdx.y * 128 + threadIdx.x) * VEC;
+  float acc[R][VEC];
 #pragma unroll
-  for (int r = 0; r < R; r++) acc[r] = 0.f;
+  for (int r = 0; r < R; r++)
+#pragma unroll
+    for (int e = 0; e < VEC; e++) acc[r][e] = 0.f;
+  auto get = [&](float* o, const float* p) {
+    if (VEC == 4) {
+      const float4 v = load4(p);
+      o[0] = v.x; o[1 % VEC] = v.y; o[2 % VEC] = v.z; o[3 % VEC] = v.w;
+    } else {
+      o[0] = *p;
+    }
+  };
   for (int j0 = 0; j0 < rank; j0 += LRD_SLAB) {
     const int nj = min(LRD_SLAB, rank - j0);
     __syncthreads();
-    for (int idx = threadIdx.x; idx < R * LRD_SLAB; idx += 128) {
-      const int r = idx / LRD_SLAB, j = idx % LRD_SLAB;
-      if (j < nj) ts[j][r] = m0 + r < M ? tanhf(low[(size_t)(m0 + r) * ldl + j0 + j]) : 0.f;
+    for (int idx = threadIdx.x; idx < R * nj; idx += 128) {
+      const int r = idx / nj, j = idx - r * nj;
+      ts[j][r] = m0 + r < M ? tanhf(low[(size_t)(m0 + r) * ldl + j0 + j]) : 0.f;
     }
     __syncthreads();
     if (c < C) {
-      for (int j = 0; j < nj; j += 8) {
-        float wv[8];
+      for (int j = 0; j < nj; j += 4) {
+        float wv[4][VEC];      // four rows of w2 are asked for before the first is used
 #pragma unroll
-        for (int q = 0; q < 8; q++) wv[q] = j + q < nj ? w2[(size_t)(j0 + j + q) * C + c] : 0.f;
+        for (int q = 0; q < 4; q++) {
+          if (j + q < nj) get(wv[q], w2 + (size_t)(j0 + j + q) * C + c);
+          else
 #pragma unroll
-        for (int q = 0; q < 8; q++)
+            for (int e = 0; e < VEC; e++) wv[q][e] = 0.f;
+        }
+#pragma unroll
+        for (int q = 0; q < 4; q++)
           if (j + q < nj)
 #pragma unroll
-            for (int r = 0; r < R; r++) acc[r] = fmaf(ts[j + q][r], wv[q], acc[r]);
+            for (int r = 0; r < R; r++) {
+              const float t = ts[j + q][r];
+#pragma unroll
+              for (int e = 0; e < VEC; e++) acc[r][e] = fmaf(t, wv[q][e], acc[r][e]);
+            }
       }
     }
   }
   if (c >= C) return;
-  const float z0 = w0[c];
+  float z0[VEC];
+  get(z0, w0 + c);
 #pragma unroll
-  for (int r = 0; r < R; r++)
-    if (m0 + r < M) out[(size_t)(m0 + r) * C + c] = expf(-expf(acc[r] + z0));
+  for (int r = 0; r < R; r++) {
+    if (m0 + r >= M) break;
+    float o[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; e++) o[e] = expf(-expf(acc[r][e] + z0[e]));
+    float* dst = out + (size_t)(m0 + r) * C + c;
+    if (VEC == 4) store4(dst, make_float4(o[0], o[1 % VEC], o[2 % VEC], o[3 % VEC]));
+    else *dst = o[0];
+  }
 }
 
 LEB_API int leb_low_rank_decay(float* out, const float* low, int ldl, const float* w2, const float* w0, int M, int C, int rank,
@@ -175,13 +202,14 @@ LEB_API int leb_low_rank_decay(float* out, const float* low, int ldl, const floa
   if (M <= 0 || C <= 0) return 0;
   LEB_REQUIRE(rank >= 1, "leb_low_rank_decay: a rank of %d", rank);
   LebPlainLaunches plain(true);
-  const dim3 block(128);
-  if (M > 16) {
-    const dim3 grid(ceil_div(M, LRD_ROWS), ceil_div(C, 128));
-    leb_launch(low_rank_decay_kernel<LRD_ROWS>, grid, block, 0, st, out, low, ldl, w2, w0, M, C, rank);
-  } else {
-    leb_launch(low_rank_decay_kernel<1>, dim3(M, ceil_div(C, 128)), block, 0, st, out, low, ldl, w2, w0, M, C, rank);
-  }
+  const bool vec = C % 4 == 0 && (((uintptr_t)out | (uintptr_t)w2 | (uintptr_t)w0) & 15) == 0;
+#define LEB_LRD(R_, V_) \
+  leb_launch(low_rank_decay_kernel<R_, V_>, dim3(ceil_div(M, R_), ceil_div(C, 128 * V_)), dim3(128), 0, st, out, low, ldl, w2, w0, M, C, rank)
+  // a few rows: a channel a thread, so that a decode step has blocks for more SMs
+  if (M <= 16) LEB_LRD(1, 1);
+  else if (vec) LEB_LRD(8, 4);
+  else LEB_LRD(8, 1);
+#undef LEB_LRD
   LEB_CHECK_LAUNCH("leb_low_rank_decay");
   return 0;
 }
